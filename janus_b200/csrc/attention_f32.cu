@@ -10,6 +10,8 @@
 // 32 keys that start at multiples of 32 of the absolute key index, so a
 // token's result does not depend on how its sequence was cut into steps.
 //
+// The values may be the first `vd` numbers of rows of hd numbers (latent attention: a row is key and value at once).
+//
 // Cache layout of one layer: [page][kv_head][PAGE][hd]; block_table[slot][i] is
 // the page of keys [i*PAGE, (i+1)*PAGE) of the sequence in `slot`.
 #include <math_constants.h>
@@ -20,16 +22,17 @@
 namespace {
 
 constexpr int WARPS = 4;
-constexpr int MAX_HD = 256;
+constexpr int SMALL_HD = 256, MAX_HD = 1280;
 
-// VEC: head sizes that are multiples of 4 (16-byte loads of the keys).
-template <bool VEC>
+// VEC: head sizes that are multiples of 4 (16-byte loads of the keys).  HDM bounds the head size; U value rows are
+// loaded at a time.
+template <bool VEC, int HDM, int U>
 __global__ void __launch_bounds__(WARPS * 32) attention_f32_kernel(
     const float* __restrict__ q, const float* __restrict__ k_cache, const float* __restrict__ v_cache,
     float* __restrict__ out, const int* __restrict__ block_table, const int* __restrict__ token_slot,
-    const int* __restrict__ positions, int T, int nh, int nkv, int hd, int page_size, int max_pages,
+    const int* __restrict__ positions, int T, int nh, int nkv, int hd, int vd, int page_size, int max_pages,
     int window, float scale, int chunk, float softcap, float sink) {
-  __shared__ __align__(16) float q_s[WARPS][MAX_HD];
+  __shared__ __align__(16) float q_s[WARPS][HDM];
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const long long item = (long long)blockIdx.x * WARPS + warp;
   if (item >= (long long)T * nh) return;  // whole warp leaves together
@@ -45,9 +48,9 @@ __global__ void __launch_bounds__(WARPS * 32) attention_f32_kernel(
   __syncwarp();
 
   float m = -CUDART_INF_F, l = 0.0f;
-  float acc[MAX_HD / 32];
+  float acc[HDM / 32];
 #pragma unroll
-  for (int j = 0; j < MAX_HD / 32; ++j) acc[j] = 0.0f;
+  for (int j = 0; j < HDM / 32; ++j) acc[j] = 0.0f;
 
   for (int c0 = (kstart / 32) * 32; c0 <= pos; c0 += 32) {
     const int key = c0 + lane;
@@ -80,42 +83,42 @@ __global__ void __launch_bounds__(WARPS * 32) attention_f32_kernel(
     const float corr = expf(m - m_new);  // exp(-inf) = 0 on the first chunk
     l = l * corr + jb::warp_sum(p);
 #pragma unroll
-    for (int j = 0; j < MAX_HD / 32; ++j) acc[j] *= corr;
+    for (int j = 0; j < HDM / 32; ++j) acc[j] *= corr;
     const int n_keys = min(32, pos - c0 + 1);
-    // eight value rows are loaded before their products are added, in key order (the same sums as one by one,
-    // with eight rows' latencies at a time instead of one)
+    // several value rows are loaded before their products are added, in key order (the same sums as one by one,
+    // with the rows' latencies side by side)
     const int first = max(c0, kstart) - c0;
-    for (int kk0 = first; kk0 < n_keys; kk0 += 8) {
-      float vreg[8][MAX_HD / 32];
+    for (int kk0 = first; kk0 < n_keys; kk0 += U) {
+      float vreg[U][HDM / 32];
 #pragma unroll
-      for (int u = 0; u < 8; ++u) {
+      for (int u = 0; u < U; ++u) {
         const int key2 = c0 + min(kk0 + u, n_keys - 1);
         const int page = pages[key2 / page_size], row = key2 % page_size;
         const float* vr = v_cache + (((size_t)page * nkv + kvh) * page_size + row) * hd;
 #pragma unroll
-        for (int j = 0; j < MAX_HD / 32; ++j) {
+        for (int j = 0; j < HDM / 32; ++j) {
           const int d = lane + 32 * j;
-          vreg[u][j] = d < hd ? vr[d] : 0.0f;
+          vreg[u][j] = d < vd ? vr[d] : 0.0f;
         }
       }
 #pragma unroll
-      for (int u = 0; u < 8; ++u) {
+      for (int u = 0; u < U; ++u) {
         if (kk0 + u < n_keys) {   // uniform across the warp
           const float pk = __shfl_sync(0xffffffffu, p, kk0 + u);
 #pragma unroll
-          for (int j = 0; j < MAX_HD / 32; ++j)
-            if (lane + 32 * j < hd) acc[j] = fmaf(pk, vreg[u][j], acc[j]);
+          for (int j = 0; j < HDM / 32; ++j)
+            if (lane + 32 * j < vd) acc[j] = fmaf(pk, vreg[u][j], acc[j]);
         }
       }
     }
     m = m_new;
   }
   if (sink > 0.0f) l += sink * expf(m == -CUDART_INF_F ? 0.0f : -m);
-  float* o = out + ((size_t)t * nh + h) * hd;
+  float* o = out + ((size_t)t * nh + h) * vd;
 #pragma unroll
-  for (int j = 0; j < MAX_HD / 32; ++j) {
+  for (int j = 0; j < HDM / 32; ++j) {
     const int d = lane + 32 * j;
-    if (d < hd) o[d] = acc[j] / l;
+    if (d < vd) o[d] = acc[j] / l;
   }
 }
 
@@ -123,21 +126,28 @@ __global__ void __launch_bounds__(WARPS * 32) attention_f32_kernel(
 
 JB_EXPORT int jb_attention_f32(const float* q, const float* k_cache, const float* v_cache, float* out,
                                const int* block_table, const int* token_slot, const int* positions, int T,
-                               int nh, int nkv, int hd, int page_size, int max_pages, int window, float scale,
+                               int nh, int nkv, int hd, int vd, int page_size, int max_pages, int window, float scale,
                                int chunk, float softcap, float sink, cudaStream_t stream) {
   if (T <= 0) return 0;
-  JB_REFUSE(hd > MAX_HD || hd <= 0, "attention_f32: head_dim %d is outside (0, %d]", hd, MAX_HD);
+  JB_REFUSE(hd > MAX_HD || hd <= 0 || vd <= 0 || vd > hd, "attention_f32: head_dim %d is outside (0, %d], or its values (%d) are wider",
+            hd, MAX_HD, vd);
   JB_REFUSE(nkv <= 0 || nh % nkv != 0, "attention_f32: %d heads are not a multiple of %d kv heads", nh, nkv);
   const long long items = (long long)T * nh;
   const unsigned blocks = (unsigned)((items + WARPS - 1) / WARPS);
-  if (hd % 4 == 0 && (((uintptr_t)k_cache) & 15) == 0)
-    attention_f32_kernel<true><<<blocks, WARPS * 32, 0, stream>>>(q, k_cache, v_cache, out, block_table, token_slot,
-                                                                  positions, T, nh, nkv, hd, page_size, max_pages,
-                                                                  window, scale, chunk, softcap, sink);
-  else
-    attention_f32_kernel<false><<<blocks, WARPS * 32, 0, stream>>>(q, k_cache, v_cache, out, block_table, token_slot,
-                                                                   positions, T, nh, nkv, hd, page_size, max_pages,
-                                                                   window, scale, chunk, softcap, sink);
+  const bool vec = hd % 4 == 0 && (((uintptr_t)k_cache) & 15) == 0;
+#define JB_GO(VEC, HDM, U)                                                                                         \
+  attention_f32_kernel<VEC, HDM, U><<<blocks, WARPS * 32, 0, stream>>>(q, k_cache, v_cache, out, block_table,      \
+                                                                       token_slot, positions, T, nh, nkv, hd, vd,  \
+                                                                       page_size, max_pages, window, scale, chunk, \
+                                                                       softcap, sink)
+  if (hd <= SMALL_HD) {
+    if (vec) JB_GO(true, SMALL_HD, 8);
+    else JB_GO(false, SMALL_HD, 8);
+  } else {
+    if (vec) JB_GO(true, MAX_HD, 2);
+    else JB_GO(false, MAX_HD, 2);
+  }
+#undef JB_GO
   JB_CHECK_LAUNCH();
   return 0;
 }

@@ -1,10 +1,12 @@
 // Causal grouped-query flash attention for prefill on the 5th-generation tensor
-// cores (tcgen05) of sm_100a, over the paged cache.  Built for a row of 64, 128 or 256 dims in shared memory
-// (-DJB_HEAD_DIM; rows of 256 have the one-tile kernel only, with a ring of two pages: O alone takes 256
-// columns of tensor memory); the head size itself is an argument, any multiple of 8 up to that: the tensor maps
+// cores (tcgen05) of sm_100a, over the paged cache, or over keys and values that lie in one matrix (a row per
+// token, the heads' keys side by side, then the heads' values; latent attention makes such a matrix for a step).
+// Built for a row of 64, 128, 192 or 256 dims in shared memory
+// (-DJB_HEAD_DIM; rows above 128 have the one-tile kernel only, rows of 256 with a ring of two pages: O alone takes
+// 256 columns of tensor memory); the head size itself is an argument, any multiple of 8 up to that: the tensor maps
 // have the true extent, so the copy engine fills the rest of a row with zeros, the score product skips
-// the 16-dim steps that are all zero, the P.V product has N = the head size rounded up to 16, and the
-// epilogue stores the true columns only.  Any number of query heads per kv head up to 128: a tile holds
+// the 16-dim steps that are all zero, the P.V product has N = the value size (at most the head size) rounded up
+// to 16, and the epilogue stores the true columns only.  Any number of query heads per kv head up to 128: a tile holds
 // floor(128 / G) tokens x G heads, and the rows left over (2 of 128 with 3, 6 or 7 heads per kv head)
 // belong to no token.
 //
@@ -43,11 +45,11 @@ namespace {
 typedef __nv_bfloat16 bf16;
 
 constexpr int HD = JB_HEAD_DIM;
-static_assert(HD == 64 || HD == 128 || HD == 256, "the tcgen05 attention kernel is built for rows of 64, 128 or 256 dims");
+static_assert(HD == 64 || HD == 128 || HD == 192 || HD == 256, "the tcgen05 attention kernel is built for rows of 64, 128, 192 or 256 dims");
 constexpr int NH64 = HD / 64;          // 64-column halves of a row
 constexpr int BM = 128;                // rows per CTA = TMEM lanes
 constexpr int PAGE = 64;               // keys per block
-constexpr int STAGES = HD > 128 ? 2 : 3;
+constexpr int STAGES = HD > 192 ? 2 : 3;
 constexpr int MAX_NT = 1;              // row tiles per CTA of prefill_tc_kernel<NT> (written for 1 or 2; 1 is what runs)
 constexpr int threads_for(int nt) { return 64 + nt * 128; }
 constexpr int Q_BYTES = NH64 * BM * 128;
@@ -277,6 +279,14 @@ struct Cap {
   int chunk;
   float cap_s, inv_cap, sink;
 };
+// Where keys and values lie.  start null: in pages.  Else in a matrix: the key of position p of sequence s is row
+// start[s] + p, head h's key begins at column h hd of the keys' map and its value at column h vd of the values' map.
+// (A 64-column box at a head's end may take in the head behind: those columns of Q are zeros, those of O unused.)
+// Heads have vd <= hd value numbers.
+struct Keys {
+  const int* start;
+  int vd;
+};
 __device__ __forceinline__ int chunk_lo(int lo, int pos, int chunk) {
   return (chunk > 0 && pos >= 0) ? max(lo, (pos / chunk) * chunk) : lo;
 }
@@ -295,7 +305,7 @@ __global__ void __launch_bounds__(threads_for(NT), 1) prefill_tc_kernel(
     const __grid_constant__ CUtensorMap map_q, const __grid_constant__ CUtensorMap map_k,
     const __grid_constant__ CUtensorMap map_v, bf16* __restrict__ out, const int* __restrict__ block_table,
     const int* __restrict__ q_start, const int* __restrict__ kv_len, int nh, int nkv, int hd, int max_pages, int window,
-    float scale_log2, int heads_slowest, int* __restrict__ status, Cap cap) {
+    float scale_log2, int heads_slowest, int* __restrict__ status, Cap cap, Keys keys) {
   // S of tile w: two buffers of 64 columns at w * 128; O behind them (HD columns a tile; 512 in all for rows of 256)
   constexpr int N_BARS = bars_for(NT), TMEM_COLS = HD > 128 ? 512 : NT * 256, TMEM_S0 = 0, TMEM_O0 = NT * 128;
   static_assert(NT * 128 + NT * HD <= TMEM_COLS, "tensor memory of one CTA");
@@ -369,28 +379,29 @@ __global__ void __launch_bounds__(threads_for(NT), 1) prefill_tc_kernel(
   if (active && warp == 0) {
     // ---------------- producer ----------------
     if (lane == 0) {
-      mbar_expect_tx(q_full, NT * NH64 * tpt * G * 128);   // the box holds tpt tokens x G heads: its bytes, not the tile's
+      const int nk64 = (hd + 63) / 64, nv64 = (keys.vd + 63) / 64;   // 64-column slabs that hold anything
+      const int xk = keys.start ? kvh * hd : 0, xv = keys.start ? kvh * keys.vd : 0;
+      const int dense0 = keys.start ? keys.start[seq] : 0;
+      mbar_expect_tx(q_full, NT * nk64 * tpt * G * 128);   // the box holds tpt tokens x G heads: its bytes, not the tile's
       for (int w = 0; w < NT; ++w)   // a tile past the sequence's end reads rows that no one uses (or zeros past the tensor)
-        for (int h = 0; h < NH64; ++h)
+        for (int h = 0; h < nk64; ++h)
           tma_load_4d(q_s + w * Q_BYTES + h * BM * 128, &map_q, q_full, h * 64, 0, kvh, qs + tok_first + w * tpt);
       const int* pages = block_table + (size_t)seq * max_pages;
       for (int j = 0; j < nb; ++j) {
         const int s = j % STAGES;
         if (j >= STAGES && !mbar_wait(kv_empty + 8 * s, ((j / STAGES) - 1) & 1, status, 11)) break;
         const uint32_t bar = kv_full + 8 * s, stage = kv_s + s * STAGE_BYTES;
-        mbar_expect_tx(bar, STAGE_BYTES);
-        const int row0 = (pages[kb_start + j] * nkv + kvh) * PAGE;
-        for (int h = 0; h < NH64; ++h) {
-          tma_load_2d(stage + h * PAGE * 128, &map_k, bar, h * 64, row0);
-          tma_load_2d(stage + K_BYTES + h * PAGE * 128, &map_v, bar, h * 64, row0);
-        }
+        mbar_expect_tx(bar, (nk64 + nv64) * PAGE * 128);
+        const int row0 = keys.start ? dense0 + (kb_start + j) * PAGE : (pages[kb_start + j] * nkv + kvh) * PAGE;
+        for (int h = 0; h < nk64; ++h) tma_load_2d(stage + h * PAGE * 128, &map_k, bar, xk + h * 64, row0);
+        for (int h = 0; h < nv64; ++h) tma_load_2d(stage + K_BYTES + h * PAGE * 128, &map_v, bar, xv + h * 64, row0);
       }
     }
   } else if (active && warp == 1) {
     // ---------------- MMA issuer ----------------
     if (lane == 0) {
       constexpr uint32_t idesc_s = instr_desc(PAGE, 0);
-      const uint32_t idesc_o = instr_desc((hd + 15) & ~15, 1);
+      const uint32_t idesc_o = instr_desc((keys.vd + 15) & ~15, 1);
       bool ok = mbar_wait(q_full, 0, status, 12);
       auto issue_s = [&](int j) -> bool {
         const int s = j % STAGES, b = j & 1;
@@ -474,7 +485,7 @@ __global__ void __launch_bounds__(threads_for(NT), 1) prefill_tc_kernel(
           const float corr = m_new == -CUDART_INF_F ? 1.0f : exp2f(m_ref - m_new);  // 0 if nothing was seen before
 #pragma unroll
           for (int c0 = 0; c0 < HD; c0 += 16) {
-            if (c0 >= hd) break;
+            if (c0 >= keys.vd) break;
             uint32_t r[16];
             tmem_ld16(lane_addr + o_col + c0, r);
             tmem_ld_wait();
@@ -500,10 +511,10 @@ __global__ void __launch_bounds__(threads_for(NT), 1) prefill_tc_kernel(
       tc_fence_after();
       if (cap.sink > 0.0f) l += cap.sink * exp2f(m_ref == -CUDART_INF_F ? 0.0f : -m_ref);
       const float inv = 1.0f / l;
-      bf16* dst = out + ((size_t)(qs + tok_first + (valid ? tl : 0)) * nh + kvh * G + row % G) * hd;
+      bf16* dst = out + ((size_t)(qs + tok_first + (valid ? tl : 0)) * nh + kvh * G + row % G) * keys.vd;
 #pragma unroll
       for (int c0 = 0; c0 < HD; c0 += 16) {
-        if (c0 >= hd) break;
+        if (c0 >= keys.vd) break;
         uint32_t r[16];
         tmem_ld16(lane_addr + o_col + c0, r);   // warp-wide: rows without a token load too and store nothing
         tmem_ld_wait();
@@ -518,7 +529,7 @@ __global__ void __launch_bounds__(threads_for(NT), 1) prefill_tc_kernel(
           w1.z = pack_bf16(__uint_as_float(r[12]) * inv, __uint_as_float(r[13]) * inv);
           w1.w = pack_bf16(__uint_as_float(r[14]) * inv, __uint_as_float(r[15]) * inv);
           *reinterpret_cast<uint4*>(dst + c0) = w0;
-          if (c0 + 8 < hd) *reinterpret_cast<uint4*>(dst + c0 + 8) = w1;
+          if (c0 + 8 < keys.vd) *reinterpret_cast<uint4*>(dst + c0 + 8) = w1;
         }
       }
     }
@@ -552,7 +563,7 @@ __global__ void __launch_bounds__(T2_THREADS, 1) prefill_tc128_kernel(
     const __grid_constant__ CUtensorMap map_q, const __grid_constant__ CUtensorMap map_k,
     const __grid_constant__ CUtensorMap map_v, bf16* __restrict__ out, const int* __restrict__ block_table,
     const int* __restrict__ q_start, const int* __restrict__ kv_len, int nh, int nkv, int hd, int max_pages, int window,
-    float scale_log2, int heads_slowest, int* __restrict__ status, Cap cap) {
+    float scale_log2, int heads_slowest, int* __restrict__ status, Cap cap, Keys keys) {
   extern __shared__ uint8_t smem_raw[];
   uint8_t* smem = (uint8_t*)(((uintptr_t)smem_raw + 1023) & ~(uintptr_t)1023);
   const uint32_t q_s = smem_u32(smem);
@@ -616,34 +627,39 @@ __global__ void __launch_bounds__(T2_THREADS, 1) prefill_tc128_kernel(
   if (active && warp == 0) {
     // ---------------- producer ----------------
     if (lane == 0) {
-      mbar_expect_tx(q_full, 2 * NH64 * tpt * G * 128);   // the box holds tpt tokens x G heads: its bytes, not the tile's
+      const int nk64 = (hd + 63) / 64, nv64 = (keys.vd + 63) / 64;   // 64-column slabs that hold anything
+      const int xk = keys.start ? kvh * hd : 0, xv = keys.start ? kvh * keys.vd : 0;
+      const int dense0 = keys.start ? keys.start[seq] : 0;
+      mbar_expect_tx(q_full, 2 * nk64 * tpt * G * 128);   // the box holds tpt tokens x G heads: its bytes, not the tile's
       for (int w = 0; w < 2; ++w)
-        for (int h = 0; h < NH64; ++h)
+        for (int h = 0; h < nk64; ++h)
           tma_load_4d(q_s + w * Q_BYTES + h * BM * 128, &map_q, q_full, h * 64, 0, kvh, qs + tok_first + w * tpt);
       const int* pages = block_table + (size_t)seq * max_pages;
       for (int j = 0; j < nb; ++j) {
         const int st = j & 1;
         // a block's second page may lie past the sequence's end: its keys are masked, any finite data will do
         int row0[2];
-        for (int half = 0; half < 2; ++half)
-          row0[half] = (pages[min(2 * (kb_start + j) + half, last_page)] * nkv + kvh) * PAGE;
+        for (int half = 0; half < 2; ++half) {
+          const int page = min(2 * (kb_start + j) + half, last_page);
+          row0[half] = keys.start ? dense0 + page * PAGE : (pages[page] * nkv + kvh) * PAGE;
+        }
         if (j >= 2 && !mbar_wait(k_empty + 8 * st, ((j >> 1) - 1) & 1, status, 11)) break;
-        mbar_expect_tx(k_full + 8 * st, K128_BYTES);
+        mbar_expect_tx(k_full + 8 * st, nk64 * KB * 128);
         for (int half = 0; half < 2; ++half)
-          for (int h = 0; h < NH64; ++h)
-            tma_load_2d(k_s + st * K128_BYTES + h * KB * 128 + half * PAGE * 128, &map_k, k_full + 8 * st, h * 64, row0[half]);
+          for (int h = 0; h < nk64; ++h)
+            tma_load_2d(k_s + st * K128_BYTES + h * KB * 128 + half * PAGE * 128, &map_k, k_full + 8 * st, xk + h * 64, row0[half]);
         if (j >= 2 && !mbar_wait(v_empty + 8 * st, ((j >> 1) - 1) & 1, status, 11)) break;
-        mbar_expect_tx(v_full + 8 * st, K128_BYTES);
+        mbar_expect_tx(v_full + 8 * st, nv64 * KB * 128);
         for (int half = 0; half < 2; ++half)
-          for (int h = 0; h < NH64; ++h)
-            tma_load_2d(v_s + st * K128_BYTES + h * KB * 128 + half * PAGE * 128, &map_v, v_full + 8 * st, h * 64, row0[half]);
+          for (int h = 0; h < nv64; ++h)
+            tma_load_2d(v_s + st * K128_BYTES + h * KB * 128 + half * PAGE * 128, &map_v, v_full + 8 * st, xv + h * 64, row0[half]);
       }
     }
   } else if (active && warp == 1) {
     // ---------------- MMA issuer ----------------
     if (lane == 0) {
       constexpr uint32_t idesc_s = instr_desc(KB, 0);
-      const uint32_t idesc_o = instr_desc((hd + 15) & ~15, 1);
+      const uint32_t idesc_o = instr_desc((keys.vd + 15) & ~15, 1);
       bool ok = mbar_wait(q_full, 0, status, 12);
       auto issue_s = [&](int w, int j) -> bool {
         const int st = j & 1;
@@ -723,7 +739,7 @@ __global__ void __launch_bounds__(T2_THREADS, 1) prefill_tc128_kernel(
           const float corr = m_new == -CUDART_INF_F ? 1.0f : exp2f(m_ref - m_new);
 #pragma unroll
           for (int c0 = 0; c0 < HD; c0 += 16) {
-            if (c0 >= hd) break;
+            if (c0 >= keys.vd) break;
             uint32_t r[16];
             tmem_ld16(lane_addr + o_col + c0, r);
             tmem_ld_wait();
@@ -748,10 +764,10 @@ __global__ void __launch_bounds__(T2_THREADS, 1) prefill_tc128_kernel(
       tc_fence_after();
       if (cap.sink > 0.0f) l += cap.sink * exp2f(m_ref == -CUDART_INF_F ? 0.0f : -m_ref);
       const float inv = 1.0f / l;
-      bf16* dst = out + ((size_t)(qs + tok_first + (valid ? tl : 0)) * nh + kvh * G + row % G) * hd;
+      bf16* dst = out + ((size_t)(qs + tok_first + (valid ? tl : 0)) * nh + kvh * G + row % G) * keys.vd;
 #pragma unroll
       for (int c0 = 0; c0 < HD; c0 += 16) {
-        if (c0 >= hd) break;
+        if (c0 >= keys.vd) break;
         uint32_t r[16];
         tmem_ld16(lane_addr + o_col + c0, r);
         tmem_ld_wait();
@@ -766,7 +782,7 @@ __global__ void __launch_bounds__(T2_THREADS, 1) prefill_tc128_kernel(
           w1.z = pack_bf16(__uint_as_float(r[12]) * inv, __uint_as_float(r[13]) * inv);
           w1.w = pack_bf16(__uint_as_float(r[14]) * inv, __uint_as_float(r[15]) * inv);
           *reinterpret_cast<uint4*>(dst + c0) = w0;
-          if (c0 + 8 < hd) *reinterpret_cast<uint4*>(dst + c0 + 8) = w1;
+          if (c0 + 8 < keys.vd) *reinterpret_cast<uint4*>(dst + c0 + 8) = w1;
         }
       }
     }
@@ -804,10 +820,11 @@ JB_EXPORT int jb_attention_tc_head_dim() { return HD; }
 // q, out: [T, nh * hd] bf16; caches: [n_pages, nkv, 64, hd] bf16.  Needs nh / nkv <= 128 and a head size
 // that is a multiple of 8 (rows of 16 bytes for the tensor maps) up to the build's row.
 namespace {
+// kv_rows > 0: keys and values are the matrix at k_cache ([kv_rows] rows of nkv (hd + vd) numbers), see `Keys`
 int tc_prefill_launch(const void* q, const void* k_cache, const void* v_cache, void* out, const int* block_table,
                       const int* q_start, const int* kv_len, int T, int n_pages, int n_seqs, int max_q_len, int nh,
                       int nkv, int hd, int page_size, int max_pages, int window, float scale, const Cap& cap,
-                      int* status, cudaStream_t stream) {
+                      int* status, cudaStream_t stream, const Keys& keys, int kv_rows = 0) {
   if (n_seqs <= 0 || max_q_len <= 0 || T <= 0) return 0;
   JB_REFUSE(hd <= 0 || hd > HD || hd % 8 != 0,
             "attention_tc: built for head sizes up to %d in steps of 8, called with %d", HD, hd);
@@ -832,8 +849,10 @@ int tc_prefill_launch(const void* q, const void* k_cache, const void* v_cache, v
       return JB_ERR_TENSORMAP;
   }
   for (int which = 0; which < 2; ++which) {
-    const cuuint64_t dims[2] = {(cuuint64_t)hd, (cuuint64_t)n_pages * nkv * PAGE};
-    const cuuint64_t strides[1] = {(cuuint64_t)hd * 2};
+    const int width = which ? keys.vd : hd;
+    const cuuint64_t dims[2] = {(cuuint64_t)(kv_rows ? nkv * width : width),
+                                kv_rows ? (cuuint64_t)kv_rows : (cuuint64_t)n_pages * nkv * PAGE};
+    const cuuint64_t strides[1] = {(cuuint64_t)(kv_rows ? nkv * (hd + keys.vd) : width) * 2};
     const cuuint32_t box[2] = {64, PAGE};
     const cuuint32_t el[2] = {1, 1};
     if (enc(which ? &mv : &mk, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, const_cast<void*>(which ? v_cache : k_cache), dims,
@@ -871,13 +890,13 @@ int tc_prefill_launch(const void* q, const void* k_cache, const void* v_cache, v
     dim3 grid(heads_slowest ? n_pairs : nkv, heads_slowest ? nkv : n_pairs, n_seqs);
     jb::Launch cfg(grid, dim3(T2_THREADS), T2_SMEM, stream);
     return (int)cudaLaunchKernelEx(&cfg.c, prefill_tc128_kernel, mq, mk, mv, (bf16*)out, block_table, q_start, kv_len, nh,
-                                   nkv, hd, max_pages, window, scale * LOG2E, heads_slowest ? 1 : 0, status, cap);
+                                   nkv, hd, max_pages, window, scale * LOG2E, heads_slowest ? 1 : 0, status, cap, keys);
   }
 #endif
   dim3 grid(heads_slowest ? n_tiles : nkv, heads_slowest ? nkv : n_tiles, n_seqs);
   jb::Launch cfg(grid, dim3(threads_for(1)), smem_for(1), stream);
   return (int)cudaLaunchKernelEx(&cfg.c, prefill_tc_kernel<1>, mq, mk, mv, (bf16*)out, block_table, q_start, kv_len, nh,
-                                 nkv, hd, max_pages, window, scale * LOG2E, heads_slowest ? 1 : 0, status, cap);
+                                 nkv, hd, max_pages, window, scale * LOG2E, heads_slowest ? 1 : 0, status, cap, keys);
 }
 }  // namespace
 
@@ -887,7 +906,7 @@ JB_EXPORT int jb_attention_tc_prefill(const void* q, const void* k_cache, const 
                                       int page_size, int max_pages, int window, float scale, int* status,
                                       cudaStream_t stream) {
   return tc_prefill_launch(q, k_cache, v_cache, out, block_table, q_start, kv_len, T, n_pages, n_seqs, max_q_len, nh,
-                           nkv, hd, page_size, max_pages, window, scale, Cap{0, 0.0f, 0.0f}, status, stream);
+                           nkv, hd, page_size, max_pages, window, scale, Cap{0, 0.0f, 0.0f}, status, stream, Keys{nullptr, hd});
 }
 
 // As jb_attention_tc_prefill, with a chunked mask (chunk > 0: a query sees only the keys of its own chunk of
@@ -901,5 +920,18 @@ JB_EXPORT int jb_attention_tc_prefill_capped(const void* q, const void* k_cache,
   JB_REFUSE(chunk < 0 || softcap < 0.0f || scale <= 0.0f, "attention_tc: a chunk, a cap and a scale cannot be negative");
   const Cap cap = softcap > 0.0f ? Cap{chunk, softcap / scale, scale / softcap, sink} : Cap{chunk, 0.0f, 0.0f, sink};
   return tc_prefill_launch(q, k_cache, v_cache, out, block_table, q_start, kv_len, T, n_pages, n_seqs, max_q_len, nh,
-                           nkv, hd, page_size, max_pages, window, scale, cap, status, stream);
+                           nkv, hd, page_size, max_pages, window, scale, cap, status, stream, Keys{nullptr, hd});
+}
+
+// Causal attention with a key and a value head per query head, keys and values in one matrix kv [kv_rows][nh hd | nh vd]
+// (bfloat16): the key of position p of sequence s is row kv_start[s] + p.  q: [T, nh hd], out: [T, nh vd]; hd and vd are
+// multiples of 8, vd <= hd <= the build's row.  max_kv_len bounds a sequence's length (it picks the order of the blocks).
+JB_EXPORT int jb_attention_tc_matrix(const void* q, const void* kv, void* out, const int* kv_start, const int* q_start,
+                                     const int* kv_len, int T, int kv_rows, int n_seqs, int max_q_len, int nh, int hd, int vd,
+                                     int max_kv_len, float scale, int* status, cudaStream_t stream) {
+  JB_REFUSE(vd <= 0 || vd > hd || vd % 8 != 0 || kv_rows <= 0 || kv_start == nullptr,
+            "attention_tc: values of %d numbers beside keys of %d, in %d rows", vd, hd, kv_rows);
+  return tc_prefill_launch(q, kv, (const bf16*)kv + (size_t)nh * hd, out, nullptr, q_start, kv_len, T, 0, n_seqs, max_q_len,
+                           nh, nh, hd, PAGE, (max_kv_len + PAGE - 1) / PAGE, 0, scale, Cap{0, 0.0f, 0.0f}, status, stream,
+                           Keys{kv_start, vd}, kv_rows);
 }

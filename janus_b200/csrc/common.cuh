@@ -110,6 +110,9 @@ __device__ __forceinline__ float gated(float g, float u, const Gate& gate) {
   return g * (1.0f / (1.0f + expf(-g))) * u;
 }
 
+// GELU by the normal distribution's own integral, 0.5 z (1 + erf(z / sqrt(2))).
+__device__ __forceinline__ float gelu_erf(float z) { return 0.5f * z * (1.0f + erff(z * 0.70710678118654752f)); }
+
 __device__ __forceinline__ float warp_sum(float v) {
 #pragma unroll
   for (int o = 16; o > 0; o >>= 1) v += __shfl_xor_sync(0xffffffffu, v, o);

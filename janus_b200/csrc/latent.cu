@@ -1,0 +1,461 @@
+// Latent attention with a rotated part: what happens around the attention kernels.  Per token a place caches one row
+// [c | p]: the latent c (n numbers, normed) and a key part p (r numbers, rotated) that all heads share; a head's key is
+// [Wuk_h c | p], its value Wuv_h c.  All arithmetic is float32 on the projections' float32 accumulators
+//
+//   proj [T, ld]:  q at q_col (H heads of d unrotated then r rotated numbers), the row's projection at c_col (n + r)
+//
+//   latent_prep      queries as heads: q_out[t, h] = [q | turned q], for attention over keys and values per head;
+//                    the token's row is normed, turned and appended to the pages (and to `rows` [T, stored], if given)
+//   latent_queries   queries in the latents' space: q_out[t, h] = [Wuk_h^T q | turned q], so that the score with the
+//                    cached row itself is the head's score; the token's row as above
+//   latent_values    out[t, h] = Wuv_h o, o = sum_j p_j c_j the attention's output in the latents' space, from rows
+//                    [T, H, n] or straight from the partial sums that the splits of the keys left; times the sigmoid
+//                    of an output gate, if there is one
+//   gather_rows      the cached rows of a step's sequences, sequence after sequence, in one matrix
+//
+// The rotation turns the pair (i, i + r/2) by the position's angle; cos and sin come from a table [positions][r/2][2].
+// Pages of one place: [page][1][page_size][stored], stored >= n + r, extra columns never written (they stay zero).
+#include <math_constants.h>
+#include <stdio.h>
+
+#include "common.cuh"
+
+namespace {
+
+typedef __nv_bfloat16 bf16;
+
+struct Row {                 // the token's own row: where it comes from and where it goes (c_cache null: none)
+  int c_col, n, r, stored;
+  const float* w;            // norm weight of the latent
+  float eps;
+  const int* dest;
+  void* c_cache;
+  void* rows;                // a second copy, row t of [T, stored] (null: none)
+};
+
+// One block norms, turns and writes the row of token t.
+template <typename TO>
+__device__ void write_row(const float* pr, const Row& row, const float* cs, int t, float* scratch) {
+  const float* x = pr + row.c_col;
+  float ss = 0.0f;
+  for (int i = threadIdx.x; i < row.n; i += blockDim.x) ss = fmaf(x[i], x[i], ss);
+  ss = jb::block_sum(ss, scratch);
+  const float inv = 1.0f / sqrtf(ss / (float)row.n + row.eps);
+  TO* out = (TO*)row.c_cache + (size_t)row.dest[t] * row.stored;
+  TO* copy = row.rows != nullptr ? (TO*)row.rows + (size_t)t * row.stored : nullptr;
+  const int half = row.r >> 1;
+  for (int i = threadIdx.x; i < row.stored; i += blockDim.x) {
+    float v;
+    if (i < row.n) {
+      v = (x[i] * inv) * row.w[i];
+    } else if (i < row.n + row.r) {
+      const int j = i - row.n;
+      v = x[i];
+      if (cs != nullptr) {
+        const int k = j < half ? j : j - half;
+        const float other = x[row.n + (j < half ? j + half : k)];
+        const float co = cs[2 * k], si = cs[2 * k + 1];
+        v = j < half ? v * co - other * si : v * co + other * si;
+      }
+    } else {
+      if (copy != nullptr) copy[i] = jb::from_f32<TO>(0.0f);
+      continue;
+    }
+    out[i] = jb::from_f32<TO>(v);
+    if (copy != nullptr) copy[i] = jb::from_f32<TO>(v);
+  }
+}
+
+template <typename TO>
+__device__ __forceinline__ void store4(TO* p, const float4& v) {
+  if constexpr (sizeof(TO) == 4) {
+    *reinterpret_cast<float4*>(p) = v;
+  } else {
+    const __nv_bfloat162 lo = __floats2bfloat162_rn(v.x, v.y), hi = __floats2bfloat162_rn(v.z, v.w);
+    uint2 u;
+    u.x = *reinterpret_cast<const uint32_t*>(&lo);
+    u.y = *reinterpret_cast<const uint32_t*>(&hi);
+    *reinterpret_cast<uint2*>(p) = u;
+  }
+}
+
+// Queries as heads (`dp` numbers each, the extra ones zero) and the token's row; one block per token.
+// VEC: d, r / 2, dp, the columns and the rows are whole groups of four at aligned addresses.
+template <typename TO, bool VEC>
+__global__ void __launch_bounds__(256) latent_prep_kernel(const float* __restrict__ proj, int ld, int q_col, int H, int d,
+                                                          int r, int dp, const float* __restrict__ table,
+                                                          const int* __restrict__ positions, TO* __restrict__ q_out,
+                                                          Row row) {
+  __shared__ float scratch[33];
+  jb::pdl_launch_dependents();
+  jb::pdl_wait();
+  const int t = blockIdx.x;
+  const float* pr = proj + (size_t)t * ld;
+  const int half = r >> 1;
+  const float* cs = table != nullptr && r > 0 ? table + (size_t)positions[t] * half * 2 : nullptr;
+  TO* q = q_out + (size_t)t * H * dp;
+  if constexpr (VEC) {
+    const int per = dp >> 2;                           // groups of four per stored head
+    for (int i = threadIdx.x; i < H * per; i += blockDim.x) {
+      const int h = i / per, j = (i - h * per) << 2;
+      const float* x = pr + q_col + (size_t)h * (d + r);
+      TO* o = q + (size_t)h * dp;
+      if (j < d || (j < d + r && cs == nullptr)) {
+        store4(o + j, *reinterpret_cast<const float4*>(x + j));
+      } else if (j < d + half) {
+        const float4 u = *reinterpret_cast<const float4*>(x + j), v = *reinterpret_cast<const float4*>(x + j + half);
+        const float4 a = *reinterpret_cast<const float4*>(cs + 2 * (j - d)), b = *reinterpret_cast<const float4*>(cs + 2 * (j - d) + 4);
+        store4(o + j, make_float4(u.x * a.x - v.x * a.y, u.y * a.z - v.y * a.w, u.z * b.x - v.z * b.y, u.w * b.z - v.w * b.w));
+        store4(o + j + half, make_float4(v.x * a.x + u.x * a.y, v.y * a.z + u.y * a.w, v.z * b.x + u.z * b.y, v.w * b.z + u.w * b.w));
+      } else if (j >= d + r) {
+        store4(o + j, make_float4(0.0f, 0.0f, 0.0f, 0.0f));
+      }
+    }
+  } else {
+    for (int i = threadIdx.x; i < H * dp; i += blockDim.x) {
+      const int h = i / dp, j = i - h * dp;
+      const float* x = pr + q_col + (size_t)h * (d + r);
+      float v = j < d + r ? x[j] : 0.0f;
+      if (j >= d && j < d + r && cs != nullptr) {
+        const int k = j - d < half ? j - d : j - d - half;
+        const float co = cs[2 * k], si = cs[2 * k + 1];
+        v = j - d < half ? v * co - x[j + half] * si : v * co + x[j - half] * si;
+      }
+      q[i] = jb::from_f32<TO>(v);
+    }
+  }
+  if (row.c_cache != nullptr) write_row<TO>(pr, row, cs, t, scratch);
+}
+
+// V numbers of a weight row as floats
+template <typename TW, int V>
+__device__ __forceinline__ void load_w(const TW* p, float (&v)[V]) {
+  if constexpr (V == 1) {
+    v[0] = jb::to_f32(*p);
+  } else if constexpr (sizeof(TW) == 2) {
+    const uint4 a = *reinterpret_cast<const uint4*>(p);
+    const uint32_t w[4] = {a.x, a.y, a.z, a.w};
+#pragma unroll
+    for (int i = 0; i < 4; ++i) {
+      v[2 * i] = __uint_as_float(w[i] << 16);
+      v[2 * i + 1] = __uint_as_float(w[i] & 0xffff0000u);
+    }
+  } else {
+    const float4 a = *reinterpret_cast<const float4*>(p);
+    v[0] = a.x, v[1] = a.y, v[2] = a.z, v[3] = a.w;
+  }
+}
+template <typename TW> struct Width { static constexpr int N = sizeof(TW) == 2 ? 8 : 4; };   // numbers in 16 bytes
+
+constexpr int QT = 8;             // tokens of a block of latent_queries
+constexpr int Q_THREADS = 128;
+
+// q_out[t, h, :n] = sum_j q[t, h, j] uk[h d + j, :], q_out[t, h, n : n + r] = the turned part, the rest zero; and, by
+// the blocks behind the heads' (blockIdx.x == H * chunks: one block per token tile), the tokens' rows.
+// A block owns (head, a chunk of COLS latent columns, QT tokens): COLS / V threads a row of uk, the others take other
+// rows j; the partial sums meet in shared memory.
+template <typename T, int V>
+__global__ void __launch_bounds__(Q_THREADS) latent_queries_kernel(
+    const float* __restrict__ proj, int ld, int q_col, int H, int d, int r, int n, int dp, const T* __restrict__ uk,
+    const float* __restrict__ table, const int* __restrict__ positions, T* __restrict__ q_out, int n_tokens, Row row) {
+  constexpr int CT = 8;                         // threads along the columns
+  constexpr int COLS = CT * V;
+  constexpr int SL = Q_THREADS / CT;            // slices of the rows j
+  extern __shared__ __align__(16) float sm[];   // q [QT][d], then the slices' sums [SL][QT][COLS]
+  __shared__ float scratch[33];
+  jb::pdl_launch_dependents();
+  jb::pdl_wait();
+  const int chunks = (n + COLS - 1) / COLS;
+  const int t0 = blockIdx.y * QT, nt = min(QT, n_tokens - t0);
+  const int half = r >> 1;
+  if (blockIdx.x == H * chunks) {
+    for (int k = 0; k < nt; ++k) {
+      const int t = t0 + k;
+      const float* cs = table != nullptr && r > 0 ? table + (size_t)positions[t] * half * 2 : nullptr;
+      write_row<T>(proj + (size_t)t * ld, row, cs, t, scratch);
+    }
+    return;
+  }
+  const int h = blockIdx.x / chunks, chunk = blockIdx.x - h * chunks;
+  float* q_s = sm;
+  float* part = sm + (QT * d + 3) / 4 * 4;
+  for (int i = threadIdx.x; i < nt * d; i += Q_THREADS)
+    q_s[i] = proj[(size_t)(t0 + i / d) * ld + q_col + (size_t)h * (d + r) + i % d];
+  if (chunk == 0) {                             // the turned part and the zero columns, once per head
+    const int extra = dp - n;
+    for (int i = threadIdx.x; i < nt * extra; i += Q_THREADS) {
+      const int t = t0 + i / extra, j = i % extra;
+      const float* x = proj + (size_t)t * ld + q_col + (size_t)h * (d + r) + d;
+      float v = j < r ? x[j] : 0.0f;
+      if (j < r && table != nullptr) {
+        const int k = j < half ? j : j - half;
+        const float* cs = table + ((size_t)positions[t] * half + k) * 2;
+        v = j < half ? v * cs[0] - x[j + half] * cs[1] : v * cs[0] + x[k] * cs[1];
+      }
+      q_out[((size_t)t * H + h) * dp + n + j] = jb::from_f32<T>(v);
+    }
+  }
+  __syncthreads();
+  const int ct = threadIdx.x % CT, sl = threadIdx.x / CT;
+  const int col = chunk * COLS + ct * V;
+  float acc[QT][V];
+#pragma unroll
+  for (int k = 0; k < QT; ++k)
+#pragma unroll
+    for (int v = 0; v < V; ++v) acc[k][v] = 0.0f;
+  if (col < n) {                                // with V > 1 n is a multiple of V: no column group is cut
+    const T* w = uk + (size_t)h * d * n + col;
+#pragma unroll 4
+    for (int j = sl; j < d; j += SL) {
+      float wv[V];
+      load_w<T, V>(w + (size_t)j * n, wv);
+#pragma unroll
+      for (int k = 0; k < QT; ++k) {
+        const float x = k < nt ? q_s[k * d + j] : 0.0f;
+#pragma unroll
+        for (int v = 0; v < V; ++v) acc[k][v] = fmaf(wv[v], x, acc[k][v]);
+      }
+    }
+  }
+#pragma unroll
+  for (int k = 0; k < QT; ++k)
+#pragma unroll
+    for (int v = 0; v < V; ++v) part[(sl * QT + k) * COLS + ct * V + v] = acc[k][v];
+  __syncthreads();
+  for (int i = threadIdx.x; i < nt * COLS; i += Q_THREADS) {
+    const int k = i / COLS, c = i % COLS;
+    if (chunk * COLS + c >= n) continue;
+    float v = 0.0f;
+#pragma unroll
+    for (int s = 0; s < SL; ++s) v += part[(s * QT + k) * COLS + c];
+    q_out[((size_t)(t0 + k) * H + h) * dp + chunk * COLS + c] = jb::from_f32<T>(v);
+  }
+}
+
+constexpr int VT = 4;              // tokens of a block of latent_values
+constexpr int V_WARPS = 8, V_ROWS = 8;
+
+// out[t, h, c] = (uv[h e + c, :] . o[t, h]) * sigmoid(gate[t, h e + c]) for c < e, zero for e <= c < ep.  o comes from
+// `o_rows` [T, H, n] (splits == 0), or from the key splits' partial sums: part_o [T, H, splits, n] and part_ml
+// [T, H, splits, 2] (maximum in units of log2, sum), o = sum_s f_s part_o[s] / sum_s f_s l_s with f_s = 2^(m_s - max).
+// A block owns (a chunk of V_WARPS * V_ROWS value rows, head, VT tokens); a warp takes rows one after another.
+template <typename T, int V>
+__global__ void __launch_bounds__(V_WARPS * 32) latent_values_kernel(
+    const T* __restrict__ o_rows, const float* __restrict__ part_o, const float* __restrict__ part_ml, int splits,
+    const T* __restrict__ uv, const float* __restrict__ gate, int ld_gate, T* __restrict__ out, int n_tokens, int H, int n,
+    int e, int ep) {
+  extern __shared__ __align__(16) float o_s[];   // [VT][n padded to V], then the splits' factors [VT][splits]
+  jb::pdl_launch_dependents();
+  jb::pdl_wait();
+  const int h = blockIdx.y, t0 = blockIdx.z * VT, nt = min(VT, n_tokens - t0);
+  const int np = (n + 7) / 8 * 8;
+  if (splits > 0) {
+    float* f_s = o_s + VT * np;
+    if (threadIdx.x < nt) {
+      const float* ml = part_ml + ((size_t)(t0 + threadIdx.x) * H + h) * splits * 2;
+      float m = -CUDART_INF_F, l = 0.0f;
+      for (int s = 0; s < splits; ++s) m = fmaxf(m, ml[2 * s]);
+      for (int s = 0; s < splits; ++s) l += ml[2 * s + 1] * exp2f(ml[2 * s] - m);   // a split without keys weighs 0
+      for (int s = 0; s < splits; ++s) f_s[threadIdx.x * splits + s] = exp2f(ml[2 * s] - m) / l;
+    }
+    __syncthreads();
+    for (int i = threadIdx.x; i < nt * n; i += blockDim.x) {
+      const int k = i / n, c = i % n;
+      const float* p = part_o + ((size_t)(t0 + k) * H + h) * splits * n + c;
+      float v = 0.0f;
+#pragma unroll 8
+      for (int s = 0; s < splits; ++s) v = fmaf(f_s[k * splits + s], p[(size_t)s * n], v);
+      o_s[k * np + c] = v;
+    }
+  } else {
+    for (int i = threadIdx.x; i < nt * n; i += blockDim.x)
+      o_s[(i / n) * np + i % n] = jb::to_f32(o_rows[((size_t)(t0 + i / n) * H + h) * n + i % n]);
+  }
+  __syncthreads();
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const int c0 = blockIdx.x * V_WARPS * V_ROWS + warp * V_ROWS;
+#pragma unroll 1
+  for (int rr = 0; rr < V_ROWS; rr += 2) {       // two rows at a time: their loads are in flight together
+    const int c = c0 + rr;
+    if (c >= ep) break;
+    float acc[2][VT];
+#pragma unroll
+    for (int q = 0; q < 2; ++q)
+#pragma unroll
+      for (int k = 0; k < VT; ++k) acc[q][k] = 0.0f;
+    const T* w0 = uv + ((size_t)h * e + min(c, e - 1)) * n;
+    const T* w1 = uv + ((size_t)h * e + min(c + 1, e - 1)) * n;
+    for (int i = lane * V; i < n; i += 32 * V) {
+      float a[V], b[V];
+      load_w<T, V>(w0 + i, a);
+      load_w<T, V>(w1 + i, b);
+#pragma unroll
+      for (int k = 0; k < VT; ++k) {
+        if (k < nt) {
+#pragma unroll
+          for (int v = 0; v < V; ++v) {
+            const float x = o_s[k * np + i + v];
+            acc[0][k] = fmaf(a[v], x, acc[0][k]);
+            acc[1][k] = fmaf(b[v], x, acc[1][k]);
+          }
+        }
+      }
+    }
+#pragma unroll
+    for (int q = 0; q < 2; ++q)
+#pragma unroll
+      for (int k = 0; k < VT; ++k) {
+        const float v = jb::warp_sum(acc[q][k]);
+        if (lane == 0 && k < nt && c + q < ep) {
+          float y = 0.0f;
+          if (c + q < e) {
+            y = v;
+            if (gate != nullptr) y *= 1.0f / (1.0f + expf(-gate[(size_t)(t0 + k) * ld_gate + (size_t)h * e + c + q]));
+          }
+          out[((size_t)(t0 + k) * H + h) * ep + c + q] = jb::from_f32<T>(y);
+        }
+      }
+  }
+}
+
+// rows[start[s] + i] = the cached row of position i of sequence s; one block per (page of the sequence, sequence),
+// rows of `vecs` 16-byte vectors.
+__global__ void __launch_bounds__(256) gather_rows_kernel(const uint4* __restrict__ cache, const int* __restrict__ block_table,
+                                                          int max_pages, int page_size, const int* __restrict__ kv_len,
+                                                          const int* __restrict__ start, uint4* __restrict__ rows, int vecs) {
+  jb::pdl_launch_dependents();
+  jb::pdl_wait();
+  const int s = blockIdx.y, first = blockIdx.x * page_size;
+  const int count = min(page_size, kv_len[s] - first);
+  if (count <= 0) return;
+  const uint4* src = cache + (size_t)block_table[(size_t)s * max_pages + blockIdx.x] * page_size * vecs;
+  uint4* dst = rows + (size_t)(start[s] + first) * vecs;
+  for (int i = threadIdx.x; i < count * vecs; i += blockDim.x) dst[i] = src[i];
+}
+
+bool aligned16(const void* p) { return ((uintptr_t)p & 15) == 0; }
+
+int check_row(int ld, int q_col, int H, int d, int r, const Row& row) {
+  JB_REFUSE(H < 1 || d < 0 || r < 0 || (r & 1) || d + r < 1, "latent: %d heads of %d + %d numbers", H, d, r);
+  JB_REFUSE(ld < q_col + H * (d + r), "latent: rows of %d floats do not hold the queries", ld);
+  JB_REFUSE(row.c_cache != nullptr && (ld < row.c_col + row.n + row.r || row.stored < row.n + row.r || row.n < 1 ||
+                                       row.r != r || row.w == nullptr || row.dest == nullptr),
+            "latent: rows of %d floats do not hold a row of %d + %d numbers, or %d columns do not store it", ld, row.n,
+            row.r, row.stored);
+  return 0;
+}
+
+}  // namespace
+
+// proj: float32 [T, ld]; q_out [T, H dp], the pages and `rows` in out_dtype; table: float32 [positions][r/2][2] or null
+// (no rotation); c_cache null: queries only; rows null: no second copy.
+JB_EXPORT int jb_latent_heads(const float* proj, int ld, int q_col, int H, int d, int r, int dp, const float* table,
+                              const int* positions, void* q_out, int out_dtype, int c_col, int n, int stored,
+                              const float* w, float eps, const int* dest, void* c_cache, void* rows, int T,
+                              cudaStream_t stream) {
+  if (T <= 0) return 0;
+  const Row row{c_col, n, r, stored, w, eps, dest, c_cache, rows};
+  if (const int bad = check_row(ld, q_col, H, d, r, row)) return bad;
+  JB_REFUSE(dp < d + r, "latent_heads: heads of %d numbers cannot be stored in %d columns", d + r, dp);
+  const bool vec = ld % 4 == 0 && q_col % 4 == 0 && d % 4 == 0 && r % 8 == 0 && dp % 4 == 0 && aligned16(proj) &&
+                   aligned16(q_out) && (table == nullptr || aligned16(table));
+  jb::Launch cfg(dim3(T), dim3(256), 0, stream);
+  cudaError_t e;
+#define JB_GO(TO, VEC) \
+  e = cudaLaunchKernelEx(&cfg.c, latent_prep_kernel<TO, VEC>, proj, ld, q_col, H, d, r, dp, table, positions, (TO*)q_out, row)
+  if (out_dtype == JB_F32) {
+    if (vec) JB_GO(float, true);
+    else JB_GO(float, false);
+  } else if (out_dtype == JB_BF16) {
+    if (vec) JB_GO(bf16, true);
+    else JB_GO(bf16, false);
+  } else {
+    return JB_ERR_BAD_DTYPE;
+  }
+#undef JB_GO
+  return (int)e;
+}
+
+// As jb_latent_heads, the queries multiplied into the latents' space: q_out [T, H dp], dp >= n + r; uk: [H d, n]
+// row-major in dtype.
+JB_EXPORT int jb_latent_queries(const float* proj, int ld, int q_col, int H, int d, int r, int n, int dp, const void* uk,
+                                const float* table, const int* positions, void* q_out, int dtype, int c_col, int stored,
+                                const float* w, float eps, const int* dest, void* c_cache, int T, cudaStream_t stream) {
+  if (T <= 0) return 0;
+  const Row row{c_col, n, r, stored, w, eps, dest, c_cache, nullptr};
+  if (const int bad = check_row(ld, q_col, H, d, r, row)) return bad;
+  JB_REFUSE(dp < n + r || n < 1 || d < 1, "latent_queries: %d + %d numbers cannot be stored in %d columns", n, r, dp);
+  const int vw = dtype == JB_BF16 ? 8 : 4;
+  const bool vec = n % vw == 0 && aligned16(uk);
+  const int cols = 8 * (vec ? vw : 1);
+  const int chunks = (n + cols - 1) / cols;
+  const size_t smem = ((size_t)(QT * d + 3) / 4 * 4 + (size_t)(Q_THREADS / 8) * QT * cols) * sizeof(float);
+  JB_REFUSE(smem > 200 * 1024, "latent_queries: heads of %d numbers (%zu bytes) do not fit shared memory", d, smem);
+  jb::Launch cfg(dim3(H * chunks + (c_cache != nullptr ? 1 : 0), (T + QT - 1) / QT), dim3(Q_THREADS), smem, stream);
+  cudaError_t e = cudaSuccess;
+#define JB_GO(T_, V_)                                                                                               \
+  do {                                                                                                              \
+    auto k = latent_queries_kernel<T_, V_>;                                                                         \
+    if (smem > 48 * 1024) e = cudaFuncSetAttribute(k, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);      \
+    if (e == cudaSuccess)                                                                                           \
+      e = cudaLaunchKernelEx(&cfg.c, k, proj, ld, q_col, H, d, r, n, dp, (const T_*)uk, table, positions, (T_*)q_out, T, row); \
+  } while (0)
+  if (dtype == JB_F32) {
+    if (vec) JB_GO(float, 4);
+    else JB_GO(float, 1);
+  } else if (dtype == JB_BF16) {
+    if (vec) JB_GO(bf16, 8);
+    else JB_GO(bf16, 1);
+  } else {
+    return JB_ERR_BAD_DTYPE;
+  }
+#undef JB_GO
+  return (int)e;
+}
+
+// uv: [H e, n] row-major; o_rows [T, H n] and out [T, H ep] in dtype; gate: float32 rows of ld_gate numbers, column
+// h e + c for number c of head h (null: no gate).  splits > 0: from part_o and part_ml instead of o_rows.
+JB_EXPORT int jb_latent_values(const void* o_rows, const float* part_o, const float* part_ml, int splits, const void* uv,
+                               const float* gate, int ld_gate, void* out, int dtype, int T, int H, int n, int e, int ep,
+                               cudaStream_t stream) {
+  if (T <= 0) return 0;
+  JB_REFUSE(e < 1 || ep < e || n < 1 || H < 1 || splits < 0, "latent_values: %d values in %d columns from %d numbers", e, ep, n);
+  JB_REFUSE(splits > 0 ? (part_o == nullptr || part_ml == nullptr) : o_rows == nullptr, "latent_values: no input");
+  const int vw = dtype == JB_BF16 ? 8 : 4;
+  const bool vec = n % vw == 0 && aligned16(uv);
+  const size_t smem = ((size_t)VT * ((n + 7) / 8 * 8) + (size_t)VT * splits) * sizeof(float);
+  JB_REFUSE(smem > 200 * 1024, "latent_values: latents of %d numbers do not fit shared memory", n);
+  const int rows = V_WARPS * V_ROWS;
+  jb::Launch cfg(dim3((ep + rows - 1) / rows, H, (T + VT - 1) / VT), dim3(V_WARPS * 32), smem, stream);
+  cudaError_t err = cudaSuccess;
+#define JB_GO(T_, V_)                                                                                               \
+  do {                                                                                                              \
+    auto k = latent_values_kernel<T_, V_>;                                                                          \
+    if (smem > 48 * 1024) err = cudaFuncSetAttribute(k, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);    \
+    if (err == cudaSuccess)                                                                                         \
+      err = cudaLaunchKernelEx(&cfg.c, k, (const T_*)o_rows, part_o, part_ml, splits, (const T_*)uv, gate, ld_gate, \
+                               (T_*)out, T, H, n, e, ep);                                                           \
+  } while (0)
+  if (dtype == JB_F32) {
+    if (vec) JB_GO(float, 4);
+    else JB_GO(float, 1);
+  } else if (dtype == JB_BF16) {
+    if (vec) JB_GO(bf16, 8);
+    else JB_GO(bf16, 1);
+  } else {
+    return JB_ERR_BAD_DTYPE;
+  }
+#undef JB_GO
+  return (int)err;
+}
+
+// cache: pages [page][1][page_size][stored] of 16-byte rows (row_bytes a multiple of 16); block_table [n_seqs][max_pages];
+// start[s]: the matrix row of position 0 of sequence s; pages: the most pages a sequence has.
+JB_EXPORT int jb_gather_rows(const void* cache, const int* block_table, int max_pages, int page_size, const int* kv_len,
+                             const int* start, void* rows, int row_bytes, int n_seqs, int pages, cudaStream_t stream) {
+  if (n_seqs <= 0 || pages <= 0) return 0;
+  JB_REFUSE(row_bytes % 16 != 0 || !aligned16(cache) || !aligned16(rows), "gather_rows: rows of %d bytes", row_bytes);
+  jb::Launch cfg(dim3(pages, n_seqs), dim3(256), 0, stream);
+  return (int)cudaLaunchKernelEx(&cfg.c, gather_rows_kernel, (const uint4*)cache, block_table, max_pages, page_size, kv_len,
+                                 start, (uint4*)rows, row_bytes / 16);
+}

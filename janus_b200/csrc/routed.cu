@@ -7,7 +7,8 @@
 //   scores (the lower index wins a tie); its weights are those scores, as they are.
 //   out[t] += sum over the chosen e of  Wd_e ( act(Wg_e x) * (Wu_e x) ),  x = s_e h[t]        (the weight is on the input)
 //   or, with the weight on the output,  out[t] += sum over the chosen e of  s_e Wd_e ( act(Wg_e h[t]) * (Wu_e h[t]) ).
-//   Scores may also be the softmax over all experts, and the choice may be limited to the best groups of neighbours.
+//   Scores may also be the softmax over all experts, and the choice may be limited to the best groups of neighbours; the
+//   choice may rest on scores with a correction per expert added, and the weights may be multiplied by a constant.
 //
 // Experts' weights: gate and up [E][F][W], down [E][W][F], row-major, float32 or bfloat16.
 #include <math_constants.h>
@@ -22,9 +23,11 @@ constexpr int MAX_TOP = 16;
 
 // one warp per token.  softmax = 0: a score is the logit's sigmoid; 1: the softmax over all experts.  groups > 0: the
 // experts form `groups` equal groups of neighbours, a group's score is its largest score, and only experts of the
-// `keep` groups with the largest scores can be chosen (the lower group wins a tie).
+// `keep` groups with the largest scores can be chosen (the lower group wins a tie).  correction (per expert, or null):
+// the choice is made by score + correction, the weight stays the score.  Weights are multiplied by `scale`.
 __global__ void route_topk_kernel(const float* __restrict__ logits, int ld, int E, int top, int* __restrict__ sel_e,
-                                  float* __restrict__ sel_w, int T, int softmax, int groups, int keep) {
+                                  float* __restrict__ sel_w, int T, int softmax, int groups, int keep,
+                                  const float* __restrict__ correction, float scale) {
   jb::pdl_launch_dependents();
   jb::pdl_wait();
   const int t = blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5), lane = threadIdx.x & 31;
@@ -39,6 +42,9 @@ __global__ void route_topk_kernel(const float* __restrict__ logits, int ld, int 
     for (int e = lane; e < E; e += 32) z_sum += expf(z[e] - z_max);
     z_sum = jb::warp_sum(z_sum);
   }
+  auto score = [&](float v) { return softmax ? expf(v - z_max) / z_sum : 1.0f / (1.0f + expf(-v)); };
+  // what a choice goes by: the logit itself, whose order the sigmoid and the softmax keep, or the corrected score
+  auto choice = [&](int e) { return correction != nullptr ? score(z[e]) + correction[e] : z[e]; };
   unsigned long long kept = ~0ull;               // bit g: experts of group g can be chosen
   const int per_group = groups > 0 ? E / groups : E;
   if (groups > 0) {
@@ -48,7 +54,7 @@ __global__ void route_topk_kernel(const float* __restrict__ logits, int ld, int 
       int arg = 0x7fffffff;
       for (int e = lane; e < E; e += 32) {
         const int g = e / per_group;
-        const float v = z[e];                    // scores keep the order of the logits
+        const float v = choice(e);
         if (!((kept >> g) & 1ull) && (v > best || (v == best && g < arg))) {
           best = v;
           arg = g;
@@ -73,7 +79,7 @@ __global__ void route_topk_kernel(const float* __restrict__ logits, int ld, int 
     for (int e = lane; e < E; e += 32) {
       bool taken = groups > 0 && !((kept >> (e / per_group)) & 1ull);
       for (int q = 0; q < k; ++q) taken |= picked[q] == e;
-      const float v = z[e];            // the sigmoid and the softmax keep the order of the logits
+      const float v = choice(e);
       if (!taken && (v > best || (v == best && e < arg))) {
         best = v;
         arg = e;
@@ -88,10 +94,11 @@ __global__ void route_topk_kernel(const float* __restrict__ logits, int ld, int 
         arg = oa;
       }
     }
+    if (arg >= E) arg = k;             // (logits that are no numbers: any expert, so that nothing is read out of range)
     picked[k] = arg;
     if (lane == 0) {
       sel_e[(size_t)t * top + k] = arg;
-      sel_w[(size_t)t * top + k] = softmax ? expf(best - z_max) / z_sum : 1.0f / (1.0f + expf(-best));
+      sel_w[(size_t)t * top + k] = score(z[arg]) * scale;
     }
   }
 }
@@ -424,14 +431,15 @@ __global__ void expert_scatter_kernel(const float* __restrict__ results, const i
 }  // namespace
 
 JB_EXPORT int jb_route_topk(const float* logits, int ld, int E, int top, int* sel_e, float* sel_w, int T, int softmax,
-                            int groups, int keep, cudaStream_t stream) {
+                            int groups, int keep, const float* correction, float scale, cudaStream_t stream) {
   if (T <= 0) return 0;
   JB_REFUSE(top < 1 || top > MAX_TOP || top > E, "route_topk: %d of %d experts (at most %d a token)", top, E, MAX_TOP);
   JB_REFUSE(groups < 0 || groups > 64 || (groups > 0 && (E % groups != 0 || keep < 1 || keep > groups ||
                                                           keep * (E / groups) < top)),
             "route_topk: %d groups of which %d are kept do not fit %d experts and %d a token", groups, keep, E, top);
   jb::Launch cfg(dim3((T + 3) / 4), dim3(128), 0, stream);
-  return (int)cudaLaunchKernelEx(&cfg.c, route_topk_kernel, logits, ld, E, top, sel_e, sel_w, T, softmax, groups, keep);
+  return (int)cudaLaunchKernelEx(&cfg.c, route_topk_kernel, logits, ld, E, top, sel_e, sel_w, T, softmax, groups, keep,
+                                 correction, scale);
 }
 
 // h: [T, W] in x_dtype; the experts' weights ([E] of them) in w_dtype; act: float32 scratch [T top, F]; out: float32

@@ -101,10 +101,10 @@ class DecoderModel:
         transforms = self.embedding_transforms
         scale = None
         if self.streams == 1:
-            # a single embedding transform that only multiplies is done by the gather itself
-            scale = getattr(transforms[0], "plain_scale", lambda: None)() if len(transforms) == 1 else None
+            # a first embedding transform that only multiplies is done by the gather itself
+            scale = getattr(transforms[0], "plain_scale", lambda: None)() if transforms else None
             if scale is not None:
-                transforms = ()
+                transforms = transforms[1:]
             ops.embed_gather(self.embedding, ctx.token_ids, residual, ctx.feedback,
                              ctx.seq_slot if ctx.feedback is not None else None, scale=1.0 if scale is None else scale)
         else:

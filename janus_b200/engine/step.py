@@ -67,6 +67,10 @@ class StepContext:
         self.q_start: torch.Tensor = None     # [n_seqs + 1] offsets of each sequence's tokens
         self.kv_len: torch.Tensor = None      # [n_seqs] length of each sequence after this step
         self.seq_slot: torch.Tensor = None    # [n_seqs] cache slot of each sequence
+        # prompt steps only: where each sequence's positions begin in a matrix with a row per position of the step's
+        # sequences, one sequence after another ([n_seqs + 1]), and that matrix's rows
+        self.kv_start: torch.Tensor = None
+        self.kv_total = 0
         self.feedback: torch.Tensor = None    # decode only: per slot the token sampled last (for ids < 0)
         self.groups: List[GroupStepView] = []
         self.workspace: Workspace = None
@@ -197,7 +201,7 @@ class Engine:
             q_start.append(q_start[-1] + n)
         W = len(wants)
         G = len(cache.groups)
-        sizes = [T, T, T, S + 1, S, S, W] + [T, S * P] * G
+        sizes = [T, T, T, S + 1, S, S, W] + [T, S * P] * G + [S + 1]
         offsets = [0]
         for s in sizes:
             offsets.append(offsets[-1] + _pad4(s))
@@ -219,6 +223,7 @@ class Engine:
                 pages = g.pages[e.slot]
                 bt[i, :len(pages)] = pages
             host[o[base + 1]:o[base + 1] + S * P] = bt.reshape(-1)
+        host[o[7 + 2 * G] + 1:o[7 + 2 * G] + S + 1] = np.cumsum(after)
         total = offsets[-1]
         self.last_step_h2d_bytes = 4 * total
         if self._pinned is None or self._pinned.numel() < total:
@@ -246,6 +251,7 @@ class Engine:
         ctx.max_kv_len_bound = P * PAGE_SIZE
         ctx.token_ids, ctx.positions, ctx.token_seq = seg(0, T), seg(1, T), seg(2, T)
         ctx.q_start, ctx.kv_len, ctx.seq_slot = seg(3, S + 1), seg(4, S), seg(5, S)
+        ctx.kv_start, ctx.kv_total = seg(7 + 2 * G, S + 1), sum(after)
         ctx.groups = [GroupStepView(seg(7 + 2 * gi, T), seg(8 + 2 * gi, S * P).view(S, P), PAGE_SIZE)
                       for gi in range(G)]
         ctx.workspace, ctx.cache, ctx.dtype = self.workspace, cache, self.dtype
@@ -278,7 +284,7 @@ class Engine:
             before = ops.launch_count()
             # a step of a shape that has run before hands the same kinds of tensors to the same kernels:
             # the faces' checks of device, dtype and shape are made the first time only
-            shape = (ctx.n_tokens, ctx.n_seqs, ctx.max_q_len, ctx.max_kv_len_bound, want_rows.shape[0])
+            shape = (ctx.n_tokens, ctx.n_seqs, ctx.max_q_len, ctx.max_kv_len_bound, ctx.kv_total, want_rows.shape[0])
             if shape in self._checked_shapes:
                 with ops.unchecked(), log.nvtx_range(f"step of {ctx.n_tokens} tokens"):
                     self.model.forward(ctx, want_rows, logits)

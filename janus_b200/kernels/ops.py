@@ -56,7 +56,7 @@ _SIGNATURES = {
     "jb_embed_gather": "pippiippfp", "jb_rmsnorm": "pppifpiiiplp", "jb_residual_add": "ppilp",
     "jb_swiglu": "ppiiip", "jb_swiglu_f32_to_bf16": "piipiip", "jb_zero_f32": "plp",
     "jb_pack_weight_bf16": "piipp", "jb_rope_cache_write": "piipipppppiiiiiiip",
-    "jb_gemm_f32": "pppiiiiiip", "jb_attention_f32": "pppppppiiiiiiififfp",
+    "jb_gemm_f32": "pppiiiiiip", "jb_attention_f32": "pppppppiiiiiiiififfp",
     "jb_gemm_bf16": "pplipiiiiiiplpiffpp", "jb_gemm_bf16_pair": "pplipiiiiiiiffpp",
     "jb_gemm_bf16_pair_grouped": "pplipiiiiipiffpp", "jb_expert_plan": "piiiippppp",
     "jb_gemm_bf16_pair_qkv_rope": "ppliippppppiiiipp",
@@ -67,7 +67,7 @@ _SIGNATURES = {
     "jb_join_norm": "pppppffpppfipipiiplplp", "jb_head_norm_gate": "ppipipfipiiiip", "jb_sigmoid_gate": "pipiiiiip",
     "jb_head_norm_rope_cache": "pippfpippipppiiiiiiiiifip",
     "jb_delta_rule": "piiiipiiippfppllppiiiiip",
-    "jb_route_topk": "piiippiiiip", "jb_experts_few_tokens": "pippipppippiiiiffip", "jb_expert_gather": "pippipiip",
+    "jb_route_topk": "piiippiiiipfp", "jb_experts_few_tokens": "pippipppippiiiiffip", "jb_expert_gather": "pippipiip",
     "jb_expert_scatter": "pppipiip",
     "jb_gla_decay": "piiippfpiip", "jb_exp_gates": "piiippfppllppiip",
     "jb_gated_linear_scan": "piiiifpiippplppiiiiiippp", "jb_scale_rows_sigmoid": "pipiiip",
@@ -81,6 +81,9 @@ _SIGNATURES = {
     "jb_sublayer_norm_add": "ppiffppiiiplplp", "jb_qk_norm_rope_cache": "pippppfpippipppiiiiiiip",
     "jb_latent_prep": "piiiipfpippiip", "jb_causal_conv_silu": "piiippipllppppiiiip",
     "jb_mamba2_scan": "piiipipppppllppiiiiiiippp", "jb_gated_group_rmsnorm": "ppipfpiiiip", "jb_pad_rows_bf16": "pipiip", "jb_scale_softcap": "plffp",
+    "jb_gelu": "ppilp", "jb_tanh_norm": "ppppffippfpipiiplplp",
+    "jb_latent_heads": "piiiiiipppiiiipfpppip", "jb_latent_queries": "piiiiiiippppiiipfppip", "jb_latent_values": "pppippipiiiiiip",
+    "jb_gather_rows": "ppiipppiiip", "jb_latent_attention": "ppppppppiiiiiiifiip", "jb_attention_tc_matrix": "ppppppiiiiiiiifpp",
 }
 _CTYPES = {"p": ctypes.c_void_p, "i": ctypes.c_int, "l": ctypes.c_longlong, "u": ctypes.c_ulonglong,
            "f": ctypes.c_float}
@@ -294,13 +297,14 @@ def gemm_f32(x: torch.Tensor, w: torch.Tensor, y: torch.Tensor, accumulate: bool
 def attention_f32(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor, out: torch.Tensor,
                   block_table: torch.Tensor, token_slot: torch.Tensor, positions: torch.Tensor,
                   nh: int, nkv: int, hd: int, page_size: int, window: int, scale: float, chunk: int = 0,
-                  softcap: float = 0.0, sink: bool = False) -> None:
-    """`chunk` > 0: a query sees only the keys of its own chunk of positions, [floor(pos / chunk) chunk, pos];
+                  softcap: float = 0.0, sink: bool = False, vd: Optional[int] = None) -> None:
+    """`vd`: the values are the first vd numbers of the value rows (None: all hd), out is [T, nh vd].  `chunk` > 0: a query sees only the keys of its own chunk of positions, [floor(pos / chunk) chunk, pos];
     `softcap` > 0: a score s becomes softcap tanh(s / softcap); `sink`: the softmax's denominator has one more
     term, exp(0), a key of score 0 that has no value."""
     T = q.shape[0]
+    vd = hd if vd is None else int(vd)
     _need(q, "attention q", torch.float32, (T, nh * hd))
-    _need(out, "attention out", torch.float32, (T, nh * hd))
+    _need(out, "attention out", torch.float32, (T, nh * vd))
     _need(k_cache, "k cache", torch.float32)
     _need(v_cache, "v cache", torch.float32)
     _need(block_table, "block table", torch.int32)
@@ -308,7 +312,7 @@ def attention_f32(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor,
     _need(positions, "positions", torch.int32, (T,))
     _check(_lib("attention_f32").jb_attention_f32(
         _ptr(q), _ptr(k_cache), _ptr(v_cache), _ptr(out), _ptr(block_table), _ptr(token_slot), _ptr(positions),
-        T, nh, nkv, hd, page_size, block_table.shape[1], int(window), scale, int(chunk), float(softcap),
+        T, nh, nkv, hd, vd, page_size, block_table.shape[1], int(window), scale, int(chunk), float(softcap),
         1.0 if sink else 0.0, _stream()), "attention_f32")
 
 
@@ -605,7 +609,8 @@ def gemm_bf16(x: torch.Tensor, w: PackedWeight, y: torch.Tensor, mode: str = "st
     mode "store": y[T, N] = result (bf16 or float32 by y's dtype);
     mode "add":   y[T, N] += result, y float32 (K may be split, sums meet by atomic adds);
     mode "swiglu": w a gated pair (`pack_gated`), y[T, N] = silu(gate) * up in bf16; with gate_limit > 0 the
-                   clamped form g sigmoid(gate_alpha g) (u + 1), g = min(gate, limit), u = clamp(up, +-limit).
+                   clamped form g sigmoid(gate_alpha g) (u + 1), g = min(gate, limit), u = clamp(up, +-limit);
+    mode "gelu":  y[T, N] = gelu(result) in bf16, gelu(z) = z (1 + erf(z / sqrt 2)) / 2.
     `split_k`, `pair`, `whole_tiles`: as `gemm_plan_whole` picks them unless given (`whole_tiles`: CTA pairs
     only, the first so many 256 x 256 output tiles of an adding product stay uncut)."""
     T, K = x.shape
@@ -625,6 +630,8 @@ def gemm_bf16(x: torch.Tensor, w: PackedWeight, y: torch.Tensor, mode: str = "st
             raise KernelError(f"gemm {mode}: the weight is a gated pair")
         if mode == "add":
             code, want = 2, torch.float32
+        elif mode == "gelu":
+            code, want = 5, torch.bfloat16
         elif mode == "store":
             code, want = (1, torch.float32) if y.dtype == torch.float32 else (0, torch.bfloat16)
         else:
@@ -945,8 +952,8 @@ def attention_tc_supported(nh: int, nkv: int, hd: int) -> bool:
 
 
 def _attention_tc_row(hd: int) -> int:
-    """The build that takes head size `hd`: rows of 64, 128 or 256 dims in shared memory."""
-    return 64 if hd <= 64 else 128 if hd <= 128 else 256
+    """The build that takes head size `hd`: rows of 64, 128, 192 or 256 dims in shared memory."""
+    return 64 if hd <= 64 else 128 if hd <= 128 else 192 if hd <= 192 else 256
 
 
 def attention_tc_prefill(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor, out: torch.Tensor,
@@ -977,6 +984,28 @@ def attention_tc_prefill(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.
         _ptr(q), _ptr(k_cache), _ptr(v_cache), _ptr(out), _ptr(block_table), _ptr(q_start), _ptr(kv_len),
         T, k_cache.shape[0], n_seqs, max_q_len, nh, nkv, hd, page_size, block_table.shape[1], int(window),
         scale, _ptr(kernel_status(q.device)), _stream()), "attention_tc_prefill")
+
+
+def attention_tc_matrix(q: torch.Tensor, kv: torch.Tensor, out: torch.Tensor, kv_start: torch.Tensor,
+                        q_start: torch.Tensor, kv_len: torch.Tensor, n_seqs: int, max_q_len: int, nh: int, hd: int,
+                        vd: int, max_kv_len: int, scale: float) -> None:
+    """Causal attention on the tcgen05 tensor cores of each sequence's new tokens (the last q_len positions of its
+    kv_len) over keys and values that lie in one matrix, kv [rows, nh hd + nh vd] bfloat16: a key and a value per query
+    head, the key of position p of sequence s in row kv_start[s] + p.  q [T, nh hd], out [T, nh vd]."""
+    T = q.shape[0]
+    _need(q, "attention q", torch.bfloat16, (T, nh * hd))
+    _need(out, "attention out", torch.bfloat16, (T, nh * vd))
+    _need(kv, "keys and values", torch.bfloat16)
+    if kv.dim() != 2 or kv.shape[1] != nh * (hd + vd):
+        raise KernelError(f"attention_tc_matrix: {tuple(kv.shape)} does not hold {nh} heads of {hd} and {vd} numbers")
+    for t, name, n in ((kv_start, "first rows", n_seqs), (q_start, "q_start", n_seqs + 1), (kv_len, "kv_len", n_seqs)):
+        _need(t, name, torch.int32)
+        if t.numel() < n:
+            raise KernelError(f"attention_tc_matrix: '{name}' holds {t.numel()} numbers")
+    lib = _lib("attention_tc", _attention_tc_row(hd), lambda h: dict({"JB_HEAD_DIM": h}, **_ATTN_TC_DEFINES))
+    _check(lib.jb_attention_tc_matrix(
+        _ptr(q), _ptr(kv), _ptr(out), _ptr(kv_start), _ptr(q_start), _ptr(kv_len), T, kv.shape[0], n_seqs, max_q_len, nh,
+        hd, vd, int(max_kv_len), float(scale), _ptr(kernel_status(q.device)), _stream()), "attention_tc_matrix")
 
 
 # -- several residual streams per token -------------------------------------------------
@@ -1196,6 +1225,13 @@ def diff_attention_prefill(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torc
         _ptr(q), _ptr(k_cache), _ptr(v_cache), _ptr(out), _ptr(block_table), _ptr(q_start), _ptr(kv_len), n_seqs,
         max_q_len, heads, kv_heads, dim, vdim, page_size, block_table.shape[1], int(window), int(keep_first), scale, lam,
         eps, out_scale, _stream()), "diff_attention_prefill")
+
+
+def gelu(x: torch.Tensor, out: torch.Tensor) -> None:
+    """out = gelu(x) elementwise, gelu(z) = z (1 + erf(z / sqrt 2)) / 2; float32 in, out's dtype out."""
+    _need(x, "activation in", torch.float32)
+    _need(out, "activation out", None, tuple(x.shape))
+    _check(_lib("elementwise").jb_gelu(_ptr(x), _ptr(out), dtype_code(out.dtype), x.numel(), _stream()), "gelu")
 
 
 # -- a gated activation with clamped branches; scale and soft cap -------------------------------
@@ -1558,20 +1594,26 @@ def delta_rule(conv: torch.Tensor, q_col: int, k_col: int, v_col: int, raw: torc
 
 # -- experts of which a token uses a few ---------------------------------------------------------------------------
 def route_topk(logits: torch.Tensor, top: int, sel_e: torch.Tensor, sel_w: torch.Tensor, softmax: bool = False,
-               groups: int = 0, keep: int = 0, experts: Optional[int] = None) -> None:
+               groups: int = 0, keep: int = 0, experts: Optional[int] = None,
+               correction: Optional[torch.Tensor] = None, scale: float = 1.0) -> None:
     """Per row of the float32 logits [T, >= E] (the first `experts` columns; None: all): the `top` largest (the lower
     index wins a tie) as indices (int32 [T, top]) and their scores as weights (float32 [T, top]): the logits' sigmoids,
     or with `softmax` the softmax over all experts.  `groups` > 0: the experts form that many equal groups of
-    neighbours, and only experts of the `keep` groups whose best expert scores highest can be chosen."""
+    neighbours, and only experts of the `keep` groups whose best expert scores highest can be chosen.  `correction`
+    (float32 [experts]): the choice goes by score + correction, the weights stay the scores.  The weights are multiplied
+    by `scale`."""
     T, ld = logits.shape
     E = ld if experts is None else int(experts)
     _need(logits, "router logits", torch.float32)
     _need(sel_e, "chosen experts", torch.int32, (T, top))
     _need(sel_w, "experts' weights", torch.float32, (T, top))
+    if correction is not None:
+        _need(correction, "router's correction", torch.float32, (E,))
     if E > ld:
         raise KernelError(f"route_topk: {E} experts in rows of {ld} logits")
     _check(_lib("routed").jb_route_topk(_ptr(logits), ld, E, int(top), _ptr(sel_e), _ptr(sel_w), T,
-                                        int(bool(softmax)), int(groups), int(keep), _stream()), "route_topk")
+                                        int(bool(softmax)), int(groups), int(keep), _ptr(correction), float(scale), _stream()),
+           "route_topk")
 
 
 def experts_few_tokens(h: torch.Tensor, sel_e: torch.Tensor, sel_w: torch.Tensor, w_gate: torch.Tensor,
@@ -1738,3 +1780,210 @@ def gated_linear_scan(proj: torch.Tensor, q_col: int, k_col: int, v_col: int, q_
         0 if scalar else heads * dim, int(scalar), _ptr(out), _ptr(divisors), _ptr(state), state.shape[1],
         _ptr(q_start), _ptr(seq_slot), n_seqs, heads, dim, vdim, int(max_q_len), seg, _ptr(scratch), _ptr(seg_decay),
         _stream()), "gated_linear_scan", kernels=4 if seg else 1)
+
+
+# -- dynamic tanh in the place of a norm -------------------------------------------------------------------------
+def tanh_norm(stream: torch.Tensor, y: Optional[torch.Tensor] = None, norm_y: Optional[tuple] = None, mult: float = 1.0,
+              replace: bool = False, norm_x: Optional[tuple] = None, x_out: Optional[torch.Tensor] = None,
+              row_index: Optional[torch.Tensor] = None, clear: Optional[torch.Tensor] = None,
+              clear2: Optional[torch.Tensor] = None) -> None:
+    """One launch over the float32 stream r [T, W], every step optional, with N(v) = tanh(alpha v) * w + b for a norm
+    (w, b, alpha): r += mult * norm_y(y) (y set to zero), or with `replace` r = norm_y(r); x_out = norm_x(r) (no norm_x:
+    the cast alone).  With `row_index` x_out's rows are norm_x(r[row_index[i]]) and r is only read.  `clear`, `clear2`:
+    float32 scratch tensors (whole 16-byte vectors) set to zero on the way."""
+    W = stream.shape[1]
+    T = stream.shape[0] if row_index is None else row_index.shape[0]
+    _need(stream, "stream", torch.float32)
+    if y is not None:
+        _need(y, "sublayer output", torch.float32, tuple(stream.shape))
+    for norm in (norm_y, norm_x):
+        if norm is not None:
+            _need(norm[0], "norm weight", torch.float32, (W,))
+            _need(norm[1], "norm bias", torch.float32, (W,))
+    if x_out is not None:
+        _need(x_out, "normed rows", None, (T, W))
+    if row_index is not None:
+        _need(row_index, "row index", torch.int32)
+    for c in (clear, clear2):
+        if c is not None:
+            _need(c, "buffer to clear", torch.float32)
+    wa, ba, aa = norm_y if norm_y is not None else (None, None, 0.0)
+    wb, bb, ab = norm_x if norm_x is not None else (None, None, 0.0)
+    _check(_lib("tanh_norm").jb_tanh_norm(
+        _ptr(stream), _ptr(y), _ptr(wa), _ptr(ba), float(aa), float(mult), int(bool(replace)), _ptr(wb), _ptr(bb), float(ab),
+        _ptr(x_out), dtype_code(x_out.dtype) if x_out is not None else F32, _ptr(row_index), T, W, _ptr(clear),
+        0 if clear is None else clear.numel(), _ptr(clear2), 0 if clear2 is None else clear2.numel(), _stream()),
+        "tanh_norm")
+
+
+# -- latent attention with a rotated part ------------------------------------------------------------------------
+LATENT_MAX_ROW = 1280          # numbers a cached row may have (the float32 attention kernel's limit)
+
+
+def _latent_row(proj, q_out, d, r, table, positions, row):
+    """Checks shared by the two faces below; `row`: None, or (column, n, stored, weight, eps, dest, pages)."""
+    T = q_out.shape[0]
+    _need(proj, "projections", torch.float32)
+    _need(q_out, "q_out")
+    _need(positions, "positions", torch.int32, (T,))
+    if proj.shape[0] != T:
+        raise KernelError("latent attention: projections and queries differ in their rows")
+    if table is not None and r > 0:
+        _need(table, "rotation table", torch.float32)
+        if tuple(table.shape[1:]) != (r // 2, 2):
+            raise KernelError(f"latent attention: table of shape {tuple(table.shape)} does not fit {r} rotated numbers")
+    if row is not None:
+        _, n, stored, weight, _, dest, pages = row
+        _need(weight, "latent norm weight", torch.float32, (n,))
+        _need(dest, "cache rows", torch.int32, (T,))
+        _need(pages, "latent pages", q_out.dtype)
+        if pages.shape[-1] != stored:
+            raise KernelError(f"latent attention: pages {tuple(pages.shape)} do not hold rows of {stored}")
+
+
+def latent_heads(proj: torch.Tensor, q_col: int, heads: int, d: int, r: int, stored_head: int,
+                 table: Optional[torch.Tensor], positions: torch.Tensor, q_out: torch.Tensor,
+                 row: Optional[tuple] = None, rows: Optional[torch.Tensor] = None) -> None:
+    """Queries as heads: q_out [T, heads stored_head] = [d numbers as projected | r numbers turned | zeros] from the
+    columns at q_col of proj (float32 [T, >=]).  `row` = (column, n, stored, weight, eps, dest, pages): the token's own
+    row [n numbers divided by their root mean square times weight | r numbers turned] from the columns there is appended
+    to the pages at row dest, and copied to `rows` [T, stored] if given."""
+    T = q_out.shape[0]
+    _latent_row(proj, q_out, d, r, table, positions, row)
+    _need(q_out, "q_out", None, (T, heads * stored_head))
+    col, n, stored, weight, eps, dest, pages = row if row is not None else (0, 0, 0, None, 0.0, None, None)
+    if rows is not None:
+        _need(rows, "rows", q_out.dtype, (T, stored))
+    _check(_lib("latent").jb_latent_heads(
+        _ptr(proj), proj.shape[1], int(q_col), heads, d, r, stored_head, _ptr(table) if r else None, _ptr(positions),
+        _ptr(q_out), dtype_code(q_out.dtype), int(col), n, stored, _ptr(weight), float(eps), _ptr(dest), _ptr(pages),
+        _ptr(rows), T, _stream()), "latent_heads")
+
+
+def latent_queries(proj: torch.Tensor, q_col: int, heads: int, d: int, r: int, n: int, stored: int, uk: torch.Tensor,
+                   table: Optional[torch.Tensor], positions: torch.Tensor, q_out: torch.Tensor,
+                   row: Optional[tuple] = None) -> None:
+    """Queries in the latents' space: q_out [T, heads stored] = [uk_h^T q_h (n numbers) | the turned part | zeros], with
+    uk [heads d, n] in q_out's dtype and q_h the head's d numbers as projected (float32).  `row`: as in `latent_heads`."""
+    T = q_out.shape[0]
+    _latent_row(proj, q_out, d, r, table, positions, row)
+    _need(q_out, "q_out", None, (T, heads * stored))
+    _need(uk, "keys' matrix", q_out.dtype, (heads * d, n))
+    col, _, _, weight, eps, dest, pages = row if row is not None else (0, 0, 0, None, 0.0, None, None)
+    _check(_lib("latent").jb_latent_queries(
+        _ptr(proj), proj.shape[1], int(q_col), heads, d, r, n, stored, _ptr(uk), _ptr(table) if r else None,
+        _ptr(positions), _ptr(q_out), dtype_code(q_out.dtype), int(col), stored, _ptr(weight), float(eps), _ptr(dest),
+        _ptr(pages), T, _stream()), "latent_queries")
+
+
+def latent_values(o: Optional[torch.Tensor], partial: Optional[tuple], uv: torch.Tensor, gate: Optional[torch.Tensor],
+                  out: torch.Tensor, heads: int, n: int, e: int, stored: int) -> None:
+    """out[t, h, :e] = uv_h o[t, h] (times sigmoid(gate[t, h, :]), float32 columns), zeros up to `stored`; uv
+    [heads e, n].  o [T, heads n], or `partial` = (sums, maxima, splits): what the splits of `latent_attention` left."""
+    T = out.shape[0]
+    _need(out, "head outputs", None, (T, heads * stored))
+    _need(uv, "values' matrix", out.dtype, (heads * e, n))
+    sums, maxima, splits = partial if partial is not None else (None, None, 0)
+    if partial is None:
+        _need(o, "attention's output", out.dtype, (T, heads * n))
+    else:
+        _need(sums, "partial sums", torch.float32)
+        _need(maxima, "partial maxima", torch.float32)
+        if sums.numel() < T * heads * splits * n or maxima.numel() < T * heads * splits * 2:
+            raise KernelError("latent_values: the partial sums are too small")
+    if gate is not None and (gate.dtype != torch.float32 or gate.stride(1) != 1 or tuple(gate.shape) != (T, heads * e)):
+        raise KernelError("latent_values: the gate must be float32 columns, one for each number of the heads")
+    _check(_lib("latent").jb_latent_values(
+        _ptr(o), _ptr(sums), _ptr(maxima), int(splits), _ptr(uv), _ptr(gate), gate.stride(0) if gate is not None else 0,
+        _ptr(out), dtype_code(out.dtype), T, heads, n, e, stored, _stream()), "latent_values")
+
+
+def gather_rows(pages: torch.Tensor, block_table: torch.Tensor, kv_len: torch.Tensor, start: torch.Tensor,
+                rows: torch.Tensor, page_size: int, n_seqs: int) -> None:
+    """rows[start[s] + i] = the cached row of position i of sequence s (one key head a page)."""
+    _need(pages, "pages", rows.dtype)
+    _need(rows, "rows")
+    for t, name in ((block_table, "block table"), (kv_len, "kv_len"), (start, "first rows")):
+        _need(t, name, torch.int32)
+    if pages.shape[-1] != rows.shape[1]:
+        raise KernelError(f"gather_rows: pages {tuple(pages.shape)} do not fit rows {tuple(rows.shape)}")
+    _check(_lib("latent").jb_gather_rows(
+        _ptr(pages), _ptr(block_table), block_table.shape[1], page_size, _ptr(kv_len), _ptr(start), _ptr(rows),
+        rows.shape[1] * rows.element_size(), n_seqs, block_table.shape[1], _stream()), "gather_rows")
+
+
+def _latent_attention_lib(stored: int, n: int):
+    return _lib("latent_attention", (int(stored), int(n)), lambda k: {"JB_LATENT_D": k[0], "JB_LATENT_N": k[1]})
+
+
+def latent_attention_smem(stored: int, n: int, blocks: int, stages: Optional[int] = None) -> int:
+    """Shared memory of a CTA of the bfloat16 latent attention kernel with the given row blocks (in step with the
+    constants of csrc/latent_attention.cu); 0 if its rows do not fit."""
+    ld = (stored + 15) // 16 * 16 + 8
+    kt = 32 if stored > 320 else 64
+    ks = 8 // (kt // 8)
+    rows = 16 * blocks
+    fixed = rows * ld * 2 + ks * rows * (kt + 4) * 4 + rows * (kt + 8) * 2 + 2 * rows * 4 + 64
+    fit = min(4, (227 * 1024 - fixed) // (kt * ld * 2)) if stages is None else stages
+    return fixed + fit * kt * ld * 2 if fit >= 2 else 0
+
+
+def latent_attention_supported(stored: int, n: int) -> bool:
+    return stored % 8 == 0 and latent_attention_smem(stored, n, 1) > 0
+
+
+# Constants of the estimate in `latent_splits_for`, in microseconds: they rank split counts, they forecast no time.
+_LATENT_CTA_US = 2.5
+_LATENT_TILE_US_PER_KB = 0.021      # a tile of the ring, by its size
+_LATENT_SPLIT_US = 0.06             # what one more split costs the kernel that joins them
+
+
+@functools.lru_cache(maxsize=4096)
+def latent_splits_for(n_seqs: int, row_tiles: int, max_kv_len: int, stored: int, n: int, blocks: int) -> int:
+    """Splits of the key range: waves of CTAs over the SMs times a CTA's tiles.  `max_kv_len` is the bound a step was
+    laid out for; sequences are taken to be three quarters of it."""
+    kt = 32 if stored > 320 else 64
+    tile_us = 0.15 + _LATENT_TILE_US_PER_KB * kt * stored * 2 / 1024
+    tiles = max(1, (3 * max_kv_len // 4 + kt - 1) // kt)
+    per_sm = max(1, min(4, 228 * 1024 // (latent_attention_smem(stored, n, blocks) + 1024)))
+    places = SM_COUNT_TARGET // 2 * per_sm
+    best = (float("inf"), 1)
+    for splits in (1, 2, 3, 4, 6, 8, 12, 16, 18, 24, 32, 48, 64):
+        if splits > 1 and splits > tiles // 2:
+            break
+        waves = (n_seqs * row_tiles * splits + places - 1) // places
+        cost = waves * (_LATENT_CTA_US + (tiles + splits - 1) // splits * tile_us)
+        cost += _LATENT_SPLIT_US * splits if splits > 1 else 0.0
+        if cost < best[0] - 1e-9:
+            best = (cost, splits)
+    return best[1]
+
+
+def latent_attention(q: torch.Tensor, pages: torch.Tensor, out: Optional[torch.Tensor], block_table: torch.Tensor,
+                     q_start: torch.Tensor, kv_len: torch.Tensor, n_seqs: int, max_q_len: int, heads: int, stored: int,
+                     n: int, page_size: int, scale: float, workspace, max_kv_len: int,
+                     n_splits: Optional[int] = None) -> Optional[tuple]:
+    """bfloat16 attention of each sequence's new tokens over its cached rows: a row's `stored` numbers are the key of
+    every head, its first n numbers the value.  q [T, heads stored].  With one split writes out [T, heads n] and returns
+    None; else returns (partial sums, maxima, splits), which `latent_values` joins."""
+    T = q.shape[0]
+    _need(q, "attention q", torch.bfloat16, (T, heads * stored))
+    _need(pages, "latent pages", torch.bfloat16)
+    _need(block_table, "block table", torch.int32)
+    for t, name in ((q_start, "q_start"), (kv_len, "kv_len")):
+        _need(t, name, torch.int32)
+    blocks = 2 if max_q_len * heads > 16 and latent_attention_smem(stored, n, 2) else 1
+    if n_splits is None:
+        tiles = (max_q_len * heads + 16 * blocks - 1) // (16 * blocks)
+        n_splits = latent_splits_for(n_seqs, tiles, max_kv_len, stored, n, blocks)
+    part_o = part_ml = None
+    if n_splits > 1:
+        part_o = workspace.get("latent_part_o", (T * heads * n_splits * n,), torch.float32)
+        part_ml = workspace.get("latent_part_ml", (T * heads * n_splits * 2,), torch.float32)
+    else:
+        _need(out, "attention out", torch.bfloat16, (T, heads * n))
+    _check(_latent_attention_lib(stored, n).jb_latent_attention(
+        _ptr(q), _ptr(pages), _ptr(out), _ptr(part_o), _ptr(part_ml), _ptr(block_table), _ptr(q_start), _ptr(kv_len),
+        n_seqs, max_q_len, heads, stored, n, page_size, block_table.shape[1], float(scale), int(n_splits), blocks,
+        _stream()), "latent_attention")
+    return (part_o, part_ml, n_splits) if n_splits > 1 else None

@@ -242,6 +242,19 @@ class Norm(Part):
         tensor of the part that runs next, zeroed besides.  Needed only by models with several residual streams."""
         raise NotImplementedError
 
+    # whether `forward` takes a second buffer to clear
+    clears_two = False
+
+    def add_normed_then(self, y: torch.Tensor, residual: torch.Tensor, mult: float, next_norm: "Norm", x_out: torch.Tensor,
+                        clear: Optional[torch.Tensor] = None) -> None:
+        """residual += mult * norm(y), y <- 0, then x_out = next_norm(residual): what an arrangement with norms on both
+        sides of a sublayer does between two sublayers.  A norm may do it in one launch."""
+        self.add_normed(y, residual, mult)
+        if clear is None:
+            next_norm.forward(residual, x_out)
+        else:
+            next_norm.forward(residual, x_out, clear=clear)
+
     def add_normed(self, y: Optional[torch.Tensor], residual: torch.Tensor, mult: float,
                    x_out: Optional[torch.Tensor] = None, clear: Optional[torch.Tensor] = None,
                    clear2: Optional[torch.Tensor] = None) -> None:

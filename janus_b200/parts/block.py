@@ -173,3 +173,75 @@ class OutputNormBlock:
 
 
 register_part("arrangement", "output_norm", OutputNormBlock)
+
+
+class _SandwichWrite:
+    """As `_NormedWrite`, for a sublayer that follows with a norm of its own in front."""
+
+    def __init__(self, norm):
+        self.norm = norm
+
+    def write(self, residual: torch.Tensor, y: torch.Tensor) -> None:
+        self.norm.add_normed(y, residual, 1.0)
+
+    def write_then_norm(self, residual: torch.Tensor, y: torch.Tensor, next_norm, x: torch.Tensor, clear=None) -> None:
+        self.norm.add_normed_then(y, residual, 1.0, next_norm, x, clear)
+
+
+class SandwichNormBlock:
+    """A norm before and a norm after each sublayer: x <- x + out_norm(mixer(norm(x))), then
+    x <- x + out_norm(feed_forward(norm(x))).  `parts`: mixer_norm, mixer, mixer_out_norm, and, unless the layer has no
+    feed-forward, feed_forward_norm, feed_forward, feed_forward_out_norm.  A sublayer adds its output into a zeroed
+    float32 [T, hidden_size] buffer; where the norms can, one launch then norms it, adds it to the residual stream,
+    zeroes the buffer and norms the stream for the sublayer that follows (also the next layer's mixer: the last sum of
+    a layer waits for it)."""
+
+    def __init__(self, parts: dict, hidden_size: int, dtype: torch.dtype):
+        unknown = set(parts) - {"mixer_norm", "mixer", "mixer_out_norm", "feed_forward_norm", "feed_forward",
+                                "feed_forward_out_norm"}
+        if unknown:
+            raise ValueError(f"the sandwich_norm arrangement has no use for the parts {sorted(unknown)}")
+        try:
+            self.mixer_norm, self.mixer = parts["mixer_norm"], parts["mixer"]
+            self._mixer_write = _SandwichWrite(parts["mixer_out_norm"])
+            self.feed_forward = parts.get("feed_forward")
+            if self.feed_forward is not None:
+                self.feed_forward_norm = parts["feed_forward_norm"]
+                self._ff_write = _SandwichWrite(parts["feed_forward_out_norm"])
+        except KeyError as e:
+            raise ValueError(f"the sandwich_norm arrangement needs the part {e.args[0]!r}") from None
+        self.hidden_size, self.dtype = hidden_size, dtype
+
+    def forward(self, residual: torch.Tensor, ctx, cache_view, writes_cache: bool = True) -> None:
+        T = residual.shape[0]
+        x = ctx.workspace.get("normed", (T, self.hidden_size), self.dtype)
+        y = ctx.workspace.get("sublayer_out", (T, self.hidden_size), torch.float32)
+        pending = ctx.pending_write
+        ctx.pending_write = None
+        # a mixer may name a scratch buffer that it wants zeroed; the launch before it does that in passing
+        wants = getattr(self.mixer, "scratch_to_clear", None)
+        scratch = wants(ctx, T, writes_cache) if wants is not None else None
+        if pending is not None and pending[1] is y and hasattr(pending[0], "write_then_norm"):
+            pending[0].write_then_norm(residual, y, self.mixer_norm, x, clear=scratch)
+        else:
+            if pending is not None:
+                pending[0].write(residual, pending[1])
+            clears = {} if scratch is None else {"clear": scratch}
+            if self.mixer_norm.clears_two and y.numel() % 4 == 0:    # the norm's launch also zeroes the sublayers' buffer
+                clears["clear2"] = y
+            else:
+                y.zero_()
+            self.mixer_norm.forward(residual, x, **clears)
+        if scratch is not None:
+            self.mixer.forward(x, y, ctx, cache_view, writes_cache, scratch_cleared=True)
+        else:
+            self.mixer.forward(x, y, ctx, cache_view, writes_cache)
+        last = self._mixer_write
+        if self.feed_forward is not None:
+            last.write_then_norm(residual, y, self.feed_forward_norm, x)
+            self.feed_forward.forward(x, y, ctx)
+            last = self._ff_write
+        ctx.pending_write = (last, y)
+
+
+register_part("arrangement", "sandwich_norm", SandwichNormBlock)

@@ -6,7 +6,7 @@ from __future__ import annotations
 import torch
 
 from .base import FeedForward, register_part
-from .linear import GatedLinear, Linear
+from .linear import GatedLinear, GeluLinear, Linear
 
 
 class SwiGLUFeedForward(FeedForward):
@@ -94,6 +94,31 @@ class GeluGLUFeedForward(FeedForward):
         self.down.forward_add(act, residual)
 
 
+class GeluFeedForward(FeedForward):
+    """down( gelu(up(x)) ), gelu(z) = z (1 + erf(z / sqrt 2)) / 2, added into the residual stream: no gate."""
+
+    def __init__(self, hidden_size: int, intermediate_size: int,
+                 dtype: torch.dtype = torch.bfloat16, device: torch.device = torch.device("cuda")):
+        self.hidden_size, self.intermediate_size = hidden_size, intermediate_size
+        self.dtype, self.device = dtype, device
+        self.up = GeluLinear(hidden_size, intermediate_size, dtype, device, name="up", pad_width=True)
+        self.down = Linear(intermediate_size, hidden_size, dtype, device, name="down", pad_width=True)
+
+    def weight_shapes(self):
+        return {"up": ((self.intermediate_size, self.hidden_size), "normal"),
+                "down": ((self.hidden_size, self.intermediate_size), "normal")}
+
+    def load(self, up: torch.Tensor, down: torch.Tensor) -> None:
+        self.up.load([up])
+        self.down.load([down])
+
+    def forward(self, x: torch.Tensor, residual: torch.Tensor, ctx) -> None:
+        act = ctx.workspace.get("ffn_act", (x.shape[0], self.intermediate_size), self.dtype)
+        self.up.forward(x, act, ctx)
+        self.down.forward_add(act, residual)
+
+
 register_part("feed_forward", "swiglu", SwiGLUFeedForward)
+register_part("feed_forward", "gelu_mlp", GeluFeedForward)
 register_part("feed_forward", "gelu_glu", GeluGLUFeedForward)
 register_part("feed_forward", "clamped_glu", ClampedGLUFeedForward)

@@ -136,6 +136,22 @@ class Linear:
             ops.gemm_bf16(x, self.weight, residual, mode="add", label=self.name)
 
 
+class GeluLinear(Linear):
+    """out = gelu(x W^T) in the engine dtype, gelu(z) = z (1 + erf(z / sqrt 2)) / 2: in the product's own epilogue, or,
+    where a decode-sized step would leave SMs idle with K uncut (and in float32), behind a plain product."""
+
+    def forward(self, x: torch.Tensor, out: torch.Tensor, ctx) -> None:
+        T = x.shape[0]
+        if self.dtype == torch.float32 or self.meets_by_adds(T, torch.float32) and T <= 64:
+            z = ctx.workspace.get("gelu_in", (T, self.out_features), torch.float32)
+            super().forward(x, z)
+            ops.gelu(z, out)
+            return
+        if self._padded is not None:
+            x = self._padded.rows(x)
+        ops.gemm_bf16(x, self.weight, out, mode="gelu", label=self.name)
+
+
 class GatedLinear:
     """out = silu(x Wg^T) * (x Wu^T) with Wg stacked over Wu
     (crates/janus-engine/src/model/block.rs:383-430).  With `limit` > 0 the activation is the clamped form

@@ -54,6 +54,7 @@ class LayerNorm(Norm):
     statistics in float32 (the mean first, then the mean of the squared deviations)."""
 
     CENTER = True
+    clears_two = True
 
     def __init__(self, width: int, eps: float, dtype: torch.dtype, device: torch.device):
         self.width, self.eps = int(width), float(eps)
@@ -81,3 +82,48 @@ class LayerNorm(Norm):
 
 
 register_part("norm", "layer_norm", LayerNorm)
+
+
+class DynamicTanh(Norm):
+    """y = tanh(alpha * x) * gamma + beta feature by feature, alpha one number: an elementwise stand-in for a norm that
+    needs no mean and no variance.  All in float32."""
+
+    clears_two = True
+
+    def __init__(self, width: int, dtype: torch.dtype, device: torch.device):
+        self.width = int(width)
+        self.dtype, self.device = dtype, device
+        self.args: Optional[tuple] = None        # (gamma, beta, alpha) as the kernel takes them
+
+    def weight_shapes(self):
+        return {"gamma": ((self.width,), "ones"), "beta": ((self.width,), "normal"), "alpha": ((), "ones")}
+
+    def load(self, gamma: torch.Tensor, beta: torch.Tensor, alpha: torch.Tensor) -> None:
+        if tuple(gamma.shape) != (self.width,) or tuple(beta.shape) != (self.width,) or alpha.numel() != 1:
+            raise ValueError(f"norm weights of shapes {tuple(gamma.shape)}, {tuple(beta.shape)}, {tuple(alpha.shape)} do "
+                             f"not fit a width of {self.width}")
+        f32 = lambda t: t.to(device=self.device, dtype=torch.float32).contiguous()     # noqa: E731
+        self.args = (f32(gamma), f32(beta), float(alpha))
+
+    def forward(self, x: torch.Tensor, out: torch.Tensor, row_index: Optional[torch.Tensor] = None,
+                clear: Optional[torch.Tensor] = None, clear2: Optional[torch.Tensor] = None) -> None:
+        ops.tanh_norm(x, norm_x=self.args, x_out=out, row_index=row_index, clear=clear, clear2=clear2)
+
+    def add_normed(self, y: Optional[torch.Tensor], residual: torch.Tensor, mult: float,
+                   x_out: Optional[torch.Tensor] = None, clear: Optional[torch.Tensor] = None,
+                   clear2: Optional[torch.Tensor] = None) -> None:
+        ops.tanh_norm(residual, y=y, norm_y=self.args, mult=mult, x_out=x_out, clear=clear, clear2=clear2)
+
+    def add_normed_then(self, y: torch.Tensor, residual: torch.Tensor, mult: float, next_norm: Norm, x_out: torch.Tensor,
+                        clear: Optional[torch.Tensor] = None) -> None:
+        if not isinstance(next_norm, DynamicTanh):
+            super().add_normed_then(y, residual, mult, next_norm, x_out, clear)
+            return
+        ops.tanh_norm(residual, y=y, norm_y=self.args, mult=mult, norm_x=next_norm.args, x_out=x_out, clear=clear)
+
+    def replace(self, x: torch.Tensor) -> None:
+        """x = norm(x) in place."""
+        ops.tanh_norm(x, norm_y=self.args, replace=True)
+
+
+register_part("norm", "dynamic_tanh", DynamicTanh)

@@ -21,7 +21,9 @@ its largest score, and only experts of the `keep` best groups can be chosen.  `w
 multiplies the expert's output, out = sum over the chosen e of s_e expert_e(h).  `shared_size`: one more gated
 feed-forward of that inner width runs for every token and is added; with `shared_gate` it is multiplied by
 sigmoid(wsg . h), one number per token (the gate's row rides along in the router's product, and because the last
-product is linear the gate multiplies the rows that product reads).
+product is linear the gate multiplies the rows that product reads).  `correction`: a number per expert is added to the
+scores that the choice goes by, and to nothing else (a token's experts are those with the largest corrected scores, its
+weights their scores without the correction).  `scale`: the weights are multiplied by it.
 """
 from __future__ import annotations
 
@@ -41,13 +43,15 @@ MAX_STREAM_PAIRS = 65535  # pairs of one launch of the streaming kernels
 class RoutedExperts(FeedForward):
     def __init__(self, hidden_size: int, intermediate_size: int, experts: int, top: int, score: str = "sigmoid",
                  groups: Optional[tuple] = None, weight_on: str = "input", shared_size: Optional[int] = None,
-                 shared_gate: bool = False,
+                 shared_gate: bool = False, correction: bool = False, scale: float = 1.0,
                  dtype: torch.dtype = torch.bfloat16, device: torch.device = torch.device("cuda")):
         if not 1 <= top <= experts:
             raise ValueError(f"a token uses {top} of {experts} experts")
         if score not in ("sigmoid", "softmax") or weight_on not in ("input", "output"):
             raise ValueError(f"scores are 'sigmoid' or 'softmax' and weigh the 'input' or the 'output', got "
                              f"{score!r}, {weight_on!r}")
+        self.has_correction, self.weight_scale = bool(correction), float(scale)
+        self.correction: Optional[torch.Tensor] = None
         self.softmax, self.weight_on_output = score == "softmax", weight_on == "output"
         self.groups, self.keep = (0, 0) if groups is None else (int(groups[0]), int(groups[1]))
         if groups is not None and (self.groups < 1 or self.groups > 64 or experts % self.groups
@@ -80,6 +84,8 @@ class RoutedExperts(FeedForward):
     def weight_shapes(self):
         W, F = self.hidden_size, self.intermediate_size
         shapes = {"router": ((self.experts, W), "normal")}
+        if self.has_correction:
+            shapes["correction"] = ((self.experts,), "normal")
         for e in range(self.experts):
             shapes.update({f"e{e}_gate": ((F, W), "normal"), f"e{e}_up": ((F, W), "normal"),
                            f"e{e}_down": ((W, F), "normal")})
@@ -92,7 +98,12 @@ class RoutedExperts(FeedForward):
 
     def load(self, router: torch.Tensor, shared_gate: Optional[torch.Tensor] = None,
              shared_up: Optional[torch.Tensor] = None, shared_down: Optional[torch.Tensor] = None,
-             shared_sg: Optional[torch.Tensor] = None, **experts: torch.Tensor) -> None:
+             shared_sg: Optional[torch.Tensor] = None, correction: Optional[torch.Tensor] = None,
+             **experts: torch.Tensor) -> None:
+        if self.has_correction:
+            if correction is None or tuple(correction.shape) != (self.experts,):
+                raise ValueError(f"the router needs a correction for each of its {self.experts} experts")
+            self.correction = correction.to(device=self.device, dtype=torch.float32).contiguous()
         self.router.load([router] + ([shared_sg] if self.shared_gate else []))
         if self.shared_size is not None:
             self.shared_gate_up.load(shared_gate, shared_up)
@@ -134,7 +145,7 @@ class RoutedExperts(FeedForward):
         sel_e = ws.get("router_experts", (T, self.top), torch.int32)
         sel_w = ws.get("router_weights", (T, self.top), torch.float32)
         ops.route_topk(logits, self.top, sel_e, sel_w, softmax=self.softmax, groups=self.groups, keep=self.keep,
-                       experts=self.experts)
+                       experts=self.experts, correction=self.correction, scale=self.weight_scale)
         pairs = T * self.top
         if self.dtype == torch.bfloat16 and not ctx.is_decode and pairs > FEW_PAIRS:
             if self.grouped:

@@ -1,7 +1,8 @@
 """Transforms of whole tensors of a model (`ModelSpec.embedding_transforms`, `logit_transforms`).
 
 `scale_soft_cap`: t <- cap * tanh(t * scale / cap) in place on float32 (a scale on the logits and
-a soft cap that keeps them inside (-cap, cap)); without a cap it is the scale alone."""
+a soft cap that keeps them inside (-cap, cap)); without a cap it is the scale alone.
+`dynamic_tanh`: t <- tanh(alpha t) * gamma + beta feature by feature (`parts.norm`), a norm on the embedding's output."""
 from __future__ import annotations
 
 from typing import Optional
@@ -10,6 +11,7 @@ import torch
 
 from ..kernels import ops
 from .base import Transform, register_part
+from .norm import DynamicTanh
 
 
 class ScaleSoftCap(Transform):
@@ -29,3 +31,20 @@ class ScaleSoftCap(Transform):
 
 
 register_part("transform", "scale_soft_cap", ScaleSoftCap)
+
+
+class DynamicTanhTransform(Transform):
+    def __init__(self, width: int, dtype=None, device=None):
+        self.norm = DynamicTanh(width, dtype, device)
+
+    def weight_shapes(self):
+        return self.norm.weight_shapes()
+
+    def load(self, **tensors: torch.Tensor) -> None:
+        self.norm.load(**tensors)
+
+    def forward(self, t: torch.Tensor, ctx) -> None:
+        self.norm.replace(t)
+
+
+register_part("transform", "dynamic_tanh", DynamicTanhTransform)
