@@ -21,7 +21,7 @@ the same weights (`checked`).
 
 Other modes (one JSON line per item, none of them the headline): --kernels,
 --prompt-lengths, --workload 1b|13b, --deterministic, --plan-check, --cpu-baseline, --float32, --design
-(the Zivitar design, or with --design-model ramolix | mugedra | buludra another one, beside the Llama decoder at equal layer
+(the Zivitar design, or with --design-model ramolix | mugedra | buludra | forisun another one, beside the Llama decoder at equal layer
 sizes: prompt and decode throughput, a step's kernels).
 """
 import argparse
@@ -723,16 +723,34 @@ def buludra_config(width, ff, heads, kv_heads, window, vocab):
                         dict(type="parallel", mixer=side, mlp=experts)])
 
 
-DESIGNS = {"zivitar": zivitar_config, "ramolix": ramolix_config, "mugedra": mugedra_config, "buludra": buludra_config}
+def forisun_config(width, ff, heads, kv_heads, window, vocab):
+    """Four layers at the size's width of latent attention with an output gate (128 unrotated and 64 rotated numbers per
+    query, values of 128, latents of 512, so cached rows of 576 numbers), the last one over the third's rows; the first
+    with a dense feed-forward (one matrix up, no gate), the others with eight experts of half the size's feed-forward
+    each of which a token uses two (the gated dense feed-forward's products per token)."""
+    mixer = dict(heads=heads, dim=128, rot_dim=64, vdim=128, kv_rank=512, scale=192 ** -0.5,
+                 rot=dict(dims=64, base=10000.0, scaling=dict(factor=4.0, original=4096, fast=32.0, slow=1.0)))
+    dense = dict(kind="dense", ff=ff)
+    experts = dict(kind="moe", expert=dict(ff=ff // 2), router=dict(experts=8, top=2, scale=1.5))
+    kind = "latent_attention"
+    return dict(architecture="Forisun", vocab=vocab, width=width, norm=dict(eps=1e-5), embedding=dict(scale=width ** 0.5),
+                layers=[dict(type=kind, mixer=mixer, mlp=dense), dict(type=kind, mixer=mixer, mlp=experts),
+                        dict(type=kind, mixer=mixer, mlp=experts), dict(type=kind, mixer=dict(mixer, kv_from=2), mlp=experts)])
+
+
+DESIGNS = {"zivitar": zivitar_config, "ramolix": ramolix_config, "mugedra": mugedra_config, "buludra": buludra_config,
+           "forisun": forisun_config}
 # what a design is measured beside: the Llama decoder, or the design whose kernels are most like its own
-BESIDE = {"zivitar": ("llama",), "ramolix": ("llama",), "mugedra": ("ramolix", "llama"), "buludra": ("mugedra", "llama")}
+BESIDE = {"zivitar": ("llama",), "ramolix": ("llama",), "mugedra": ("ramolix", "llama"), "buludra": ("mugedra", "llama"),
+          "forisun": ("ramolix", "buludra", "llama")}
 
 
 def run_design(which, design="zivitar"):
-    """A design (Zivitar, Ramolix, Mugedra or Buludra) beside the Llama decoder, Mugedra also beside Ramolix, whose
+    """A design (Zivitar, Ramolix, Mugedra, Buludra or Forisun) beside the Llama decoder, Mugedra also beside Ramolix, whose
     mixers (a recurrence behind a short convolution, attention over part of the keys) are most like its own, and
-    Buludra also beside Mugedra (two mixers side by side, a recurrence with a matrix state, experts), at equal
-    layer sizes (random weights, four layer runs):
+    Buludra also beside Mugedra (two mixers side by side, a recurrence with a matrix state, experts), and Forisun also
+    beside Ramolix (latent attention, norms on the sublayers' outputs) and Buludra (experts weighted on their outputs), at
+    equal layer sizes (random weights, four layer runs):
     prompt steps and decode steps timed on the device, and each step's kernels one by one (`Model.profile`).  One
     JSON line per (size, model)."""
     import torch
