@@ -127,33 +127,38 @@ __global__ void __launch_bounds__(256) latent_prep_kernel(const float* __restric
   if (row.c_cache != nullptr) write_row<TO>(pr, row, cs, t, scratch);
 }
 
-// V numbers of a weight row as floats
-template <typename TW, int V>
-__device__ __forceinline__ void load_w(const TW* p, float (&v)[V]) {
-  if constexpr (V == 1) {
-    v[0] = jb::to_f32(*p);
-  } else if constexpr (sizeof(TW) == 2) {
-    const uint4 a = *reinterpret_cast<const uint4*>(p);
-    const uint32_t w[4] = {a.x, a.y, a.z, a.w};
+// V numbers of a weight row (16 bytes, or one number): the bits are loaded early and unpacked late.
+template <int V> struct Raw {
+  uint4 bits;
+  template <typename T> __device__ __forceinline__ void load(const T* p) { bits = *reinterpret_cast<const uint4*>(p); }
+  template <typename T> __device__ __forceinline__ void unpack(float (&v)[V]) const {
+    const uint32_t w[4] = {bits.x, bits.y, bits.z, bits.w};
+    if constexpr (sizeof(T) == 2) {
 #pragma unroll
-    for (int i = 0; i < 4; ++i) {
-      v[2 * i] = __uint_as_float(w[i] << 16);
-      v[2 * i + 1] = __uint_as_float(w[i] & 0xffff0000u);
+      for (int i = 0; i < 4; ++i) {
+        v[2 * i] = __uint_as_float(w[i] << 16);
+        v[2 * i + 1] = __uint_as_float(w[i] & 0xffff0000u);
+      }
+    } else {
+#pragma unroll
+      for (int i = 0; i < 4; ++i) v[i] = __uint_as_float(w[i]);
     }
-  } else {
-    const float4 a = *reinterpret_cast<const float4*>(p);
-    v[0] = a.x, v[1] = a.y, v[2] = a.z, v[3] = a.w;
   }
-}
-template <typename TW> struct Width { static constexpr int N = sizeof(TW) == 2 ? 8 : 4; };   // numbers in 16 bytes
+};
+template <> struct Raw<1> {
+  float x;
+  template <typename T> __device__ __forceinline__ void load(const T* p) { x = jb::to_f32(*p); }
+  template <typename T> __device__ __forceinline__ void unpack(float (&v)[1]) const { v[0] = x; }
+};
 
 constexpr int QT = 8;             // tokens of a block of latent_queries
 constexpr int Q_THREADS = 128;
 
 // q_out[t, h, :n] = sum_j q[t, h, j] uk[h d + j, :], q_out[t, h, n : n + r] = the turned part, the rest zero; and, by
-// the blocks behind the heads' (blockIdx.x == H * chunks: one block per token tile), the tokens' rows.
+// the blocks behind the heads' (blockIdx.x >= H * chunks: a block per token), the tokens' rows.
 // A block owns (head, a chunk of COLS latent columns, QT tokens): COLS / V threads a row of uk, the others take other
-// rows j; the partial sums meet in shared memory.
+// rows j; the partial sums meet in shared memory.  The first rows of uk are asked for before the wait on the kernel
+// that makes the projections.
 template <typename T, int V>
 __global__ void __launch_bounds__(Q_THREADS) latent_queries_kernel(
     const float* __restrict__ proj, int ld, int q_col, int H, int d, int r, int n, int dp, const T* __restrict__ uk,
@@ -164,19 +169,27 @@ __global__ void __launch_bounds__(Q_THREADS) latent_queries_kernel(
   extern __shared__ __align__(16) float sm[];   // q [QT][d], then the slices' sums [SL][QT][COLS]
   __shared__ float scratch[33];
   jb::pdl_launch_dependents();
-  jb::pdl_wait();
   const int chunks = (n + COLS - 1) / COLS;
   const int t0 = blockIdx.y * QT, nt = min(QT, n_tokens - t0);
   const int half = r >> 1;
-  if (blockIdx.x == H * chunks) {
-    for (int k = 0; k < nt; ++k) {
-      const int t = t0 + k;
-      const float* cs = table != nullptr && r > 0 ? table + (size_t)positions[t] * half * 2 : nullptr;
-      write_row<T>(proj + (size_t)t * ld, row, cs, t, scratch);
-    }
+  if (blockIdx.x >= H * chunks) {
+    jb::pdl_wait();
+    const int t = t0 + blockIdx.x - H * chunks;
+    if (t >= n_tokens) return;
+    const float* cs = table != nullptr && r > 0 ? table + (size_t)positions[t] * half * 2 : nullptr;
+    write_row<T>(proj + (size_t)t * ld, row, cs, t, scratch);
     return;
   }
   const int h = blockIdx.x / chunks, chunk = blockIdx.x - h * chunks;
+  const int ct = threadIdx.x % CT, sl = threadIdx.x / CT;
+  const int col = chunk * COLS + ct * V;
+  const bool active = col < n;                  // with V > 1 n is a multiple of V: no column group is cut
+  const T* w = uk + (size_t)h * d * n + (active ? col : 0);
+  constexpr int AHEAD = 8;                      // rows of uk a thread has in flight
+  Raw<V> raw[AHEAD];
+#pragma unroll
+  for (int i = 0; i < AHEAD; ++i) raw[i].load(w + (size_t)min(sl + i * SL, d - 1) * n);
+  jb::pdl_wait();
   float* q_s = sm;
   float* part = sm + (QT * d + 3) / 4 * 4;
   for (int i = threadIdx.x; i < nt * d; i += Q_THREADS)
@@ -196,24 +209,28 @@ __global__ void __launch_bounds__(Q_THREADS) latent_queries_kernel(
     }
   }
   __syncthreads();
-  const int ct = threadIdx.x % CT, sl = threadIdx.x / CT;
-  const int col = chunk * COLS + ct * V;
   float acc[QT][V];
 #pragma unroll
   for (int k = 0; k < QT; ++k)
 #pragma unroll
     for (int v = 0; v < V; ++v) acc[k][v] = 0.0f;
-  if (col < n) {                                // with V > 1 n is a multiple of V: no column group is cut
-    const T* w = uk + (size_t)h * d * n + col;
-#pragma unroll 4
-    for (int j = sl; j < d; j += SL) {
-      float wv[V];
-      load_w<T, V>(w + (size_t)j * n, wv);
+  for (int j0 = sl; j0 < d; j0 += AHEAD * SL) {
+    if (j0 != sl) {
 #pragma unroll
-      for (int k = 0; k < QT; ++k) {
-        const float x = k < nt ? q_s[k * d + j] : 0.0f;
+      for (int i = 0; i < AHEAD; ++i) raw[i].load(w + (size_t)min(j0 + i * SL, d - 1) * n);
+    }
 #pragma unroll
-        for (int v = 0; v < V; ++v) acc[k][v] = fmaf(wv[v], x, acc[k][v]);
+    for (int i = 0; i < AHEAD; ++i) {
+      const int j = j0 + i * SL;
+      if (j < d && active) {
+        float wv[V];
+        raw[i].template unpack<T>(wv);
+#pragma unroll
+        for (int k = 0; k < QT; ++k) {
+          const float x = k < nt ? q_s[k * d + j] : 0.0f;
+#pragma unroll
+          for (int v = 0; v < V; ++v) acc[k][v] = fmaf(wv[v], x, acc[k][v]);
+        }
       }
     }
   }
@@ -233,102 +250,143 @@ __global__ void __launch_bounds__(Q_THREADS) latent_queries_kernel(
 }
 
 constexpr int VT = 4;              // tokens of a block of latent_values
-constexpr int V_WARPS = 8, V_ROWS = 8;
+constexpr int V_WARPS = 8, V_ROWS = 4;
 
 // out[t, h, c] = (uv[h e + c, :] . o[t, h]) * sigmoid(gate[t, h e + c]) for c < e, zero for e <= c < ep.  o comes from
 // `o_rows` [T, H, n] (splits == 0), or from the key splits' partial sums: part_o [T, H, splits, n] and part_ml
 // [T, H, splits, 2] (maximum in units of log2, sum), o = sum_s f_s part_o[s] / sum_s f_s l_s with f_s = 2^(m_s - max).
-// A block owns (a chunk of V_WARPS * V_ROWS value rows, head, VT tokens); a warp takes rows one after another.
+// A block owns (a chunk of V_WARPS * V_ROWS value rows, head, VT tokens); a warp takes V_ROWS rows, whose first columns
+// it asks for before the wait on the attention kernel.
 template <typename T, int V>
 __global__ void __launch_bounds__(V_WARPS * 32) latent_values_kernel(
     const T* __restrict__ o_rows, const float* __restrict__ part_o, const float* __restrict__ part_ml, int splits,
     const T* __restrict__ uv, const float* __restrict__ gate, int ld_gate, T* __restrict__ out, int n_tokens, int H, int n,
     int e, int ep) {
-  extern __shared__ __align__(16) float o_s[];   // [VT][n padded to V], then the splits' factors [VT][splits]
+  extern __shared__ __align__(16) float o_s[];   // [VT][n padded to 8], then the splits' factors [VT][splits]
   jb::pdl_launch_dependents();
-  jb::pdl_wait();
   const int h = blockIdx.y, t0 = blockIdx.z * VT, nt = min(VT, n_tokens - t0);
-  const int np = (n + 7) / 8 * 8;
+  const int np = (n + 7) / 8 * 8, nv = np / V;
+  auto place = [&](int c) { return (c % V) * nv + c / V; };      // column c of a row of o_s: lanes read neighbours
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const int c0 = (blockIdx.x * V_WARPS + warp) * V_ROWS;
+  const T* w[V_ROWS];
+  Raw<V> raw[V_ROWS][2];                         // the columns lane V and (lane + 32) V of the warp's rows
+#pragma unroll
+  for (int q = 0; q < V_ROWS; ++q) {
+    w[q] = uv + ((size_t)h * e + min(c0 + q, e - 1)) * n;
+#pragma unroll
+    for (int x = 0; x < 2; ++x)
+      if ((lane + 32 * x) * V < n) raw[q][x].load(w[q] + (lane + 32 * x) * V);
+  }
+  jb::pdl_wait();
   if (splits > 0) {
     float* f_s = o_s + VT * np;
-    if (threadIdx.x < nt) {
-      const float* ml = part_ml + ((size_t)(t0 + threadIdx.x) * H + h) * splits * 2;
+    if (warp < nt) {                             // a warp per token: lanes over the splits
+      const float* ml = part_ml + ((size_t)(t0 + warp) * H + h) * splits * 2;
       float m = -CUDART_INF_F, l = 0.0f;
-      for (int s = 0; s < splits; ++s) m = fmaxf(m, ml[2 * s]);
-      for (int s = 0; s < splits; ++s) l += ml[2 * s + 1] * exp2f(ml[2 * s] - m);   // a split without keys weighs 0
-      for (int s = 0; s < splits; ++s) f_s[threadIdx.x * splits + s] = exp2f(ml[2 * s] - m) / l;
+      for (int s = lane; s < splits; s += 32) m = fmaxf(m, ml[2 * s]);
+      m = jb::warp_max(m);
+      for (int s = lane; s < splits; s += 32) {
+        const float f = exp2f(ml[2 * s] - m);    // a split without keys weighs 0
+        f_s[warp * splits + s] = f;
+        l = fmaf(ml[2 * s + 1], f, l);
+      }
+      const float inv = 1.0f / jb::warp_sum(l);
+      for (int s = lane; s < splits; s += 32) f_s[warp * splits + s] *= inv;
     }
     __syncthreads();
-    for (int i = threadIdx.x; i < nt * n; i += blockDim.x) {
-      const int k = i / n, c = i % n;
-      const float* p = part_o + ((size_t)(t0 + k) * H + h) * splits * n + c;
-      float v = 0.0f;
+    if (n % 4 == 0) {
+      const int n4 = n >> 2;
+      for (int i = threadIdx.x; i < nt * n4; i += blockDim.x) {
+        const int k = i / n4, c = i - k * n4;
+        const float4* p = reinterpret_cast<const float4*>(part_o + ((size_t)(t0 + k) * H + h) * splits * n) + c;
+        float4 v = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
 #pragma unroll 8
-      for (int s = 0; s < splits; ++s) v = fmaf(f_s[k * splits + s], p[(size_t)s * n], v);
-      o_s[k * np + c] = v;
+        for (int s = 0; s < splits; ++s) {
+          const float f = f_s[k * splits + s];
+          const float4 x = p[(size_t)s * n4];
+          v.x = fmaf(f, x.x, v.x), v.y = fmaf(f, x.y, v.y), v.z = fmaf(f, x.z, v.z), v.w = fmaf(f, x.w, v.w);
+        }
+        float* o = o_s + k * np;
+        o[place(4 * c)] = v.x, o[place(4 * c + 1)] = v.y, o[place(4 * c + 2)] = v.z, o[place(4 * c + 3)] = v.w;
+      }
+    } else {
+      for (int i = threadIdx.x; i < nt * n; i += blockDim.x) {
+        const int k = i / n, c = i - k * n;
+        const float* p = part_o + ((size_t)(t0 + k) * H + h) * splits * n + c;
+        float v = 0.0f;
+#pragma unroll 8
+        for (int s = 0; s < splits; ++s) v = fmaf(f_s[k * splits + s], p[(size_t)s * n], v);
+        o_s[k * np + place(c)] = v;
+      }
     }
   } else {
     for (int i = threadIdx.x; i < nt * n; i += blockDim.x)
-      o_s[(i / n) * np + i % n] = jb::to_f32(o_rows[((size_t)(t0 + i / n) * H + h) * n + i % n]);
+      o_s[(i / n) * np + place(i % n)] = jb::to_f32(o_rows[((size_t)(t0 + i / n) * H + h) * n + i % n]);
   }
   __syncthreads();
-  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-  const int c0 = blockIdx.x * V_WARPS * V_ROWS + warp * V_ROWS;
-#pragma unroll 1
-  for (int rr = 0; rr < V_ROWS; rr += 2) {       // two rows at a time: their loads are in flight together
-    const int c = c0 + rr;
-    if (c >= ep) break;
-    float acc[2][VT];
+  if (c0 >= ep) return;
+  float acc[V_ROWS][VT];
 #pragma unroll
-    for (int q = 0; q < 2; ++q)
+  for (int q = 0; q < V_ROWS; ++q)
 #pragma unroll
-      for (int k = 0; k < VT; ++k) acc[q][k] = 0.0f;
-    const T* w0 = uv + ((size_t)h * e + min(c, e - 1)) * n;
-    const T* w1 = uv + ((size_t)h * e + min(c + 1, e - 1)) * n;
-    for (int i = lane * V; i < n; i += 32 * V) {
-      float a[V], b[V];
-      load_w<T, V>(w0 + i, a);
-      load_w<T, V>(w1 + i, b);
+    for (int k = 0; k < VT; ++k) acc[q][k] = 0.0f;
+  auto add = [&](const Raw<V>* r, int stride, int i) {      // columns i .. i + V - 1 of the warp's rows
+#pragma unroll
+    for (int q = 0; q < V_ROWS; ++q) {
+      float a[V];
+      r[q * stride].template unpack<T>(a);
 #pragma unroll
       for (int k = 0; k < VT; ++k) {
         if (k < nt) {
 #pragma unroll
-          for (int v = 0; v < V; ++v) {
-            const float x = o_s[k * np + i + v];
-            acc[0][k] = fmaf(a[v], x, acc[0][k]);
-            acc[1][k] = fmaf(b[v], x, acc[1][k]);
-          }
+          for (int v = 0; v < V; ++v) acc[q][k] = fmaf(a[v], o_s[k * np + v * nv + i / V], acc[q][k]);
         }
       }
     }
+  };
 #pragma unroll
-    for (int q = 0; q < 2; ++q)
+  for (int x = 0; x < 2; ++x)
+    if ((lane + 32 * x) * V < n) add(&raw[0][x], 2, (lane + 32 * x) * V);
+  for (int i = (lane + 64) * V; i < n; i += 32 * V) {
+    Raw<V> more[V_ROWS];
 #pragma unroll
-      for (int k = 0; k < VT; ++k) {
-        const float v = jb::warp_sum(acc[q][k]);
-        if (lane == 0 && k < nt && c + q < ep) {
-          float y = 0.0f;
-          if (c + q < e) {
-            y = v;
-            if (gate != nullptr) y *= 1.0f / (1.0f + expf(-gate[(size_t)(t0 + k) * ld_gate + (size_t)h * e + c + q]));
-          }
-          out[((size_t)(t0 + k) * H + h) * ep + c + q] = jb::from_f32<T>(y);
-        }
-      }
+    for (int q = 0; q < V_ROWS; ++q) more[q].load(w[q] + i);
+    add(more, 1, i);
   }
+#pragma unroll
+  for (int q = 0; q < V_ROWS; ++q)
+#pragma unroll
+    for (int k = 0; k < VT; ++k) acc[q][k] = jb::warp_sum(acc[q][k]);
+  // lane q VT + k writes row q of token k
+#pragma unroll
+  for (int q = 0; q < V_ROWS; ++q)
+#pragma unroll
+    for (int k = 0; k < VT; ++k) {
+      const int c = c0 + q;
+      if (lane == q * VT + k && k < nt && c < ep) {
+        float y = 0.0f;
+        if (c < e) {
+          y = acc[q][k];
+          if (gate != nullptr) y *= 1.0f / (1.0f + expf(-gate[(size_t)(t0 + k) * ld_gate + (size_t)h * e + c]));
+        }
+        out[((size_t)(t0 + k) * H + h) * ep + c] = jb::from_f32<T>(y);
+      }
+    }
 }
 
-// rows[start[s] + i] = the cached row of position i of sequence s; one block per (page of the sequence, sequence),
-// rows of `vecs` 16-byte vectors.
+// rows[start[s] + i] = the cached row of position i of sequence s; a block per (GATHER rows of a page, sequence), rows
+// of `vecs` 16-byte vectors.
+constexpr int GATHER = 8;
 __global__ void __launch_bounds__(256) gather_rows_kernel(const uint4* __restrict__ cache, const int* __restrict__ block_table,
                                                           int max_pages, int page_size, const int* __restrict__ kv_len,
                                                           const int* __restrict__ start, uint4* __restrict__ rows, int vecs) {
   jb::pdl_launch_dependents();
   jb::pdl_wait();
-  const int s = blockIdx.y, first = blockIdx.x * page_size;
-  const int count = min(page_size, kv_len[s] - first);
+  const int s = blockIdx.y, first = blockIdx.x * GATHER;
+  const int count = min(GATHER, kv_len[s] - first);
   if (count <= 0) return;
-  const uint4* src = cache + (size_t)block_table[(size_t)s * max_pages + blockIdx.x] * page_size * vecs;
+  const uint4* src = cache + ((size_t)block_table[(size_t)s * max_pages + first / page_size] * page_size + first % page_size) * vecs;
   uint4* dst = rows + (size_t)(start[s] + first) * vecs;
   for (int i = threadIdx.x; i < count * vecs; i += blockDim.x) dst[i] = src[i];
 }
@@ -391,7 +449,7 @@ JB_EXPORT int jb_latent_queries(const float* proj, int ld, int q_col, int H, int
   const int chunks = (n + cols - 1) / cols;
   const size_t smem = ((size_t)(QT * d + 3) / 4 * 4 + (size_t)(Q_THREADS / 8) * QT * cols) * sizeof(float);
   JB_REFUSE(smem > 200 * 1024, "latent_queries: heads of %d numbers (%zu bytes) do not fit shared memory", d, smem);
-  jb::Launch cfg(dim3(H * chunks + (c_cache != nullptr ? 1 : 0), (T + QT - 1) / QT), dim3(Q_THREADS), smem, stream);
+  jb::Launch cfg(dim3(H * chunks + (c_cache != nullptr ? (T < QT ? T : QT) : 0), (T + QT - 1) / QT), dim3(Q_THREADS), smem, stream);
   cudaError_t e = cudaSuccess;
 #define JB_GO(T_, V_)                                                                                               \
   do {                                                                                                              \
@@ -454,8 +512,9 @@ JB_EXPORT int jb_latent_values(const void* o_rows, const float* part_o, const fl
 JB_EXPORT int jb_gather_rows(const void* cache, const int* block_table, int max_pages, int page_size, const int* kv_len,
                              const int* start, void* rows, int row_bytes, int n_seqs, int pages, cudaStream_t stream) {
   if (n_seqs <= 0 || pages <= 0) return 0;
+  JB_REFUSE(page_size % GATHER != 0, "gather_rows: pages of %d rows", page_size);
   JB_REFUSE(row_bytes % 16 != 0 || !aligned16(cache) || !aligned16(rows), "gather_rows: rows of %d bytes", row_bytes);
-  jb::Launch cfg(dim3(pages, n_seqs), dim3(256), 0, stream);
+  jb::Launch cfg(dim3(pages * (page_size / GATHER), n_seqs), dim3(256), 0, stream);
   return (int)cudaLaunchKernelEx(&cfg.c, gather_rows_kernel, (const uint4*)cache, block_table, max_pages, page_size, kv_len,
                                  start, (uint4*)rows, row_bytes / 16);
 }

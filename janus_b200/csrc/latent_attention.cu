@@ -5,11 +5,14 @@
 //
 // A block owns a tile of 16 MB rows = (token, head) pairs of one sequence (tokens outside, heads inside, as the queries
 // lie in memory) and a share of the keys (the key range cut into splits), in tiles of KT keys that come through a ring of
-// stages by cp.async.  A row of the tile in shared memory serves the scores (Q K^T, all D numbers) and the weighted sum
-// (P V, the first N): it is read from memory once.  Per tile, with eight warps:
-//   scores     a warp takes 8 keys (and, with 32 keys a tile, one half of the D numbers); partial sums in shared memory
-//   softmax    a warp takes 2 MB rows, online in float32 (exp2 of log2e-scaled scores); P in bfloat16 to shared memory
-//   sums       a warp takes every eighth group of 16 value columns of all rows, float32 in registers
+// stages by bulk copies, one a row (the copy engine puts the rows at a padded pitch, free of bank conflicts).  A row of
+// the tile in shared memory serves the scores (Q K^T, all D numbers) and the weighted sum (P V, the first N): it is read
+// from memory once.  Per tile, with sixteen warps:
+//   scores     a warp takes 8 keys and a half or a quarter of the D numbers; partial sums in shared memory
+//   softmax    a warp takes MB rows, online in float32 (exp2 of log2e-scaled scores); P in bfloat16 to shared memory
+//   sums       a warp takes every sixteenth group of 16 value columns of all rows, float32 in registers
+// Every wait for a copy is bounded in time and reports through `*status` (code 31); the rest of such a launch runs on
+// without waiting, and its result is not used.
 // Works for single tokens (their heads are the rows) and for several tokens a sequence alike; position i sees j <= i.
 // With one split the result is written as bfloat16 rows [T H, N], else as float32 partial sums (unnormalised), maxima and
 // sums for the kernel that follows.
@@ -18,6 +21,9 @@
 
 #include "common.cuh"
 
+#ifndef JB_LATENT_QREGS
+#define JB_LATENT_QREGS 40   // registers a thread may spend on its part of the queries; more of them stay in shared memory
+#endif
 #ifndef JB_LATENT_D
 #define JB_LATENT_D 576
 #endif
@@ -35,7 +41,7 @@ constexpr int DP = (D + 15) / 16 * 16;     // as the MMAs see a row
 constexpr int LD = DP + 8;                 // padded shared row: an odd number of 16-byte chunks, conflict-free ldmatrix
 constexpr int CHUNKS = D / 8;
 constexpr int PAGE = 64;
-constexpr int WARPS = 8, THREADS = WARPS * 32;
+constexpr int WARPS = 16, THREADS = WARPS * 32;
 constexpr int KT = D > 320 ? 32 : 64;      // keys per tile
 constexpr int GROUPS = KT / 8;             // groups of 8 keys
 constexpr int KS = WARPS / GROUPS;         // warps that share a group of keys, each with a part of the D numbers
@@ -49,7 +55,7 @@ constexpr float LOG2E = 1.4426950408889634f;
 constexpr int SMEM_LIMIT = 227 * 1024;
 
 constexpr int fixed_smem(int mb) {         // everything but the stages; 64 spare bytes: the last pair of steps reads past its row
-  return mb * 16 * LD * 2 + KS * mb * 16 * S_LD * 4 + mb * 16 * P_LD * 2 + 2 * mb * 16 * 4 + 64;
+  return mb * 16 * LD * 2 + KS * mb * 16 * S_LD * 4 + mb * 16 * P_LD * 2 + 2 * mb * 16 * 4 + 64 + 4 * 8;
 }
 constexpr int stages_for(int mb) {
   const int fit = (SMEM_LIMIT - fixed_smem(mb)) / (TILE * 2);
@@ -59,12 +65,41 @@ constexpr int smem_for(int mb) { return fixed_smem(mb) + stages_for(mb) * TILE *
 constexpr bool takes(int mb) { return stages_for(mb) >= 2; }
 
 __device__ __forceinline__ uint32_t smem_u32(const void* p) { return (uint32_t)__cvta_generic_to_shared(p); }
-__device__ __forceinline__ void cp_async16(void* dst, const void* src) {
-  asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(smem_u32(dst)), "l"(src) : "memory");
+constexpr unsigned long long WAIT_LIMIT_NS = 2000000000ull;
+__device__ __forceinline__ unsigned long long global_ns() {
+  unsigned long long t;
+  asm volatile("mov.u64 %0, %%globaltimer;" : "=l"(t));
+  return t;
 }
-__device__ __forceinline__ void cp_async_commit() { asm volatile("cp.async.commit_group;" ::: "memory"); }
-template <int G>
-__device__ __forceinline__ void cp_async_wait() { asm volatile("cp.async.wait_group %0;" ::"n"(G) : "memory"); }
+__device__ __forceinline__ uint32_t mbar_try(uint32_t bar, uint32_t parity) {
+  uint32_t ok;
+  asm volatile(
+      "{\n\t.reg .pred p;\n\t"
+      "mbarrier.try_wait.parity.shared::cta.b64 p, [%1], %2;\n\t"
+      "selp.u32 %0, 1, 0, p;\n\t}"
+      : "=r"(ok)
+      : "r"(bar), "r"(parity)
+      : "memory");
+  return ok;
+}
+__device__ __forceinline__ bool mbar_wait(uint32_t bar, uint32_t parity, int* status) {
+  if (mbar_try(bar, parity)) return true;
+  const unsigned long long t0 = global_ns();
+  for (;;) {
+#pragma unroll 1
+    for (int i = 0; i < 256; ++i)
+      if (mbar_try(bar, parity)) return true;
+    if (global_ns() - t0 > WAIT_LIMIT_NS) {
+      atomicCAS(status, 0, 31);
+      return false;
+    }
+  }
+}
+__device__ __forceinline__ void bulk_copy(uint32_t dst, const void* src, uint32_t bytes, uint32_t bar) {
+  asm volatile("cp.async.bulk.shared::cluster.global.mbarrier::complete_tx::bytes [%0], [%1], %2, [%3];" ::"r"(dst), "l"(src),
+               "r"(bytes), "r"(bar)
+               : "memory");
+}
 __device__ __forceinline__ void ldmatrix_x4(uint32_t (&r)[4], const void* p) {
   asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0, %1, %2, %3}, [%4];"
                : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3])
@@ -88,9 +123,9 @@ template <int MB>
 __global__ void __launch_bounds__(THREADS) latent_attention_kernel(
     const bf16* __restrict__ q, const bf16* __restrict__ cache, bf16* __restrict__ out, float* __restrict__ part_o,
     float* __restrict__ part_ml, const int* __restrict__ block_table, const int* __restrict__ q_start,
-    const int* __restrict__ kv_len, int H, int max_pages, float scale_log2, int n_splits) {
+    const int* __restrict__ kv_len, int H, int max_pages, float scale_log2, int n_splits, int* __restrict__ status) {
   constexpr int ROWS = MB * 16, STAGES = stages_for(MB), RPW = ROWS / WARPS;
-  constexpr bool Q_IN_REGS = WSTEPS * 4 * MB <= 80;
+  constexpr bool Q_IN_REGS = WSTEPS * 4 * MB <= JB_LATENT_QREGS;
   extern __shared__ __align__(16) uint8_t smem_raw[];
   bf16* q_s = reinterpret_cast<bf16*>(smem_raw);                    // [ROWS][LD]
   bf16* kv_s = q_s + ROWS * LD;                                     // [STAGES][KT][LD]
@@ -98,6 +133,7 @@ __global__ void __launch_bounds__(THREADS) latent_attention_kernel(
   bf16* p_s = reinterpret_cast<bf16*>(s_s + KS * ROWS * S_LD);      // [ROWS][P_LD]
   float* corr_s = reinterpret_cast<float*>(p_s + ROWS * P_LD);      // [ROWS]
   float* l_s = corr_s + ROWS;                                       // [ROWS]
+  uint64_t* bars = reinterpret_cast<uint64_t*>(l_s + ROWS);         // [STAGES]
   jb::pdl_launch_dependents();
   const int seq = blockIdx.z, split = blockIdx.y;
   const int qs = q_start[seq], q_len = q_start[seq + 1] - qs;
@@ -111,25 +147,33 @@ __global__ void __launch_bounds__(THREADS) latent_attention_kernel(
   const int* pages = block_table + (size_t)seq * max_pages;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
 
+  // tile j into its stage: one bulk copy a row, issued by the lanes of one warp
   auto issue = [&](int j) {
     const bf16* src = cache + ((size_t)pages[j * KT / PAGE] * PAGE + j * KT % PAGE) * D;
-    bf16* dst = kv_s + ((j - j0) % STAGES) * TILE;
-    for (int ch = threadIdx.x; ch < KT * CHUNKS; ch += THREADS)
-      cp_async16(dst + (ch / CHUNKS) * LD + ch % CHUNKS * 8, src + (size_t)ch * 8);
+    const uint32_t dst = smem_u32(kv_s + ((j - j0) % STAGES) * TILE), bar = smem_u32(bars + (j - j0) % STAGES);
+    if (lane == 0) asm volatile("mbarrier.arrive.expect_tx.shared::cta.b64 _, [%0], %1;" ::"r"(bar), "r"(KT * D * 2) : "memory");
+    __syncwarp();
+#pragma unroll
+    for (int r = lane; r < KT; r += 32) bulk_copy(dst + r * LD * 2, src + (size_t)r * D, D * 2, bar);
   };
   auto issue_first = [&]() {
-#pragma unroll
-    for (int s = 0; s < STAGES - 1; ++s) {
+#pragma unroll 1
+    for (int s = 0; s < STAGES - 1; ++s)
       if (j0 + s < j1) issue(j0 + s);
-      cp_async_commit();     // a group per stage, empty or not, keeps the count in step with the tiles
-    }
   };
+  if (threadIdx.x == 0) {
+    for (int s = 0; s < STAGES; ++s)
+      asm volatile("mbarrier.init.shared::cta.b64 [%0], 1;" ::"r"(smem_u32(bars + s)) : "memory");
+    asm volatile("fence.mbarrier_init.release.cluster;" ::: "memory");
+  }
+  __syncwarp();
   // rows below pos0 were cached by earlier steps: tiles that lie wholly below are asked for before the wait on the
-  // kernel that appends this step's rows
+  // kernel that appends this step's rows (the barriers' only other users meet them behind a barrier of the block)
   const bool early = min(j1, j0 + STAGES - 1) * KT <= pos0;
-  if (early) issue_first();
+  if (early && warp == 0) issue_first();
   jb::pdl_wait();
-  if (!early) issue_first();
+  if (!early && warp == 0) issue_first();
+  bool waits = true;
   if constexpr (DP != D) {   // columns that no load writes
     constexpr int PAD = DP > D ? DP - D : 1;
     for (int i = threadIdx.x; i < (ROWS + STAGES * KT) * PAD; i += THREADS)
@@ -172,10 +216,9 @@ __global__ void __launch_bounds__(THREADS) latent_attention_kernel(
       for (int e = 0; e < 4; ++e) o[b][u][0][e] = o[b][u][1][e] = 0.0f;
 
   for (int j = j0; j < j1; ++j) {
-    cp_async_wait<STAGES - 2>();
-    __syncthreads();         // tile j has landed for everybody, and everybody is done with tile j - 1
-    if (j + STAGES - 1 < j1) issue(j + STAGES - 1);
-    cp_async_commit();
+    __syncthreads();         // everybody is done with tile j - 1: its stage is free
+    if (warp == 0 && j + STAGES - 1 < j1) issue(j + STAGES - 1);
+    if (waits) waits = mbar_wait(smem_u32(bars + (j - j0) % STAGES), ((j - j0) / STAGES) & 1, status);
     const bf16* tile = kv_s + ((j - j0) % STAGES) * TILE;
     // ---- scores ----
     {
@@ -279,7 +322,6 @@ __global__ void __launch_bounds__(THREADS) latent_attention_kernel(
       }
     }
   }
-  cp_async_wait<0>();
   // ---- results ----
 #pragma unroll
   for (int i = 0; i < RPW; ++i) {
@@ -328,7 +370,8 @@ __global__ void __launch_bounds__(THREADS) latent_attention_kernel(
 
 template <int MB>
 int go(const bf16* q, const bf16* cache, bf16* out, float* part_o, float* part_ml, const int* block_table, const int* q_start,
-       const int* kv_len, int n_seqs, int max_q_len, int H, int max_pages, float scale, int n_splits, cudaStream_t stream) {
+       const int* kv_len, int n_seqs, int max_q_len, int H, int max_pages, float scale, int n_splits, int* status,
+       cudaStream_t stream) {
   if constexpr (takes(MB)) {
     static bool configured = false;
     if (!configured) {
@@ -340,7 +383,7 @@ int go(const bf16* q, const bf16* cache, bf16* out, float* part_o, float* part_m
     JB_REFUSE(tiles > 0x7fffffffLL, "latent_attention: %d tokens of %d heads are too many", max_q_len, H);
     jb::Launch cfg(dim3((unsigned)tiles, n_splits, n_seqs), dim3(THREADS), smem_for(MB), stream);
     return (int)cudaLaunchKernelEx(&cfg.c, latent_attention_kernel<MB>, q, cache, out, part_o, part_ml, block_table, q_start,
-                                   kv_len, H, max_pages, scale * LOG2E, n_splits);
+                                   kv_len, H, max_pages, scale * LOG2E, n_splits, status);
   } else {
     JB_REFUSE(true, "latent_attention: %d rows of %d numbers do not fit shared memory", MB * 16, D);
     return 0;
@@ -357,7 +400,7 @@ JB_EXPORT int jb_latent_attention_blocks() { return takes(2) ? 2 : takes(1) ? 1 
 JB_EXPORT int jb_latent_attention(const void* q, const void* cache, void* out, float* part_o, float* part_ml,
                                   const int* block_table, const int* q_start, const int* kv_len, int n_seqs, int max_q_len,
                                   int H, int d, int n, int page_size, int max_pages, float scale, int n_splits, int blocks,
-                                  cudaStream_t stream) {
+                                  int* status, cudaStream_t stream) {
   if (n_seqs <= 0 || max_q_len <= 0) return 0;
   JB_REFUSE(d != D || n != N, "latent_attention: built for rows of %d with values of %d, called with %d and %d", D, N, d, n);
   JB_REFUSE(page_size != PAGE, "latent_attention: page size %d (need %d)", page_size, PAGE);
@@ -366,7 +409,7 @@ JB_EXPORT int jb_latent_attention(const void* q, const void* cache, void* out, f
   JB_REFUSE(((uintptr_t)q | (uintptr_t)cache) & 15, "latent_attention: operands must be 16-byte aligned");
   if (blocks == 2)
     return go<2>((const bf16*)q, (const bf16*)cache, (bf16*)out, part_o, part_ml, block_table, q_start, kv_len, n_seqs,
-                 max_q_len, H, max_pages, scale, n_splits, stream);
+                 max_q_len, H, max_pages, scale, n_splits, status, stream);
   return go<1>((const bf16*)q, (const bf16*)cache, (bf16*)out, part_o, part_ml, block_table, q_start, kv_len, n_seqs,
-               max_q_len, H, max_pages, scale, n_splits, stream);
+               max_q_len, H, max_pages, scale, n_splits, status, stream);
 }

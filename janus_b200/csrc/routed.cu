@@ -324,6 +324,147 @@ __global__ void __launch_bounds__(DN_WARPS * 32) expert_down_kernel(
   }
 }
 
+// ---- the same two products on the tensor cores (bfloat16, widths of whole 32-number blocks) -----------------------
+// A warp multiplies 16 rows of one expert's matrix with up to 8 NG of the pairs that chose it (mma.sync m16n8k16: rows
+// of the weight on M, pairs on N), over every TC_WARPS-th block of 32 columns; the warps' sums meet in shared memory.
+// Nothing is staged: a lane holds eight neighbouring numbers of its row (one 16-byte load straight from memory), which
+// are two steps' fragments under a permutation of the columns that the pairs' fragments share (a dot product does not
+// mind the order), so the weights stream once, 16 bytes a lane, and the pairs' rows come from L2 the same way.
+constexpr int TC_WARPS = 8, NG = 4;
+
+__device__ __forceinline__ void mma_16816(float (&d)[4], uint32_t a0, uint32_t a1, uint32_t a2, uint32_t a3, uint32_t b0,
+                                          uint32_t b1) {
+  asm volatile(
+      "mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0, %1, %2, %3}, {%4, %5, %6, %7}, {%8, %9}, "
+      "{%0, %1, %2, %3};"
+      : "+f"(d[0]), "+f"(d[1]), "+f"(d[2]), "+f"(d[3])
+      : "r"(a0), "r"(a1), "r"(a2), "r"(a3), "r"(b0), "r"(b1));
+}
+__device__ __forceinline__ uint4 scaled(uint4 v, float s) {
+  uint32_t w[4] = {v.x, v.y, v.z, v.w};
+#pragma unroll
+  for (int i = 0; i < 4; ++i) {
+    const __nv_bfloat162 h = __floats2bfloat162_rn(__uint_as_float(w[i] << 16) * s, __uint_as_float(w[i] & 0xffff0000u) * s);
+    w[i] = *reinterpret_cast<const uint32_t*>(&h);
+  }
+  return make_uint4(w[0], w[1], w[2], w[3]);
+}
+// weights are read once: past L1, and first to leave L2
+__device__ __forceinline__ uint4 stream16(const bf16* p) {
+  uint4 v;
+  asm volatile("ld.global.nc.L1::no_allocate.L2::128B.v4.u32 {%0, %1, %2, %3}, [%4];"
+               : "=r"(v.x), "=r"(v.y), "=r"(v.z), "=r"(v.w)
+               : "l"(p));
+  return v;
+}
+
+// MATS = 2: act[pair][f] = gated(Wg_e[f] . x, Wu_e[f] . x), bfloat16, x = h[token of the pair] (times its weight with
+// weigh_input), 16 f a block.  MATS = 1: out[token of the pair][c] += (weight of the pair) Wd_e[c] . act[pair], 16
+// c a block.  K: the rows' width (a multiple of 32), R: the number of rows.
+template <int MATS>
+__global__ void __launch_bounds__(TC_WARPS * 32, 2) expert_tc_kernel(
+    const bf16* __restrict__ x, const int* __restrict__ sel_e, const float* __restrict__ sel_w, int top, int n_pairs,
+    const bf16* __restrict__ wa, const bf16* __restrict__ wb, bf16* __restrict__ act, float* __restrict__ out, int K, int R,
+    jb::Gate gate, int weigh) {
+  __shared__ float sum_s[TC_WARPS][MATS][16][8 * NG + 1];
+  __shared__ int list[TC_WARPS * 32];
+  __shared__ int count;
+  jb::pdl_launch_dependents();
+  jb::pdl_wait();
+  const int e = blockIdx.y, r0 = blockIdx.x * 16;
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, g = lane >> 2, c = lane & 3;
+  const size_t base_row = (size_t)e * R;
+  const bf16* rows[MATS][2];
+#pragma unroll
+  for (int q = 0; q < 2; ++q) {
+    const size_t off = (base_row + min(r0 + g + 8 * q, R - 1)) * K + 8 * c;
+    rows[0][q] = wa + off;
+    if constexpr (MATS == 2) rows[1][q] = wb + off;
+  }
+  const int blocks = K >> 5;
+  for (int base = 0; base < n_pairs; base += blockDim.x) {
+    const int n = pairs_of_expert(sel_e, n_pairs, base, e, list, &count);
+    for (int p0 = 0; p0 < n; p0 += 8 * NG) {
+      const int nb = min(8 * NG, n - p0), groups = (nb + 7) >> 3;
+      const bf16* xs[NG];
+      float sx[NG];
+#pragma unroll
+      for (int q = 0; q < NG; ++q) {
+        const int pair = list[p0 + min(8 * q + g, nb - 1)];       // (columns past the pairs repeat the last one)
+        xs[q] = x + (size_t)(MATS == 2 ? pair / top : pair) * K + 8 * c;
+        sx[q] = MATS == 2 && weigh ? sel_w[pair] : 1.0f;
+      }
+      float d[MATS][NG][4];
+#pragma unroll
+      for (int m = 0; m < MATS; ++m)
+#pragma unroll
+        for (int q = 0; q < NG; ++q) d[m][q][0] = d[m][q][1] = d[m][q][2] = d[m][q][3] = 0.0f;
+      constexpr int AHEAD = MATS == 2 ? 4 : 8;     // blocks of columns a warp has in flight
+      for (int b0 = warp; b0 < blocks; b0 += AHEAD * TC_WARPS) {
+        uint4 a[AHEAD][MATS][2];
+#pragma unroll
+        for (int i = 0; i < AHEAD; ++i) {
+          const int b = min(b0 + i * TC_WARPS, blocks - 1);
+#pragma unroll
+          for (int m = 0; m < MATS; ++m)
+#pragma unroll
+            for (int q = 0; q < 2; ++q) a[i][m][q] = stream16(rows[m][q] + (size_t)b * 32);
+        }
+#pragma unroll
+        for (int i = 0; i < AHEAD; ++i) {
+          const int b = b0 + i * TC_WARPS;
+          if (b >= blocks) break;
+#pragma unroll
+          for (int q = 0; q < NG; ++q) {
+            if (q >= groups) break;
+            uint4 v = *reinterpret_cast<const uint4*>(xs[q] + (size_t)b * 32);
+            if (MATS == 2 && weigh) v = scaled(v, sx[q]);
+#pragma unroll
+            for (int m = 0; m < MATS; ++m) {
+              const uint4 lo = a[i][m][0], hi = a[i][m][1];
+              mma_16816(d[m][q], lo.x, hi.x, lo.y, hi.y, v.x, v.y);
+              mma_16816(d[m][q], lo.z, hi.z, lo.w, hi.w, v.z, v.w);
+            }
+          }
+        }
+      }
+#pragma unroll
+      for (int m = 0; m < MATS; ++m)
+#pragma unroll
+        for (int q = 0; q < NG; ++q) {
+          if (q >= groups) break;
+          const int col = 8 * q + 2 * c;
+          sum_s[warp][m][g][col] = d[m][q][0];
+          sum_s[warp][m][g][col + 1] = d[m][q][1];
+          sum_s[warp][m][g + 8][col] = d[m][q][2];
+          sum_s[warp][m][g + 8][col + 1] = d[m][q][3];
+        }
+      __syncthreads();
+      for (int i = threadIdx.x; i < 16 * nb; i += blockDim.x) {
+        const int r = i & 15, k = i >> 4;
+        if (r0 + r >= R) continue;
+        float v[MATS];
+#pragma unroll
+        for (int m = 0; m < MATS; ++m) {
+          v[m] = 0.0f;
+#pragma unroll
+          for (int w = 0; w < TC_WARPS; ++w) v[m] += sum_s[w][m][r][k];
+        }
+        const int pair = list[p0 + k];
+        if constexpr (MATS == 2) {
+          act[(size_t)pair * R + r0 + r] = __float2bfloat16_rn(jb::gated(v[0], v[1], gate));
+        } else {
+          float* dst = out + (size_t)(pair / top) * R + r0 + r;
+          const float y = weigh ? v[0] * sel_w[pair] : v[0];
+          if (top == 1) *dst += y;                  // the token's only pair: nobody else adds here
+          else atomicAdd(dst, y);
+        }
+      }
+      __syncthreads();
+    }
+  }
+}
+
 constexpr int PLAN_THREADS = 1024, PLAN_MAX_EXPERTS = 1024;
 
 // Sorts the (token, choice) pairs by expert and lists the tiles of the two grouped products, in one block, so that
@@ -501,6 +642,28 @@ JB_EXPORT int jb_experts_few_tokens(const void* h, int x_dtype, const int* sel_e
 #undef JB_LAUNCH_GU
 #undef JB_LAUNCH_DN
   return (int)e;
+}
+
+// The bfloat16 form on the tensor cores: as jb_experts_few_tokens, W and F multiples of 32, act: bfloat16 scratch
+// [T top, F].
+JB_EXPORT int jb_experts_few_tokens_tc(const void* h, const int* sel_e, const float* sel_w, int top, const void* w_gate,
+                                       const void* w_up, const void* w_down, void* act, float* out, int T, int W, int F,
+                                       int E, float gate_limit, float gate_alpha, int weight_on_output, cudaStream_t stream) {
+  if (T <= 0) return 0;
+  const int pairs = T * top;
+  JB_REFUSE(E < 1 || E > 65535 || W % 32 || F % 32, "experts: %d experts of %d x %d", E, F, W);
+  JB_REFUSE(((uintptr_t)h | (uintptr_t)w_gate | (uintptr_t)w_up | (uintptr_t)w_down | (uintptr_t)act) & 15,
+            "experts: operands must be 16-byte aligned");
+  const jb::Gate gate{gate_limit, gate_alpha};
+  jb::Launch c1(dim3((F + 15) / 16, E), dim3(TC_WARPS * 32), 0, stream);
+  cudaError_t e = cudaLaunchKernelEx(&c1.c, expert_tc_kernel<2>, (const bf16*)h, sel_e, sel_w, top, pairs,
+                                     (const bf16*)w_gate, (const bf16*)w_up, (bf16*)act, (float*)nullptr, W, F, gate,
+                                     weight_on_output ? 0 : 1);
+  if (e != cudaSuccess) return (int)e;
+  jb::Launch c2(dim3((W + 15) / 16, E), dim3(TC_WARPS * 32), 0, stream);
+  return (int)cudaLaunchKernelEx(&c2.c, expert_tc_kernel<1>, (const bf16*)act, sel_e, sel_w, top, pairs,
+                                 (const bf16*)w_down, (const bf16*)nullptr, (bf16*)nullptr, out, F, W, gate,
+                                 weight_on_output);
 }
 
 // order, where: [pairs]; gu, dn: tables of the grouped products (4 ints and 4 more per item), see the kernel

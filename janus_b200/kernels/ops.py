@@ -67,7 +67,7 @@ _SIGNATURES = {
     "jb_join_norm": "pppppffpppfipipiiplplp", "jb_head_norm_gate": "ppipipfipiiiip", "jb_sigmoid_gate": "pipiiiiip",
     "jb_head_norm_rope_cache": "pippfpippipppiiiiiiiiifip",
     "jb_delta_rule": "piiiipiiippfppllppiiiiip",
-    "jb_route_topk": "piiippiiiipfp", "jb_experts_few_tokens": "pippipppippiiiiffip", "jb_expert_gather": "pippipiip",
+    "jb_route_topk": "piiippiiiipfp", "jb_experts_few_tokens": "pippipppippiiiiffip", "jb_expert_gather": "pippipiip", "jb_experts_few_tokens_tc": "pppipppppiiiiffip",
     "jb_expert_scatter": "pppipiip",
     "jb_gla_decay": "piiippfpiip", "jb_exp_gates": "piiippfppllppiip",
     "jb_gated_linear_scan": "piiiifpiippplppiiiiiippp", "jb_scale_rows_sigmoid": "pipiiip",
@@ -83,7 +83,7 @@ _SIGNATURES = {
     "jb_mamba2_scan": "piiipipppppllppiiiiiiippp", "jb_gated_group_rmsnorm": "ppipfpiiiip", "jb_pad_rows_bf16": "pipiip", "jb_scale_softcap": "plffp",
     "jb_gelu": "ppilp", "jb_tanh_norm": "ppppffippfpipiiplplp",
     "jb_latent_heads": "piiiiiipppiiiipfpppip", "jb_latent_queries": "piiiiiiippppiiipfppip", "jb_latent_values": "pppippipiiiiiip",
-    "jb_gather_rows": "ppiipppiiip", "jb_latent_attention": "ppppppppiiiiiiifiip", "jb_attention_tc_matrix": "ppppppiiiiiiiifpp",
+    "jb_gather_rows": "ppiipppiiip", "jb_latent_attention": "ppppppppiiiiiiifiipp", "jb_attention_tc_matrix": "ppppppiiiiiiiifpp",
 }
 _CTYPES = {"p": ctypes.c_void_p, "i": ctypes.c_int, "l": ctypes.c_longlong, "u": ctypes.c_ulonglong,
            "f": ctypes.c_float}
@@ -599,6 +599,7 @@ _GEMM_DEFINES = _defines_from_env("JANUS_GEMM_DEFINES") or None
 _PAIR_DEFINES = _defines_from_env("JANUS_GEMM_PAIR_DEFINES") or None
 _ATTN_TC_DEFINES = _defines_from_env("JANUS_ATTN_TC_DEFINES")
 _ATTN_DEFINES = _defines_from_env("JANUS_ATTN_DEFINES")
+_LATENT_DEFINES = _defines_from_env("JANUS_LATENT_DEFINES")
 _ATTN_TC = os.environ.get("JANUS_ATTN_TC", "1") != "0"     # 0: prompts attend on the mma.sync kernel
 
 
@@ -1641,6 +1642,25 @@ def experts_few_tokens(h: torch.Tensor, sel_e: torch.Tensor, sel_w: torch.Tensor
         int(bool(weight_on_output)), _stream()), "experts_few_tokens", kernels=2)
 
 
+def experts_few_tokens_tc(h: torch.Tensor, sel_e: torch.Tensor, sel_w: torch.Tensor, w_gate: torch.Tensor,
+                          w_up: torch.Tensor, w_down: torch.Tensor, act: torch.Tensor, out: torch.Tensor,
+                          gate_limit: float = 0.0, gate_alpha: float = 1.0, weight_on_output: bool = False) -> None:
+    """`experts_few_tokens` for bfloat16 rows of whole 32-number blocks, on the tensor cores: an expert's rows are
+    streamed once for up to 32 of the tokens that chose it; act: bfloat16 scratch [T top, F]."""
+    T, W = h.shape
+    E, F, _ = w_gate.shape
+    top = sel_e.shape[1]
+    for t, name, shape in ((h, "expert input", (T, W)), (w_gate, "experts' gate", (E, F, W)), (w_up, "experts' up", (E, F, W)),
+                           (w_down, "experts' down", (E, W, F)), (act, "experts' scratch", (T * top, F))):
+        _need(t, name, torch.bfloat16, shape)
+    _need(sel_e, "chosen experts", torch.int32, (T, top))
+    _need(sel_w, "experts' weights", torch.float32, (T, top))
+    _need(out, "experts' out", torch.float32, (T, W))
+    _check(_lib("routed").jb_experts_few_tokens_tc(
+        _ptr(h), _ptr(sel_e), _ptr(sel_w), top, _ptr(w_gate), _ptr(w_up), _ptr(w_down), _ptr(act), _ptr(out), T, W, F, E,
+        float(gate_limit), float(gate_alpha), int(bool(weight_on_output)), _stream()), "experts_few_tokens_tc", kernels=2)
+
+
 EXPERT_PLAN_MAX_EXPERTS = 1024
 
 
@@ -1913,7 +1933,7 @@ def gather_rows(pages: torch.Tensor, block_table: torch.Tensor, kv_len: torch.Te
 
 
 def _latent_attention_lib(stored: int, n: int):
-    return _lib("latent_attention", (int(stored), int(n)), lambda k: {"JB_LATENT_D": k[0], "JB_LATENT_N": k[1]})
+    return _lib("latent_attention", (int(stored), int(n)), lambda k: dict({"JB_LATENT_D": k[0], "JB_LATENT_N": k[1]}, **_LATENT_DEFINES))
 
 
 def latent_attention_smem(stored: int, n: int, blocks: int, stages: Optional[int] = None) -> int:
@@ -1921,9 +1941,9 @@ def latent_attention_smem(stored: int, n: int, blocks: int, stages: Optional[int
     constants of csrc/latent_attention.cu); 0 if its rows do not fit."""
     ld = (stored + 15) // 16 * 16 + 8
     kt = 32 if stored > 320 else 64
-    ks = 8 // (kt // 8)
+    ks = 16 // (kt // 8)
     rows = 16 * blocks
-    fixed = rows * ld * 2 + ks * rows * (kt + 4) * 4 + rows * (kt + 8) * 2 + 2 * rows * 4 + 64
+    fixed = rows * ld * 2 + ks * rows * (kt + 4) * 4 + rows * (kt + 8) * 2 + 2 * rows * 4 + 64 + 32
     fit = min(4, (227 * 1024 - fixed) // (kt * ld * 2)) if stages is None else stages
     return fixed + fit * kt * ld * 2 if fit >= 2 else 0
 
@@ -1945,7 +1965,7 @@ def latent_splits_for(n_seqs: int, row_tiles: int, max_kv_len: int, stored: int,
     kt = 32 if stored > 320 else 64
     tile_us = 0.15 + _LATENT_TILE_US_PER_KB * kt * stored * 2 / 1024
     tiles = max(1, (3 * max_kv_len // 4 + kt - 1) // kt)
-    per_sm = max(1, min(4, 228 * 1024 // (latent_attention_smem(stored, n, blocks) + 1024)))
+    per_sm = max(1, min(2, 228 * 1024 // (latent_attention_smem(stored, n, blocks) + 1024)))
     places = SM_COUNT_TARGET // 2 * per_sm
     best = (float("inf"), 1)
     for splits in (1, 2, 3, 4, 6, 8, 12, 16, 18, 24, 32, 48, 64):
@@ -1985,5 +2005,5 @@ def latent_attention(q: torch.Tensor, pages: torch.Tensor, out: Optional[torch.T
     _check(_latent_attention_lib(stored, n).jb_latent_attention(
         _ptr(q), _ptr(pages), _ptr(out), _ptr(part_o), _ptr(part_ml), _ptr(block_table), _ptr(q_start), _ptr(kv_len),
         n_seqs, max_q_len, heads, stored, n, page_size, block_table.shape[1], float(scale), int(n_splits), blocks,
-        _stream()), "latent_attention")
+        _ptr(kernel_status(q.device)), _stream()), "latent_attention")
     return (part_o, part_ml, n_splits) if n_splits > 1 else None

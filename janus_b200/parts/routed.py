@@ -6,8 +6,9 @@ largest scores (the lower index wins a tie) and their weights are those scores a
 weight multiplies the expert's INPUT: out = sum over the chosen e of expert_e(s_e h).
 
 Steps of few (token, expert) pairs, every single-token step among them, stream each chosen expert's rows once for
-up to four of the tokens that chose it (`ops.experts_few_tokens`: two launches with a block per (rows, expert),
-float32 sums, nothing read back by the host, so the step can be recorded into a CUDA graph).  Prompt steps of the
+up to 32 of the tokens that chose it (`ops.experts_few_tokens_tc`: two launches with a block per (rows, expert),
+float32 sums, nothing read back by the host, so the step can be recorded into a CUDA graph; widths that are no multiples
+of 32, and the float32 engine, take up to four tokens at a time on the CUDA cores, `ops.experts_few_tokens`).  Prompt steps of the
 bfloat16 engine with more pairs sort the (token, choice) pairs by expert, gather the weighted rows in that order and
 run the experts' two products on the tensor cores over their rows; the results are added back token by token in the
 order of the token's choices.  Where the sizes allow it (width and inner width multiples of 128) the sort is a kernel
@@ -80,6 +81,8 @@ class RoutedExperts(FeedForward):
         self.grouped = (dtype == torch.bfloat16 and hidden_size % 128 == 0 and intermediate_size % 128 == 0
                         and experts <= ops.EXPERT_PLAN_MAX_EXPERTS)
         self.gate_up_stack = self.down_stack = None
+        # steps of few pairs: on the tensor cores where rows are whole blocks of 32 numbers
+        self.streams_on_tensor_cores = (dtype == torch.bfloat16 and hidden_size % 32 == 0 and intermediate_size % 32 == 0)
 
     def weight_shapes(self):
         W, F = self.hidden_size, self.intermediate_size
@@ -152,6 +155,11 @@ class RoutedExperts(FeedForward):
                 self._grouped(x, sel_e, sel_w, residual, ctx)
             else:
                 self._by_expert(x, sel_e, sel_w, residual, ctx)
+            return
+        if self.streams_on_tensor_cores:
+            act = ws.get("experts_act_rows", (pairs, self.intermediate_size), self.dtype)
+            ops.experts_few_tokens_tc(x, sel_e, sel_w, self.w_gate, self.w_up, self.w_down, act, residual,
+                                      weight_on_output=self.weight_on_output)
             return
         act = ws.get("experts_act", (pairs, self.intermediate_size), torch.float32)
         rows = max(1, MAX_STREAM_PAIRS // self.top)

@@ -653,6 +653,35 @@ def test_router_with_corrected_choice_and_scaled_weights():
     assert se.tolist() == [[0, 1]] and rel_err(sw.cpu(), torch.sigmoid(z[:, :2].to(P.DT))) < 1e-6
 
 
+@gpu
+@pytest.mark.parametrize("on_output", [True, False])
+@pytest.mark.parametrize("T,W,F,E,top", [(3, 64, 96, 6, 2), (1, 32, 32, 3, 3), (40, 128, 160, 2, 1), (150, 96, 64, 5, 3),
+                                         (8, 2048, 1440, 4, 2)])
+def test_experts_of_few_pairs_on_the_tensor_cores_against_the_formula(T, W, F, E, top, on_output):
+    """Few and many pairs per expert (more than one launch group of 32 and one list of 256), experts that nobody chose,
+    the weight on the output and on the input; the results are added to what is there."""
+    from janus_b200.kernels import ops
+    g = torch.Generator().manual_seed(8)
+    h = bf(torch.randn(T, W, generator=g))
+    m = {k: bf(torch.randn(*shape, generator=g) * shape[-1] ** -0.5) for k, shape in
+         (("gate", (E, F, W)), ("up", (E, F, W)), ("down", (E, W, F)))}
+    pick = torch.stack([torch.randperm(max(E - 1, top), generator=g)[:top] for _ in range(T)])      # the last expert idles
+    weight = torch.rand(T, top, generator=g) + 0.2
+    out = torch.randn(T, W, generator=g)
+    want = out.to(P.DT)
+    for t in range(T):
+        for j in range(top):
+            e = int(pick[t, j])
+            x = h[t] if on_output else bf(h[t] * weight[t, j])
+            y = m["down"][e] @ bf(P.silu(m["gate"][e] @ x) * (m["up"][e] @ x))
+            want[t] += y * weight[t, j].to(P.DT) if on_output else y
+    cu = lambda t: t.to(torch.bfloat16).cuda()       # noqa: E731
+    got, act = out.cuda(), torch.empty(T * top, F, dtype=torch.bfloat16, device="cuda")
+    ops.experts_few_tokens_tc(cu(h), pick.int().cuda(), weight.cuda(), cu(m["gate"]), cu(m["up"]), cu(m["down"]), act, got,
+                              weight_on_output=on_output)
+    assert rel_err(got.cpu(), want) < 4e-3
+
+
 # ------------------------------------------------------------------------------------------------
 # on the device: the engine
 # ------------------------------------------------------------------------------------------------
