@@ -15,6 +15,7 @@
 //
 // The rotation turns the pair (i, i + r/2) by the position's angle; cos and sin come from a table [positions][r/2][2].
 // Pages of one place: [page][1][page_size][stored], stored >= n + r, extra columns never written (they stay zero).
+#include <cooperative_groups.h>
 #include <math_constants.h>
 #include <stdio.h>
 
@@ -22,6 +23,7 @@
 
 namespace {
 
+namespace cg = cooperative_groups;
 typedef __nv_bfloat16 bf16;
 
 struct Row {                 // the token's own row: where it comes from and where it goes (c_cache null: none)
@@ -79,7 +81,8 @@ __device__ __forceinline__ void store4(TO* p, const float4& v) {
   }
 }
 
-// Queries as heads (`dp` numbers each, the extra ones zero) and the token's row; one block per token.
+// Queries as heads (`dp` numbers each, the extra ones zero), one block per token (blockIdx.y == 0), and the token's row,
+// another one (blockIdx.y == 1).
 // VEC: d, r / 2, dp, the columns and the rows are whole groups of four at aligned addresses.
 template <typename TO, bool VEC>
 __global__ void __launch_bounds__(256) latent_prep_kernel(const float* __restrict__ proj, int ld, int q_col, int H, int d,
@@ -93,6 +96,10 @@ __global__ void __launch_bounds__(256) latent_prep_kernel(const float* __restric
   const float* pr = proj + (size_t)t * ld;
   const int half = r >> 1;
   const float* cs = table != nullptr && r > 0 ? table + (size_t)positions[t] * half * 2 : nullptr;
+  if (blockIdx.y == 1) {
+    write_row<TO>(pr, row, cs, t, scratch);
+    return;
+  }
   TO* q = q_out + (size_t)t * H * dp;
   if constexpr (VEC) {
     const int per = dp >> 2;                           // groups of four per stored head
@@ -124,7 +131,6 @@ __global__ void __launch_bounds__(256) latent_prep_kernel(const float* __restric
       q[i] = jb::from_f32<TO>(v);
     }
   }
-  if (row.c_cache != nullptr) write_row<TO>(pr, row, cs, t, scratch);
 }
 
 // V numbers of a weight row (16 bytes, or one number): the bits are loaded early and unpacked late.
@@ -256,7 +262,8 @@ constexpr int V_WARPS = 8, V_ROWS = 4;
 // `o_rows` [T, H, n] (splits == 0), or from the key splits' partial sums: part_o [T, H, splits, n] and part_ml
 // [T, H, splits, 2] (maximum in units of log2, sum), o = sum_s f_s part_o[s] / sum_s f_s l_s with f_s = 2^(m_s - max).
 // A block owns (a chunk of V_WARPS * V_ROWS value rows, head, VT tokens); a warp takes V_ROWS rows, whose first columns
-// it asks for before the wait on the attention kernel.
+// it asks for before the wait on the attention kernel.  The blocks of a head's chunks form a cluster: each of them joins
+// a part of o's columns and leaves it in the shared memory of all.
 template <typename T, int V>
 __global__ void __launch_bounds__(V_WARPS * 32) latent_values_kernel(
     const T* __restrict__ o_rows, const float* __restrict__ part_o, const float* __restrict__ part_ml, int splits,
@@ -264,6 +271,9 @@ __global__ void __launch_bounds__(V_WARPS * 32) latent_values_kernel(
     int e, int ep) {
   extern __shared__ __align__(16) float o_s[];   // [VT][n padded to 8], then the splits' factors [VT][splits]
   jb::pdl_launch_dependents();
+  cg::cluster_group cluster = cg::this_cluster();
+  const int members = (int)cluster.num_blocks(), rank = (int)cluster.block_rank();
+  if (members > 1) asm volatile("barrier.cluster.arrive.relaxed.aligned;" ::: "memory");   // (waited for before the first write to another block)
   const int h = blockIdx.y, t0 = blockIdx.z * VT, nt = min(VT, n_tokens - t0);
   const int np = (n + 7) / 8 * 8, nv = np / V;
   auto place = [&](int c) { return (c % V) * nv + c / V; };      // column c of a row of o_s: lanes read neighbours
@@ -279,6 +289,10 @@ __global__ void __launch_bounds__(V_WARPS * 32) latent_values_kernel(
       if ((lane + 32 * x) * V < n) raw[q][x].load(w[q] + (lane + 32 * x) * V);
   }
   jb::pdl_wait();
+  // the sum this lane will write: row my_c of token my_k; its gate is asked for early (no gate: z -> infinity, sigmoid 1)
+  const int my_c = c0 + (lane >> 1) / VT, my_k = (lane >> 1) % VT;
+  float z = CUDART_INF_F;
+  if (gate != nullptr && my_k < nt && my_c < e) z = gate[(size_t)(t0 + my_k) * ld_gate + (size_t)h * e + my_c];
   if (splits > 0) {
     float* f_s = o_s + VT * np;
     if (warp < nt) {                             // a warp per token: lanes over the splits
@@ -295,9 +309,17 @@ __global__ void __launch_bounds__(V_WARPS * 32) latent_values_kernel(
       for (int s = lane; s < splits; s += 32) f_s[warp * splits + s] *= inv;
     }
     __syncthreads();
+    if (members > 1) asm volatile("barrier.cluster.wait.aligned;" ::: "memory");
+    auto put = [&](int at, float v) {
+      if (members == 1) {
+        o_s[at] = v;
+      } else {
+        for (int m = 0; m < members; ++m) *cluster.map_shared_rank(o_s + at, m) = v;
+      }
+    };
     if (n % 4 == 0) {
       const int n4 = n >> 2;
-      for (int i = threadIdx.x; i < nt * n4; i += blockDim.x) {
+      for (int i = threadIdx.x + rank * blockDim.x; i < nt * n4; i += blockDim.x * members) {
         const int k = i / n4, c = i - k * n4;
         const float4* p = reinterpret_cast<const float4*>(part_o + ((size_t)(t0 + k) * H + h) * splits * n) + c;
         float4 v = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
@@ -307,30 +329,30 @@ __global__ void __launch_bounds__(V_WARPS * 32) latent_values_kernel(
           const float4 x = p[(size_t)s * n4];
           v.x = fmaf(f, x.x, v.x), v.y = fmaf(f, x.y, v.y), v.z = fmaf(f, x.z, v.z), v.w = fmaf(f, x.w, v.w);
         }
-        float* o = o_s + k * np;
-        o[place(4 * c)] = v.x, o[place(4 * c + 1)] = v.y, o[place(4 * c + 2)] = v.z, o[place(4 * c + 3)] = v.w;
+        const int o = k * np;
+        put(o + place(4 * c), v.x), put(o + place(4 * c + 1), v.y), put(o + place(4 * c + 2), v.z), put(o + place(4 * c + 3), v.w);
       }
     } else {
-      for (int i = threadIdx.x; i < nt * n; i += blockDim.x) {
+      for (int i = threadIdx.x + rank * blockDim.x; i < nt * n; i += blockDim.x * members) {
         const int k = i / n, c = i - k * n;
         const float* p = part_o + ((size_t)(t0 + k) * H + h) * splits * n + c;
         float v = 0.0f;
 #pragma unroll 8
         for (int s = 0; s < splits; ++s) v = fmaf(f_s[k * splits + s], p[(size_t)s * n], v);
-        o_s[k * np + place(c)] = v;
+        put(k * np + place(c), v);
       }
     }
+    if (members > 1) cluster.sync();
   } else {
     for (int i = threadIdx.x; i < nt * n; i += blockDim.x)
       o_s[(i / n) * np + place(i % n)] = jb::to_f32(o_rows[((size_t)(t0 + i / n) * H + h) * n + i % n]);
+    if (members > 1) asm volatile("barrier.cluster.wait.aligned;" ::: "memory");
   }
   __syncthreads();
   if (c0 >= ep) return;
-  float acc[V_ROWS][VT];
+  float acc[V_ROWS * VT];
 #pragma unroll
-  for (int q = 0; q < V_ROWS; ++q)
-#pragma unroll
-    for (int k = 0; k < VT; ++k) acc[q][k] = 0.0f;
+  for (int i = 0; i < V_ROWS * VT; ++i) acc[i] = 0.0f;
   auto add = [&](const Raw<V>* r, int stride, int i) {      // columns i .. i + V - 1 of the warp's rows
 #pragma unroll
     for (int q = 0; q < V_ROWS; ++q) {
@@ -340,7 +362,7 @@ __global__ void __launch_bounds__(V_WARPS * 32) latent_values_kernel(
       for (int k = 0; k < VT; ++k) {
         if (k < nt) {
 #pragma unroll
-          for (int v = 0; v < V; ++v) acc[q][k] = fmaf(a[v], o_s[k * np + v * nv + i / V], acc[q][k]);
+          for (int v = 0; v < V; ++v) acc[q * VT + k] = fmaf(a[v], o_s[k * np + v * nv + i / V], acc[q * VT + k]);
         }
       }
     }
@@ -354,25 +376,21 @@ __global__ void __launch_bounds__(V_WARPS * 32) latent_values_kernel(
     for (int q = 0; q < V_ROWS; ++q) more[q].load(w[q] + i);
     add(more, 1, i);
   }
+  // the warp's 16 sums: every exchange halves what a lane still holds, so lanes 2 i and 2 i + 1 end with sum i
+  static_assert(V_ROWS * VT == 16, "sixteen sums a warp");
 #pragma unroll
-  for (int q = 0; q < V_ROWS; ++q)
+  for (int half = 8; half >= 1; half >>= 1) {
+    const bool upper = lane & (2 * half);
 #pragma unroll
-    for (int k = 0; k < VT; ++k) acc[q][k] = jb::warp_sum(acc[q][k]);
-  // lane q VT + k writes row q of token k
-#pragma unroll
-  for (int q = 0; q < V_ROWS; ++q)
-#pragma unroll
-    for (int k = 0; k < VT; ++k) {
-      const int c = c0 + q;
-      if (lane == q * VT + k && k < nt && c < ep) {
-        float y = 0.0f;
-        if (c < e) {
-          y = acc[q][k];
-          if (gate != nullptr) y *= 1.0f / (1.0f + expf(-gate[(size_t)(t0 + k) * ld_gate + (size_t)h * e + c]));
-        }
-        out[((size_t)(t0 + k) * H + h) * ep + c] = jb::from_f32<T>(y);
-      }
+    for (int i = 0; i < half; ++i) {
+      const float send = upper ? acc[i] : acc[i + half];
+      const float keep = upper ? acc[i + half] : acc[i];
+      acc[i] = keep + __shfl_xor_sync(0xffffffffu, send, 2 * half);
     }
+  }
+  const float sum = acc[0] + __shfl_xor_sync(0xffffffffu, acc[0], 1);
+  if (lane % 2 == 0 && my_k < nt && my_c < ep)
+    out[((size_t)(t0 + my_k) * H + h) * ep + my_c] = jb::from_f32<T>(my_c < e ? sum * (1.0f / (1.0f + expf(-z))) : 0.0f);
 }
 
 // rows[start[s] + i] = the cached row of position i of sequence s; a block per (GATHER rows of a page, sequence), rows
@@ -417,7 +435,7 @@ JB_EXPORT int jb_latent_heads(const float* proj, int ld, int q_col, int H, int d
   JB_REFUSE(dp < d + r, "latent_heads: heads of %d numbers cannot be stored in %d columns", d + r, dp);
   const bool vec = ld % 4 == 0 && q_col % 4 == 0 && d % 4 == 0 && r % 8 == 0 && dp % 4 == 0 && aligned16(proj) &&
                    aligned16(q_out) && (table == nullptr || aligned16(table));
-  jb::Launch cfg(dim3(T), dim3(256), 0, stream);
+  jb::Launch cfg(dim3(T, c_cache != nullptr ? 2 : 1), dim3(256), 0, stream);
   cudaError_t e;
 #define JB_GO(TO, VEC) \
   e = cudaLaunchKernelEx(&cfg.c, latent_prep_kernel<TO, VEC>, proj, ld, q_col, H, d, r, dp, table, positions, (TO*)q_out, row)
@@ -484,7 +502,15 @@ JB_EXPORT int jb_latent_values(const void* o_rows, const float* part_o, const fl
   const size_t smem = ((size_t)VT * ((n + 7) / 8 * 8) + (size_t)VT * splits) * sizeof(float);
   JB_REFUSE(smem > 200 * 1024, "latent_values: latents of %d numbers do not fit shared memory", n);
   const int rows = V_WARPS * V_ROWS;
-  jb::Launch cfg(dim3((ep + rows - 1) / rows, H, (T + VT - 1) / VT), dim3(V_WARPS * 32), smem, stream);
+  const int chunks = (ep + rows - 1) / rows;
+  jb::Launch cfg(dim3(chunks, H, (T + VT - 1) / VT), dim3(V_WARPS * 32), smem, stream);
+  cudaLaunchAttribute attrs[2];
+  attrs[0].id = cudaLaunchAttributeClusterDimension;
+  attrs[0].val.clusterDim.x = chunks % 8 == 0 ? 8 : chunks % 4 == 0 ? 4 : chunks % 2 == 0 ? 2 : 1;
+  attrs[0].val.clusterDim.y = attrs[0].val.clusterDim.z = 1;
+  if (cfg.c.numAttrs) attrs[1] = cfg.attr[0];
+  cfg.c.attrs = attrs;
+  cfg.c.numAttrs += 1;
   cudaError_t err = cudaSuccess;
 #define JB_GO(T_, V_)                                                                                               \
   do {                                                                                                              \

@@ -330,7 +330,7 @@ __global__ void __launch_bounds__(DN_WARPS * 32) expert_down_kernel(
 // Nothing is staged: a lane holds eight neighbouring numbers of its row (one 16-byte load straight from memory), which
 // are two steps' fragments under a permutation of the columns that the pairs' fragments share (a dot product does not
 // mind the order), so the weights stream once, 16 bytes a lane, and the pairs' rows come from L2 the same way.
-constexpr int TC_WARPS = 8, NG = 4;
+constexpr int TC_WARPS = 8, NG = 2;
 
 __device__ __forceinline__ void mma_16816(float (&d)[4], uint32_t a0, uint32_t a1, uint32_t a2, uint32_t a3, uint32_t b0,
                                           uint32_t b1) {
@@ -400,24 +400,30 @@ __global__ void __launch_bounds__(TC_WARPS * 32, 2) expert_tc_kernel(
 #pragma unroll
         for (int q = 0; q < NG; ++q) d[m][q][0] = d[m][q][1] = d[m][q][2] = d[m][q][3] = 0.0f;
       constexpr int AHEAD = MATS == 2 ? 4 : 8;     // blocks of columns a warp has in flight
-      for (int b0 = warp; b0 < blocks; b0 += AHEAD * TC_WARPS) {
+      // a warp's blocks come in neighbouring pairs (128 bytes of a row): pair p of the warp is pair p TC_WARPS + warp
+      const auto block = [&](int i) { return ((i >> 1) * TC_WARPS + warp) * 2 + (i & 1); };
+      for (int i0 = 0; block(i0) < blocks; i0 += AHEAD) {
         uint4 a[AHEAD][MATS][2];
 #pragma unroll
         for (int i = 0; i < AHEAD; ++i) {
-          const int b = min(b0 + i * TC_WARPS, blocks - 1);
+          const int b = min(block(i0 + i), blocks - 1);
 #pragma unroll
           for (int m = 0; m < MATS; ++m)
 #pragma unroll
             for (int q = 0; q < 2; ++q) a[i][m][q] = stream16(rows[m][q] + (size_t)b * 32);
         }
+        uint4 first[AHEAD];                                  // the first eight pairs' numbers for the same columns
+#pragma unroll
+        for (int i = 0; i < AHEAD; ++i)
+          first[i] = *reinterpret_cast<const uint4*>(xs[0] + (size_t)min(block(i0 + i), blocks - 1) * 32);
 #pragma unroll
         for (int i = 0; i < AHEAD; ++i) {
-          const int b = b0 + i * TC_WARPS;
+          const int b = block(i0 + i);
           if (b >= blocks) break;
 #pragma unroll
           for (int q = 0; q < NG; ++q) {
             if (q >= groups) break;
-            uint4 v = *reinterpret_cast<const uint4*>(xs[q] + (size_t)b * 32);
+            uint4 v = q == 0 ? first[i] : *reinterpret_cast<const uint4*>(xs[q] + (size_t)b * 32);
             if (MATS == 2 && weigh) v = scaled(v, sx[q]);
 #pragma unroll
             for (int m = 0; m < MATS; ++m) {

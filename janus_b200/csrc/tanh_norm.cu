@@ -126,8 +126,9 @@ JB_EXPORT int jb_tanh_norm(float* stream, float* y, const float* wa, const float
                    aligned16(bb) && aligned16(x_out);
   const size_t n = (size_t)rows * W / (vec ? 4 : 1);
   JB_REFUSE(n >= 0x7fffffffull, "tanh_norm: %d rows of %d numbers are too many", rows, W);
-  const size_t want = (n + 255) / 256;
-  jb::Launch cfg(dim3((unsigned)(want < 148 * 16 ? want : 148 * 16)), dim3(256), 0, s);
+  const int threads = n <= 148 * 256 ? 64 : 256;      // few numbers: spread over the SMs
+  const size_t want = (n + threads - 1) / threads;
+  jb::Launch cfg(dim3((unsigned)(want < 148 * 16 ? want : 148 * 16)), dim3(threads), 0, s);
   const Squash na{wa, ba, alpha_a}, nb{wb, bb, alpha_b};
   cudaError_t e;
 #define JB_GO(TO, V)                                                                                             \

@@ -1646,7 +1646,7 @@ def experts_few_tokens_tc(h: torch.Tensor, sel_e: torch.Tensor, sel_w: torch.Ten
                           w_up: torch.Tensor, w_down: torch.Tensor, act: torch.Tensor, out: torch.Tensor,
                           gate_limit: float = 0.0, gate_alpha: float = 1.0, weight_on_output: bool = False) -> None:
     """`experts_few_tokens` for bfloat16 rows of whole 32-number blocks, on the tensor cores: an expert's rows are
-    streamed once for up to 32 of the tokens that chose it; act: bfloat16 scratch [T top, F]."""
+    streamed once for up to 16 of the tokens that chose it; act: bfloat16 scratch [T top, F]."""
     T, W = h.shape
     E, F, _ = w_gate.shape
     top = sel_e.shape[1]

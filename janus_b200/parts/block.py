@@ -238,8 +238,14 @@ class SandwichNormBlock:
             self.mixer.forward(x, y, ctx, cache_view, writes_cache)
         last = self._mixer_write
         if self.feed_forward is not None:
-            last.write_then_norm(residual, y, self.feed_forward_norm, x)
-            self.feed_forward.forward(x, y, ctx)
+            # so may a feed-forward
+            wants = getattr(self.feed_forward, "scratch_to_clear", None)
+            scratch = wants(ctx, T) if wants is not None else None
+            last.write_then_norm(residual, y, self.feed_forward_norm, x, clear=scratch)
+            if scratch is not None:
+                self.feed_forward.forward(x, y, ctx, scratch_cleared=True)
+            else:
+                self.feed_forward.forward(x, y, ctx)
             last = self._ff_write
         ctx.pending_write = (last, y)
 

@@ -112,9 +112,12 @@ class GeluFeedForward(FeedForward):
         self.up.load([up])
         self.down.load([down])
 
-    def forward(self, x: torch.Tensor, residual: torch.Tensor, ctx) -> None:
+    def scratch_to_clear(self, ctx, tokens: int):
+        return self.up.scratch_to_clear(ctx, tokens)
+
+    def forward(self, x: torch.Tensor, residual: torch.Tensor, ctx, scratch_cleared: bool = False) -> None:
         act = ctx.workspace.get("ffn_act", (x.shape[0], self.intermediate_size), self.dtype)
-        self.up.forward(x, act, ctx)
+        self.up.forward(x, act, ctx, scratch_cleared)
         self.down.forward_add(act, residual)
 
 

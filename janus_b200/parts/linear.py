@@ -140,11 +140,21 @@ class GeluLinear(Linear):
     """out = gelu(x W^T) in the engine dtype, gelu(z) = z (1 + erf(z / sqrt 2)) / 2: in the product's own epilogue, or,
     where a decode-sized step would leave SMs idle with K uncut (and in float32), behind a plain product."""
 
-    def forward(self, x: torch.Tensor, out: torch.Tensor, ctx) -> None:
+    def _behind(self, T: int) -> bool:
+        return T <= 64 and self.meets_by_adds(T, torch.float32)
+
+    def scratch_to_clear(self, ctx, tokens: int):
+        """The plain product's float32 result, if slices of K are added into it: the launch before may clear it."""
+        if not self._behind(tokens):
+            return None
+        z = ctx.workspace.get("gelu_in", (tokens, self.out_features), torch.float32)
+        return z if z.numel() % 4 == 0 else None
+
+    def forward(self, x: torch.Tensor, out: torch.Tensor, ctx, scratch_cleared: bool = False) -> None:
         T = x.shape[0]
-        if self.dtype == torch.float32 or self.meets_by_adds(T, torch.float32) and T <= 64:
+        if self.dtype == torch.float32 or self._behind(T):
             z = ctx.workspace.get("gelu_in", (T, self.out_features), torch.float32)
-            super().forward(x, z)
+            super().forward(x, z, y_is_zero=scratch_cleared)
             ops.gelu(z, out)
             return
         if self._padded is not None:

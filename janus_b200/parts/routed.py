@@ -6,7 +6,7 @@ largest scores (the lower index wins a tie) and their weights are those scores a
 weight multiplies the expert's INPUT: out = sum over the chosen e of expert_e(s_e h).
 
 Steps of few (token, expert) pairs, every single-token step among them, stream each chosen expert's rows once for
-up to 32 of the tokens that chose it (`ops.experts_few_tokens_tc`: two launches with a block per (rows, expert),
+up to 16 of the tokens that chose it (`ops.experts_few_tokens_tc`: two launches with a block per (rows, expert),
 float32 sums, nothing read back by the host, so the step can be recorded into a CUDA graph; widths that are no multiples
 of 32, and the float32 engine, take up to four tokens at a time on the CUDA cores, `ops.experts_few_tokens`).  Prompt steps of the
 bfloat16 engine with more pairs sort the (token, choice) pairs by expert, gather the weighted rows in that order and
@@ -134,11 +134,19 @@ class RoutedExperts(FeedForward):
                 self.gate_up.append(gu)
                 self.down.append(dn)
 
-    def forward(self, x: torch.Tensor, residual: torch.Tensor, ctx) -> None:
+    def scratch_to_clear(self, ctx, tokens: int) -> Optional[torch.Tensor]:
+        """The router's float32 logits, if this step's product adds slices of K into them: the launch before this part
+        may clear them in passing."""
+        if not self.router.meets_by_adds(tokens, torch.float32):
+            return None
+        buf = ctx.workspace.get("router_logits", (tokens, self.router.out_features), torch.float32)
+        return buf if buf.numel() % 4 == 0 else None
+
+    def forward(self, x: torch.Tensor, residual: torch.Tensor, ctx, scratch_cleared: bool = False) -> None:
         T = x.shape[0]
         ws = ctx.workspace
         logits = ws.get("router_logits", (T, self.router.out_features), torch.float32)
-        self.router.forward(x, logits)
+        self.router.forward(x, logits, y_is_zero=scratch_cleared)
         if self.shared_size is not None:
             shared = ws.get("shared_act", (T, self.shared_size), self.dtype)
             self.shared_gate_up.forward(x, shared, ctx)
