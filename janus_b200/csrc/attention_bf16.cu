@@ -1,6 +1,7 @@
 // bfloat16 grouped-query attention over the paged cache, compiled for one head
 // size (-DJB_HEAD_DIM=..., a multiple of 8 up to 256; in shared memory rows are
-// zero-padded to the next multiple of 16, the k extent of one MMA).
+// zero-padded to the next multiple of 16, the k extent of one MMA).  Values may
+// have a size of their own (-DJB_VALUE_DIM=..., default: the keys').
 //
 // Rows of a tile are (token, query head of one kv group) pairs, so the query
 // heads that share a kv head share every K/V tile that is read.  Scores and
@@ -15,7 +16,7 @@
 // Formulas: crates/janus-engine/src/compute/shaders/attention.wgsl:96-115,170-185 and
 // softmax.wgsl:29-50; kv head of query head h is floor(h * nkv / nh).
 //
-// Cache layout of one layer: [page][kv_head][64][HD]; block_table[seq][i] is the
+// Cache layout of one layer: [page][kv_head][64][HD] (values: VD); block_table[seq][i] is the
 // page of keys [64 i, 64 i + 64).
 #include <math_constants.h>
 #include <stdio.h>
@@ -25,26 +26,32 @@
 #ifndef JB_HEAD_DIM
 #define JB_HEAD_DIM 128
 #endif
+#ifndef JB_VALUE_DIM
+#define JB_VALUE_DIM JB_HEAD_DIM
+#endif
 
 namespace {
 
 typedef __nv_bfloat16 bf16;
 
 constexpr int HD = JB_HEAD_DIM;
+constexpr int VD = JB_VALUE_DIM;
 static_assert(HD % 8 == 0 && HD >= 8 && HD <= 256, "head size must be a multiple of 8 in [8, 256]");
+static_assert(VD % 8 == 0 && VD >= 8 && VD <= 256, "value size must be a multiple of 8 in [8, 256]");
 constexpr int HDP = (HD + 15) / 16 * 16;  // head size as the MMAs see it
 constexpr int PAGE = 64;
 constexpr int LD = HDP + 8;           // padded smem row: an odd number of 16-byte chunks, conflict-free ldmatrix
 constexpr int CHUNKS = HD / 8;        // 16-byte chunks per row that exist in global memory
+constexpr int VDP = (VD + 15) / 16 * 16, LDV = VDP + 8, V_CHUNKS = VD / 8;   // the same of the values
 constexpr int THREADS = 128;
-constexpr int KV_TILE = PAGE * LD;    // elements
+constexpr int K_TILE = PAGE * LD, V_TILE = PAGE * LDV, KV_STAGE = K_TILE + V_TILE;   // elements
 constexpr float LOG2E = 1.4426950408889634f;
 // K/V pages in the decode kernel's ring: picked at the launch from 2, 3 and 5 (`decode_stages_for`);
 // JB_DECODE_STAGES forces one depth.
 #ifndef JB_DECODE_STAGES
 #define JB_DECODE_STAGES 0
 #endif
-constexpr int RED_LD = HD + 8;                   // row stride (floats) of the warps' exchange of partial outputs
+constexpr int RED_LD = VD + 8;                   // row stride (floats) of the warps' exchange of partial outputs
 
 __device__ __forceinline__ uint32_t smem_u32(const void* p) { return (uint32_t)__cvta_generic_to_shared(p); }
 
@@ -98,20 +105,30 @@ __device__ __forceinline__ uint32_t pack_bf16(float lo, float hi) {
   return *reinterpret_cast<uint32_t*>(&v);
 }
 
-// Copy one [64, HD] page tile into padded shared memory (all 128 threads).
+// Copy one [64, SIZE] page tile into padded shared memory (all 128 threads).
+template <int SIZE, int ROW>
 __device__ __forceinline__ void load_page(bf16* dst, const bf16* src) {
-  for (int ch = threadIdx.x; ch < PAGE * CHUNKS; ch += THREADS) {
-    const int row = ch / CHUNKS, col = ch % CHUNKS;
-    cp_async16(dst + row * LD + col * 8, src + (size_t)row * HD + col * 8, true);
+  constexpr int N = SIZE / 8;
+  for (int ch = threadIdx.x; ch < PAGE * N; ch += THREADS) {
+    const int row = ch / N, col = ch % N;
+    cp_async16(dst + row * ROW + col * 8, src + (size_t)row * SIZE + col * 8, true);
   }
 }
 
-// The columns [HD, HDP) of `rows` padded rows are never written by a load: zero them once.
-__device__ __forceinline__ void zero_pad_columns(bf16* base, int rows) {
-  if constexpr (HDP != HD) {
-    constexpr int PAD = HDP - HD;
+// The columns behind the first SIZE of `rows` padded rows are never written by a load: zero them once.
+template <int SIZE, int SIZE_PADDED, int ROW>
+__device__ __forceinline__ void zero_columns(bf16* base, int rows) {
+  if constexpr (SIZE_PADDED != SIZE) {
+    constexpr int PAD = SIZE_PADDED - SIZE;
     for (int i = threadIdx.x; i < rows * PAD; i += THREADS)
-      base[(i / PAD) * LD + HD + i % PAD] = __float2bfloat16_rn(0.0f);
+      base[(i / PAD) * ROW + SIZE + i % PAD] = __float2bfloat16_rn(0.0f);
+  }
+}
+// ... of the stages of a ring of key and value tiles
+__device__ __forceinline__ void zero_ring_columns(bf16* kv_s, int stages) {
+  for (int st = 0; st < stages; ++st) {
+    zero_columns<HD, HDP, LD>(kv_s + (size_t)st * KV_STAGE, PAGE);
+    zero_columns<VD, VDP, LDV>(kv_s + (size_t)st * KV_STAGE + K_TILE, PAGE);
   }
 }
 
@@ -119,12 +136,12 @@ __device__ __forceinline__ void zero_pad_columns(bf16* base, int rows) {
 // owns rows g and g + 8.
 struct RowState {
   float m[2], l[2];
-  float o[HDP / 8][4];
+  float o[VDP / 8][4];
   __device__ __forceinline__ void init() {
     m[0] = m[1] = -CUDART_INF_F;
     l[0] = l[1] = 0.0f;
 #pragma unroll
-    for (int j = 0; j < HDP / 8; ++j) o[j][0] = o[j][1] = o[j][2] = o[j][3] = 0.0f;
+    for (int j = 0; j < VDP / 8; ++j) o[j][0] = o[j][1] = o[j][2] = o[j][3] = 0.0f;
   }
 };
 
@@ -154,20 +171,42 @@ __device__ __forceinline__ void qk_product(float (&s)[NT][4], const bf16* q_rows
 // chunk > 0: a query sees only the keys of its own chunk of positions, [floor(pos / chunk) chunk, pos];
 // cap_log2 > 0: scores are capped, s -> cap tanh(s scale / cap), with cap_log2 = cap log2(e), inv_cap = scale / cap.
 // sink = 1: the softmax's denominator has one more term, exp(0) (a key of score 0 that has no value).
+// slopes (one per query head, or null): slope (position - key position) is taken off the scaled score.
+// sinks (one per query head, or null): the denominator has one more term, exp(sinks[head]).
+// gate (float32 rows of ld_gate numbers, a row per token, a number per query head, or null): a head's output is multiplied
+// by the number's sigmoid.
 struct Cap {
   int chunk;
   float cap_log2;
   float inv_cap;
   float sink;
+  const float* slopes;
+  const float* sinks;
+  const float* gate;
+  int ld_gate;
 };
+// A denominator l relative to the maximum m (in units of log2), with what a sink adds to it.
+__device__ __forceinline__ float with_sink(float l, float m, const Cap& cap, int head) {
+  const float ref = m == -CUDART_INF_F ? 0.0f : m;
+  if (cap.sink > 0.0f) l += cap.sink * exp2f(-ref);
+  if (cap.sinks != nullptr) l += exp2f(cap.sinks[head] * LOG2E - ref);
+  return l;
+}
+__device__ __forceinline__ float head_gate(const Cap& cap, int token, int head) {
+  return cap.gate == nullptr ? 1.0f : 1.0f / (1.0f + expf(-cap.gate[(size_t)token * cap.ld_gate + head]));
+}
+// The slope of a head's distance bias in units of log2(e) (0: none).
+__device__ __forceinline__ float head_slope(const Cap& cap, int head) {
+  return cap.slopes == nullptr ? 0.0f : cap.slopes[head] * LOG2E;
+}
 __device__ __forceinline__ int chunk_lo(int lo, int pos, int chunk) {
   return (chunk > 0 && pos >= 0) ? max(lo, (pos / chunk) * chunk) : lo;
 }
 
 template <int NT>
 __device__ __forceinline__ void softmax_pv(RowState& st, float (&s)[NT][4], const bf16* v_tile, int key_pos0,
-                                           const int (&row_pos)[2], const int (&row_lo)[2], float scale_log2,
-                                           const Cap& cap, int lane) {
+                                           const int (&row_pos)[2], const int (&row_lo)[2], const float (&slope)[2],
+                                           float scale_log2, const Cap& cap, int lane) {
   const int c = lane & 3;
   float mx[2] = {-CUDART_INF_F, -CUDART_INF_F};
 #pragma unroll
@@ -178,7 +217,8 @@ __device__ __forceinline__ void softmax_pv(RowState& st, float (&s)[NT][4], cons
       const int kp = key_pos0 + j * 8 + 2 * c + (e & 1);
       const bool ok = kp <= row_pos[r] && kp >= row_lo[r];
       // with a cap c the score s becomes c tanh(s / c), here in units of log2(e)
-      const float sc = cap.cap_log2 > 0.0f ? cap.cap_log2 * tanhf(s[j][e] * cap.inv_cap) : s[j][e] * scale_log2;
+      float sc = cap.cap_log2 > 0.0f ? cap.cap_log2 * tanhf(s[j][e] * cap.inv_cap) : s[j][e] * scale_log2;
+      if (cap.slopes != nullptr) sc = fmaf(slope[r], (float)(kp - row_pos[r]), sc);
       s[j][e] = ok ? sc : -CUDART_INF_F;
       mx[r] = fmaxf(mx[r], s[j][e]);
     }
@@ -195,7 +235,7 @@ __device__ __forceinline__ void softmax_pv(RowState& st, float (&s)[NT][4], cons
     st.l[r] *= corr[r];
   }
 #pragma unroll
-  for (int j = 0; j < HDP / 8; ++j) {
+  for (int j = 0; j < VDP / 8; ++j) {
     st.o[j][0] *= corr[0];
     st.o[j][1] *= corr[0];
     st.o[j][2] *= corr[1];
@@ -218,9 +258,9 @@ __device__ __forceinline__ void softmax_pv(RowState& st, float (&s)[NT][4], cons
     a[2] = pack_bf16(s[2 * kk + 1][0], s[2 * kk + 1][1]);
     a[3] = pack_bf16(s[2 * kk + 1][2], s[2 * kk + 1][3]);
 #pragma unroll
-    for (int j = 0; j < HDP / 8; j += 2) {
+    for (int j = 0; j < VDP / 8; j += 2) {
       uint32_t b[4];
-      ldmatrix_x4_trans(b, v_tile + (kk * 16 + (lane & 15)) * LD + j * 8 + (lane >> 4) * 8);
+      ldmatrix_x4_trans(b, v_tile + (kk * 16 + (lane & 15)) * LDV + j * 8 + (lane >> 4) * 8);
       mma_bf16(st.o[j], a, b[0], b[1]);
       mma_bf16(st.o[j + 1], a, b[2], b[3]);
     }
@@ -236,7 +276,7 @@ __global__ void __launch_bounds__(THREADS) prefill_kernel(
   jb::pdl_launch_dependents();
   jb::pdl_wait();
   bf16* q_s = reinterpret_cast<bf16*>(smem_raw);  // [64][LD]
-  bf16* kv_s = q_s + 64 * LD;                     // [2 stages][K, V][64][LD]
+  bf16* kv_s = q_s + 64 * LD;                     // [2 stages][K [64][LD], V [64][LDV]]
   const int G = nh / nkv;
   const int tpt = 64 / G;                         // tokens per tile
   // kv heads run fastest in the order CTAs are handed out and tiles go backwards: across all heads the
@@ -251,7 +291,8 @@ __global__ void __launch_bounds__(THREADS) prefill_kernel(
   const int* pages = block_table + (size_t)seq * max_pages;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
 
-  zero_pad_columns(q_s, 64 + 4 * PAGE);  // q tile and the four K/V tiles lie back to back
+  zero_columns<HD, HDP, LD>(q_s, 64);
+  zero_ring_columns(kv_s, 2);
   // Q rows: r -> (token tok0 + r / G, head kvh * G + r % G)
   for (int ch = threadIdx.x; ch < 64 * CHUNKS; ch += THREADS) {
     const int r = ch / CHUNKS, col = ch % CHUNKS;
@@ -265,17 +306,19 @@ __global__ void __launch_bounds__(THREADS) prefill_kernel(
   const int kb_start = chunk_lo(window > 0 ? max(0, pos0 - window + 1) : 0, pos0, cap.chunk) / PAGE;
   auto issue = [&](int kb, int stage) {
     const size_t page = (size_t)pages[kb];
-    const size_t off = (page * nkv + kvh) * PAGE * HD;
-    load_page(kv_s + (size_t)stage * 2 * KV_TILE, k_cache + off);
-    load_page(kv_s + (size_t)stage * 2 * KV_TILE + KV_TILE, v_cache + off);
+    const size_t rows = (page * nkv + kvh) * PAGE;
+    load_page<HD, LD>(kv_s + (size_t)stage * KV_STAGE, k_cache + rows * HD);
+    load_page<VD, LDV>(kv_s + (size_t)stage * KV_STAGE + K_TILE, v_cache + rows * VD);
   };
   issue(kb_start, 0);
   cp_async_commit();
 
   int row_pos[2], row_lo[2];
+  float slope[2];
 #pragma unroll
   for (int r = 0; r < 2; ++r) {
     const int row = warp * 16 + (lane >> 2) + 8 * r;
+    slope[r] = head_slope(cap, kvh * G + row % G);
     const int tl = row / G;
     row_pos[r] = tl < n_tok ? pos0 + tl : -1;
     row_lo[r] = chunk_lo(window > 0 ? max(0, row_pos[r] - window + 1) : 0, row_pos[r], cap.chunk);
@@ -292,10 +335,10 @@ __global__ void __launch_bounds__(THREADS) prefill_kernel(
       cp_async_wait<0>();
     }
     __syncthreads();
-    const bf16* k_tile = kv_s + (size_t)stage * 2 * KV_TILE;
+    const bf16* k_tile = kv_s + (size_t)stage * KV_STAGE;
     float s[8][4];
     qk_product<8>(s, q_s + warp * 16 * LD, k_tile, lane);
-    softmax_pv<8>(st, s, k_tile + KV_TILE, kb * PAGE, row_pos, row_lo, scale_log2, cap, lane);
+    softmax_pv<8>(st, s, k_tile + K_TILE, kb * PAGE, row_pos, row_lo, slope, scale_log2, cap, lane);
     __syncthreads();
   }
 #pragma unroll
@@ -306,12 +349,12 @@ __global__ void __launch_bounds__(THREADS) prefill_kernel(
     const int row = warp * 16 + (lane >> 2) + 8 * r;
     const int tl = row / G;
     if (tl < n_tok) {
-      if (cap.sink > 0.0f) l += cap.sink * exp2f(st.m[r] == -CUDART_INF_F ? 0.0f : -st.m[r]);
-      const float inv = 1.0f / l;
-      bf16* o = out + ((size_t)(qs + tok0 + tl) * nh + kvh * G + row % G) * HD + 2 * (lane & 3);
+      const int head = kvh * G + row % G, token = qs + tok0 + tl;
+      const float inv = head_gate(cap, token, head) / with_sink(l, st.m[r], cap, head);
+      bf16* o = out + ((size_t)token * nh + head) * VD + 2 * (lane & 3);
 #pragma unroll
-      for (int j = 0; j < HDP / 8; ++j)
-        if (j * 8 < HD)
+      for (int j = 0; j < VDP / 8; ++j)
+        if (j * 8 < VD)
           *reinterpret_cast<uint32_t*>(o + j * 8) = pack_bf16(st.o[j][2 * r] * inv, st.o[j][2 * r + 1] * inv);
     }
   }
@@ -321,7 +364,8 @@ __global__ void __launch_bounds__(THREADS) prefill_kernel(
 // Optional fused input of the decode kernel: instead of rotated bf16 queries and a cache that
 // already holds the new token, the q/k/v projection's float32 output [seq][q heads | k heads | v heads];
 // the kernel rotates q and k at the token's position (cos_sin null = no rotation), appends k and v
-// to the cache (write_kv) and uses them.  qkv == nullptr turns this off.
+// to the cache (write_kv) and uses them.  qkv == nullptr turns this off.  With `first` (rows of first_stride numbers, the
+// kv heads' values of the same tokens in another layer) the value is (1 - mix) v + mix first.
 struct FusedInput {
   const float* qkv;
   int qkv_stride;
@@ -330,6 +374,9 @@ struct FusedInput {
   bf16* k_out;
   bf16* v_out;
   int write_kv;
+  const float* first;
+  int first_stride;
+  float mix;
 };
 
 __device__ __forceinline__ void rotate_pair(float x0, float x1, const float* cs, int i, float& y0, float& y1) {
@@ -343,7 +390,7 @@ __device__ __forceinline__ void rotate_pair(float x0, float x1, const float* cs,
   y1 = x0 * s + x1 * c;
 }
 
-// part_o: [seq][head][split][HD] float32 (unnormalised), part_ml: [seq][head][split][2] (max, sum).
+// part_o: [seq][head][split][VD] float32 (unnormalised), part_ml: [seq][head][split][2] (max, sum).
 template <int DECODE_STAGES>
 __global__ void __launch_bounds__(THREADS) decode_kernel(
     const bf16* __restrict__ q, const bf16* __restrict__ k_cache, const bf16* __restrict__ v_cache,
@@ -353,8 +400,8 @@ __global__ void __launch_bounds__(THREADS) decode_kernel(
   extern __shared__ __align__(16) uint8_t smem_raw[];
   jb::pdl_launch_dependents();
   bf16* q_s = reinterpret_cast<bf16*>(smem_raw);  // [16][LD]
-  bf16* new_kv = q_s + 16 * LD;                   // [2][LD]: the new token's rotated key and its value (fused input)
-  bf16* kv_s = new_kv + 2 * LD;                   // [DECODE_STAGES][K, V][64][LD]; reused as float scratch at the end
+  bf16* new_kv = q_s + 16 * LD;                   // [LD], [LDV]: the new token's rotated key and its value (fused input)
+  bf16* kv_s = new_kv + LD + LDV;                 // [DECODE_STAGES][K [64][LD], V [64][LDV]]; float scratch at the end
   const int G = nh / nkv;
   const int n_rb = (G + 15) / 16;
   const int seq = blockIdx.x, kvh = blockIdx.y / n_rb, rb = blockIdx.y % n_rb, split = blockIdx.z;
@@ -385,12 +432,19 @@ __global__ void __launch_bounds__(THREADS) decode_kernel(
   const uint64_t kv_pol = kv_policy();
   auto issue = [&](int kb, int stage) {
     const size_t page = (size_t)pages[kb];
-    const size_t off = ((page * nkv + kvh) * PAGE + warp * 16) * HD;
-    bf16* k_rows = kv_s + (size_t)stage * 2 * KV_TILE + warp * 16 * LD;
+    const size_t row0 = (page * nkv + kvh) * PAGE + warp * 16;
+    bf16* k_rows = kv_s + (size_t)stage * KV_STAGE + warp * 16 * LD;
+    bf16* v_rows = kv_s + (size_t)stage * KV_STAGE + K_TILE + warp * 16 * LDV;
     for (int ch = lane; ch < 16 * CHUNKS; ch += 32) {
       const int row = ch / CHUNKS, col = ch % CHUNKS;
-      cp_async16_kv(k_rows + row * LD + col * 8, k_cache + off + (size_t)row * HD + col * 8, kv_pol);
-      cp_async16_kv(k_rows + KV_TILE + row * LD + col * 8, v_cache + off + (size_t)row * HD + col * 8, kv_pol);
+      cp_async16_kv(k_rows + row * LD + col * 8, k_cache + (row0 + row) * HD + col * 8, kv_pol);
+      if constexpr (VD == HD) cp_async16_kv(v_rows + row * LDV + col * 8, v_cache + (row0 + row) * VD + col * 8, kv_pol);
+    }
+    if constexpr (VD != HD) {
+      for (int ch = lane; ch < 16 * V_CHUNKS; ch += 32) {
+        const int row = ch / V_CHUNKS, col = ch % V_CHUNKS;
+        cp_async16_kv(v_rows + row * LDV + col * 8, v_cache + (row0 + row) * VD + col * 8, kv_pol);
+      }
     }
   };
   // ring of DECODE_STAGES pages: DECODE_STAGES - 1 loads are in flight while one page is computed
@@ -404,7 +458,8 @@ __global__ void __launch_bounds__(THREADS) decode_kernel(
   if (kb_start <= kb_end && early) issue_first_pages();
   jb::pdl_wait();
   if (kb_start <= kb_end) {
-    zero_pad_columns(q_s, 16 + 2 + 2 * DECODE_STAGES * PAGE);
+    zero_columns<HD, HDP, LD>(q_s, 16);
+    zero_ring_columns(kv_s, DECODE_STAGES);
     const bool patch_new = appends_here && kb_end == kb_last;  // this CTA sees the new key
     if (!early) issue_first_pages();
     if (fused.qkv == nullptr) {
@@ -434,28 +489,36 @@ __global__ void __launch_bounds__(THREADS) decode_kernel(
         q_s[(idx / HD) * LD + idx % HD] = __float2bfloat16_rn(0.0f);
       if (patch_new) {
         const float* kx = row + (size_t)(nh + kvh) * HD;
-        const float* vx = row + (size_t)(nh + nkv + kvh) * HD;
+        const float* vx = row + (size_t)(nh + nkv) * HD + (size_t)kvh * VD;
+        const float* v1st = fused.first != nullptr ? fused.first + (size_t)seq * fused.first_stride + (size_t)kvh * VD : nullptr;
         const int dst = fused.dest[seq];
-        const size_t g_off = (((size_t)(dst / PAGE) * nkv + kvh) * PAGE + dst % PAGE) * HD;
+        const size_t g_row = ((size_t)(dst / PAGE) * nkv + kvh) * PAGE + dst % PAGE;
+        bf16* k_out = fused.k_out + g_row * HD;
+        bf16* v_out = fused.v_out + g_row * VD;
         for (int i = threadIdx.x; i < HALF; i += THREADS) {
           float y0, y1;
           rotate_pair(kx[i], kx[i + HALF], cs, i, y0, y1);
           const bf16 k0 = __float2bfloat16_rn(y0), k1 = __float2bfloat16_rn(y1);
-          const bf16 v0 = __float2bfloat16_rn(vx[i]), v1 = __float2bfloat16_rn(vx[i + HALF]);
           new_kv[i] = k0; new_kv[i + HALF] = k1;
-          new_kv[LD + i] = v0; new_kv[LD + i + HALF] = v1;
           if (rb == 0) {  // one CTA per (sequence, kv head) appends to the cache for the steps to come
-            fused.k_out[g_off + i] = k0; fused.k_out[g_off + i + HALF] = k1;
-            fused.v_out[g_off + i] = v0; fused.v_out[g_off + i + HALF] = v1;
+            k_out[i] = k0; k_out[i + HALF] = k1;
           }
+        }
+        for (int i = threadIdx.x; i < VD; i += THREADS) {
+          const bf16 v = __float2bfloat16_rn(v1st != nullptr ? (1.0f - fused.mix) * vx[i] + fused.mix * v1st[i] : vx[i]);
+          new_kv[LD + i] = v;
+          if (rb == 0) v_out[i] = v;
         }
       }
     }
     int row_pos[2], row_lo[2];
+    float slope[2];
 #pragma unroll
     for (int r = 0; r < 2; ++r) {
-      row_pos[r] = ((lane >> 2) + 8 * r) < n_rows ? pos : -1;
+      const int head_row = (lane >> 2) + 8 * r;
+      row_pos[r] = head_row < n_rows ? pos : -1;
       row_lo[r] = lo;
+      slope[r] = head_slope(cap, kvh * G + g0 + min(head_row, n_rows - 1));
     }
     __syncthreads();  // q (and the new key and value) are in shared memory for every warp
     for (int kb = kb_start; kb <= kb_end; ++kb) {
@@ -465,21 +528,19 @@ __global__ void __launch_bounds__(THREADS) decode_kernel(
       cp_async_commit();
       cp_async_wait<DECODE_STAGES - 1>();  // everything but the newest DECODE_STAGES - 1 groups: page kb has landed
       __syncwarp();
-      bf16* k_tile = kv_s + (size_t)stage * 2 * KV_TILE;
+      bf16* k_tile = kv_s + (size_t)stage * KV_STAGE;
       if (patch_new && kb == kb_last && warp == (pos % PAGE) / 16) {
         // the page as loaded holds a stale row at the new position: the warp that owns the row puts the
         // new key and value there
         const int r = pos % PAGE;
-        for (int i = lane; i < 2 * HD; i += 32) {
-          const int which = i / HD, d = i % HD;
-          k_tile[which * KV_TILE + r * LD + d] = new_kv[which * LD + d];
-        }
+        for (int i = lane; i < HD; i += 32) k_tile[r * LD + i] = new_kv[i];
+        for (int i = lane; i < VD; i += 32) k_tile[K_TILE + r * LDV + i] = new_kv[LD + i];
         __syncwarp();
       }
       // this warp's 16 keys of the page
       float s[2][4];
       qk_product<2>(s, q_s, k_tile + warp * 16 * LD, lane);
-      softmax_pv<2>(st, s, k_tile + KV_TILE + warp * 16 * LD, kb * PAGE + warp * 16, row_pos, row_lo,
+      softmax_pv<2>(st, s, k_tile + K_TILE + warp * 16 * LDV, kb * PAGE + warp * 16, row_pos, row_lo, slope,
                     scale_log2, cap, lane);
       __syncwarp();  // the warp is done with its rows of this stage before its next loads overwrite them
     }
@@ -499,8 +560,8 @@ __global__ void __launch_bounds__(THREADS) decode_kernel(
       red_ml[(warp * 16 + row) * 2 + 1] = l;
     }
 #pragma unroll
-    for (int j = 0; j < HDP / 8; ++j) {
-      if (j * 8 < HD) {
+    for (int j = 0; j < VDP / 8; ++j) {
+      if (j * 8 < VD) {
         float* o = red_o + ((size_t)(warp * 16 + row)) * RED_LD + j * 8 + 2 * (lane & 3);
         o[0] = st.o[j][2 * r];
         o[1] = st.o[j][2 * r + 1];
@@ -508,8 +569,8 @@ __global__ void __launch_bounds__(THREADS) decode_kernel(
     }
   }
   __syncthreads();
-  for (int idx = threadIdx.x; idx < n_rows * HD; idx += THREADS) {
-    const int row = idx / HD, d = idx % HD;
+  for (int idx = threadIdx.x; idx < n_rows * VD; idx += THREADS) {
+    const int row = idx / VD, d = idx % VD;
     float m = -CUDART_INF_F;
 #pragma unroll
     for (int w = 0; w < 4; ++w) m = fmaxf(m, red_ml[(w * 16 + row) * 2]);
@@ -523,11 +584,10 @@ __global__ void __launch_bounds__(THREADS) decode_kernel(
     }
     const int head = kvh * G + g0 + row;
     if (n_splits == 1) {
-      if (cap.sink > 0.0f) l += cap.sink * exp2f(-m_use);
-      out[((size_t)seq * nh + head) * HD + d] = __float2bfloat16_rn(o / l);
+      out[((size_t)seq * nh + head) * VD + d] = __float2bfloat16_rn(o / with_sink(l, m, cap, head) * head_gate(cap, seq, head));
     } else {
       const size_t base = ((size_t)seq * nh + head) * n_splits + split;
-      part_o[base * HD + d] = o;
+      part_o[base * VD + d] = o;
       if (d == 0) {
         part_ml[base * 2] = m;
         part_ml[base * 2 + 1] = l;
@@ -537,30 +597,31 @@ __global__ void __launch_bounds__(THREADS) decode_kernel(
 }
 
 __global__ void decode_combine_kernel(const float* __restrict__ part_o, const float* __restrict__ part_ml,
-                                      bf16* __restrict__ out, int n_splits, float sink) {
+                                      bf16* __restrict__ out, int n_splits, int nh, Cap cap) {
   jb::pdl_launch_dependents();
   jb::pdl_wait();
   const size_t item = blockIdx.x;  // seq * nh + head
+  const int head = (int)(item % nh);
   const float* ml = part_ml + item * n_splits * 2;
   float m = -CUDART_INF_F;
   for (int s = 0; s < n_splits; ++s) m = fmaxf(m, ml[2 * s]);
-  for (int d = threadIdx.x; d < HD; d += blockDim.x) {
+  const float open = head_gate(cap, (int)(item / nh), head);
+  for (int d = threadIdx.x; d < VD; d += blockDim.x) {
     float o = 0.0f, l = 0.0f;
     for (int s = 0; s < n_splits; ++s) {
       const float f = exp2f(ml[2 * s] - m);  // a split without keys has max -inf and weighs 0
-      o += part_o[(item * n_splits + s) * HD + d] * f;
+      o += part_o[(item * n_splits + s) * VD + d] * f;
       l += ml[2 * s + 1] * f;
     }
-    if (sink > 0.0f) l += sink * exp2f(m == -CUDART_INF_F ? 0.0f : -m);
-    out[item * HD + d] = __float2bfloat16_rn(o / l);
+    out[item * VD + d] = __float2bfloat16_rn(o / with_sink(l, m, cap, head) * open);
   }
 }
 
-constexpr int PREFILL_SMEM = (64 * LD + 4 * KV_TILE) * 2;
+constexpr int PREFILL_SMEM = (64 * LD + 2 * KV_STAGE) * 2;
 constexpr int DECODE_RED_BYTES = (4 * 16 * RED_LD + 4 * 16 * 2) * 4;
 constexpr int decode_smem(int stages) {
-  const int kv = 2 * stages * KV_TILE * 2;
-  return (16 + 2) * LD * 2 + (kv > DECODE_RED_BYTES ? kv : DECODE_RED_BYTES);
+  const int kv = stages * KV_STAGE * 2;
+  return (17 * LD + LDV) * 2 + (kv > DECODE_RED_BYTES ? kv : DECODE_RED_BYTES);
 }
 constexpr int SMEM_PER_SM = 228 * 1024;   // of which every resident CTA takes 1 KB for the system besides its own
 constexpr int ctas_per_sm(int stages) { return SMEM_PER_SM / (decode_smem(stages) + 1024); }
@@ -608,7 +669,7 @@ cudaError_t decode_go(dim3 grid, cudaStream_t stream, bool pdl, const bf16* q, c
 cudaError_t decode_dispatch(dim3 grid, cudaStream_t stream, bool pdl, const bf16* q, const bf16* k_cache,
                             const bf16* v_cache, bf16* out, float* part_o, float* part_ml, const int* block_table,
                             const int* kv_len, int nh, int nkv, int max_pages, int window, float scale_log2,
-                            int n_splits, const FusedInput& fused, const Cap& cap = Cap{0, 0.0f, 0.0f}) {
+                            int n_splits, const FusedInput& fused, const Cap& cap = Cap{}) {
   const long long ctas = (long long)grid.x * grid.y * grid.z;
   const int stages = decode_stages_for(ctas, max(1, max_pages / max(1, n_splits)));
 #define JB_DECODE_GO(ST)                                                                                      \
@@ -630,8 +691,10 @@ cudaError_t decode_dispatch(dim3 grid, cudaStream_t stream, bool pdl, const bf16
 JB_EXPORT int jb_attention_bf16_head_dim() { return HD; }
 
 namespace {
-Cap make_cap(int chunk, float softcap, float scale, float sink) {
-  return softcap > 0.0f ? Cap{chunk, softcap * LOG2E, scale / softcap, sink} : Cap{chunk, 0.0f, 0.0f, sink};
+Cap make_cap(int chunk, float softcap, float scale, float sink, const float* slopes, const float* sinks, const float* gate,
+             int ld_gate) {
+  const bool capped = softcap > 0.0f;
+  return Cap{chunk, capped ? softcap * LOG2E : 0.0f, capped ? scale / softcap : 0.0f, sink, slopes, sinks, gate, ld_gate};
 }
 
 int prefill_launch(const void* q, const void* k_cache, const void* v_cache, void* out,
@@ -664,28 +727,32 @@ JB_EXPORT int jb_attention_bf16_prefill(const void* q, const void* k_cache, cons
                                         int n_seqs, int max_q_len, int nh, int nkv, int hd, int page_size,
                                         int max_pages, int window, float scale, cudaStream_t stream) {
   return prefill_launch(q, k_cache, v_cache, out, block_table, q_start, kv_len, n_seqs, max_q_len, nh, nkv, hd,
-                        page_size, max_pages, window, scale, Cap{0, 0.0f, 0.0f}, stream);
+                        page_size, max_pages, window, scale, Cap{}, stream);
 }
 
 // As jb_attention_bf16_prefill, with a chunked mask (chunk > 0: a query sees only the keys of its own chunk of
-// positions), capped scores (softcap > 0: s -> softcap tanh(s / softcap)) and a sink (sink = 1: one more term exp(0)
-// in the softmax's denominator).
+// positions), capped scores (softcap > 0: s -> softcap tanh(s / softcap)), a sink (sink = 1: one more term exp(0)
+// in the softmax's denominator; sinks [nh]: one more term exp(sinks[head])), a distance bias (slopes [nh]:
+// slopes[head] (position - key position) is taken off) and an output gate (gate: float32 rows of ld_gate numbers, a row a
+// token, column `head` for each head; its sigmoid multiplies the head's output).  slopes, sinks, gate: device memory or null.
 JB_EXPORT int jb_attention_bf16_prefill_capped(const void* q, const void* k_cache, const void* v_cache, void* out,
                                                const int* block_table, const int* q_start, const int* kv_len,
                                                int n_seqs, int max_q_len, int nh, int nkv, int hd, int page_size,
                                                int max_pages, int window, float scale, int chunk, float softcap,
-                                               float sink, cudaStream_t stream) {
+                                               float sink, const float* slopes, const float* sinks, const float* gate,
+                                               int ld_gate, cudaStream_t stream) {
   return prefill_launch(q, k_cache, v_cache, out, block_table, q_start, kv_len, n_seqs, max_q_len, nh, nkv, hd,
-                        page_size, max_pages, window, scale, make_cap(chunk, softcap, scale, sink), stream);
+                        page_size, max_pages, window, scale,
+                        make_cap(chunk, softcap, scale, sink, slopes, sinks, gate, ld_gate), stream);
 }
 
-// Scratch (when n_splits > 1): part_o float32 [n_seqs * nh * n_splits * hd], part_ml float32
+// Scratch (when n_splits > 1): part_o float32 [n_seqs * nh * n_splits * VD], part_ml float32
 // [n_seqs * nh * n_splits * 2].
 namespace {
 int decode_launch(const void* q, const void* k_cache, const void* v_cache, void* out, float* part_o, float* part_ml,
                   const int* block_table, const int* kv_len, int n_seqs, int nh, int nkv, int hd, int page_size,
                   int max_pages, int window, float scale, int n_splits, const FusedInput& fused,
-                  cudaStream_t stream, const Cap& cap = Cap{0, 0.0f, 0.0f}) {
+                  cudaStream_t stream, const Cap& cap = Cap{}) {
   if (n_seqs <= 0) return 0;
   JB_REFUSE(hd != HD, "attention_bf16: built for head_dim %d, called with %d", HD, hd);
   JB_REFUSE(page_size != PAGE, "attention_bf16: page size %d (need %d)", page_size, PAGE);
@@ -699,9 +766,9 @@ int decode_launch(const void* q, const void* k_cache, const void* v_cache, void*
                                    scale * LOG2E, n_splits, fused, cap);
   if (le != cudaSuccess) return (int)le;
   if (n_splits > 1) {
-    jb::Launch cfg2(dim3(n_seqs * nh), dim3(HD >= 128 ? 128 : 64), 0, stream);
+    jb::Launch cfg2(dim3(n_seqs * nh), dim3(VD >= 128 ? 128 : 64), 0, stream);
     le = cudaLaunchKernelEx(&cfg2.c, decode_combine_kernel, (const float*)part_o, (const float*)part_ml, (bf16*)out,
-                            n_splits, cap.sink);
+                            n_splits, nh, cap);
     if (le != cudaSuccess) return (int)le;
   }
   return 0;
@@ -717,32 +784,38 @@ JB_EXPORT int jb_attention_bf16_decode(const void* q, const void* k_cache, const
                        page_size, max_pages, window, scale, n_splits, FusedInput{}, stream);
 }
 
-// As jb_attention_bf16_decode, with a chunked mask and capped scores (see jb_attention_bf16_prefill_capped).
+// As jb_attention_bf16_decode, with the options of jb_attention_bf16_prefill_capped (gate: a row per sequence).
 JB_EXPORT int jb_attention_bf16_decode_capped(const void* q, const void* k_cache, const void* v_cache, void* out,
                                               float* part_o, float* part_ml, const int* block_table,
                                               const int* kv_len, int n_seqs, int nh, int nkv, int hd, int page_size,
                                               int max_pages, int window, float scale, int n_splits, int chunk,
-                                              float softcap, float sink, cudaStream_t stream) {
+                                              float softcap, float sink, const float* slopes, const float* sinks,
+                                              const float* gate, int ld_gate, cudaStream_t stream) {
   return decode_launch(q, k_cache, v_cache, out, part_o, part_ml, block_table, kv_len, n_seqs, nh, nkv, hd,
                        page_size, max_pages, window, scale, n_splits, FusedInput{}, stream,
-                       make_cap(chunk, softcap, scale, sink));
+                       make_cap(chunk, softcap, scale, sink, slopes, sinks, gate, ld_gate));
 }
 
 // As jb_attention_bf16_decode, but q, k and v of the new tokens come as the projection's float32
 // output qkv[seq][q heads | k heads | v heads] (row stride qkv_stride floats): the kernel rotates q
 // and k with cos_sin[position] (null = no rotation), appends k and v at cache row dest[seq]
-// (write_kv = 0: a layer that reads another layer's cache; only q is used) and attends.
+// (write_kv = 0: a layer that reads another layer's cache; only q is used) and attends.  Value heads hold VD numbers.
+// first (or null): float32 rows of first_stride numbers, [kv heads][VD] of each new token; the value that is used and
+// appended is (1 - mix) v + mix first.  The other options: as jb_attention_bf16_decode_capped.
 JB_EXPORT int jb_attention_bf16_decode_fused(const float* qkv, int qkv_stride, const float* cos_sin,
                                              const int* dest, void* k_cache, void* v_cache, void* out,
                                              float* part_o, float* part_ml, const int* block_table,
                                              const int* kv_len, int n_seqs, int nh, int nkv, int hd,
                                              int page_size, int max_pages, int window, float scale,
-                                             int n_splits, int write_kv, cudaStream_t stream) {
+                                             int n_splits, int write_kv, int chunk, float softcap, float sink,
+                                             const float* slopes, const float* sinks, const float* gate, int ld_gate,
+                                             const float* first, int first_stride, float mix, cudaStream_t stream) {
   JB_REFUSE(qkv == nullptr || (write_kv && dest == nullptr), "attention_bf16 fused decode: missing input");
   JB_REFUSE(hd % 2 != 0, "attention_bf16 fused decode: head_dim %d must be even for the rotation", hd);
-  FusedInput fused{qkv, qkv_stride, cos_sin, dest, (bf16*)k_cache, (bf16*)v_cache, write_kv};
+  FusedInput fused{qkv, qkv_stride, cos_sin, dest, (bf16*)k_cache, (bf16*)v_cache, write_kv, first, first_stride, mix};
   return decode_launch(nullptr, k_cache, v_cache, out, part_o, part_ml, block_table, kv_len, n_seqs, nh, nkv, hd,
-                       page_size, max_pages, window, scale, n_splits, fused, stream);
+                       page_size, max_pages, window, scale, n_splits, fused, stream,
+                       make_cap(chunk, softcap, scale, sink, slopes, sinks, gate, ld_gate));
 }
 
 // ---------------------------------------------------------------------------
@@ -775,7 +848,7 @@ JB_EXPORT int jb_attention_bf16_decode_noalloc(const void* q, const void* k_cach
   JB_REFUSE(nkv <= 0 || nh % nkv != 0, "attention_bf16: %d heads are not a multiple of %d kv heads", nh, nkv);
   JB_REFUSE(n_splits < 1, "attention_bf16 decode: n_splits must be at least 1, got %d", n_splits);
   // one split writes straight to `out`: no scratch is touched, whatever the batch
-  const size_t o_floats = n_splits > 1 ? (size_t)n_seqs * nh * n_splits * HD : 0;
+  const size_t o_floats = n_splits > 1 ? (size_t)n_seqs * nh * n_splits * VD : 0;
   const size_t ml_floats = n_splits > 1 ? (size_t)n_seqs * nh * n_splits * 2 : 0;
   JB_REFUSE(o_floats + ml_floats > JB_NOALLOC_SCRATCH_FLOATS,
             "attention_bf16 decode without allocation: %zu scratch floats are needed (n_seqs %d x heads %d x "
@@ -806,7 +879,7 @@ JB_EXPORT int jb_attention_bf16_decode_noalloc(const void* q, const void* k_cach
                       FusedInput{});
   if (e != cudaSuccess) return (int)e;
   if (n_splits > 1) {
-    decode_combine_kernel<<<n_seqs * nh, HD >= 128 ? 128 : 64, 0, stream>>>(part_o, part_ml, (bf16*)out, n_splits, 0.0f);
+    decode_combine_kernel<<<n_seqs * nh, VD >= 128 ? 128 : 64, 0, stream>>>(part_o, part_ml, (bf16*)out, n_splits, nh, Cap{});
     JB_CHECK_LAUNCH();
   }
   return 0;

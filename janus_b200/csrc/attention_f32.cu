@@ -10,7 +10,10 @@
 // 32 keys that start at multiples of 32 of the absolute key index, so a
 // token's result does not depend on how its sequence was cut into steps.
 //
-// The values may be the first `vd` numbers of rows of hd numbers (latent attention: a row is key and value at once).
+// The values are the first `vd` numbers of rows of ld_v numbers (latent attention: a row is key and value at once).
+// slopes (one per query head): slope (position - key position) is taken off the score; sinks (one per query head): the
+// denominator has one more term, exp(sink); gate (rows of ld_gate numbers, one a query head): its sigmoid multiplies the
+// head's output.
 //
 // Cache layout of one layer: [page][kv_head][PAGE][hd]; block_table[slot][i] is
 // the page of keys [i*PAGE, (i+1)*PAGE) of the sequence in `slot`.
@@ -31,7 +34,8 @@ __global__ void __launch_bounds__(WARPS * 32) attention_f32_kernel(
     const float* __restrict__ q, const float* __restrict__ k_cache, const float* __restrict__ v_cache,
     float* __restrict__ out, const int* __restrict__ block_table, const int* __restrict__ token_slot,
     const int* __restrict__ positions, int T, int nh, int nkv, int hd, int vd, int page_size, int max_pages,
-    int window, float scale, int chunk, float softcap, float sink) {
+    int window, float scale, int chunk, float softcap, float sink, int ld_v, const float* __restrict__ slopes,
+    const float* __restrict__ sinks, const float* __restrict__ gate, int ld_gate) {
   __shared__ __align__(16) float q_s[WARPS][HDM];
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const long long item = (long long)blockIdx.x * WARPS + warp;
@@ -47,6 +51,7 @@ __global__ void __launch_bounds__(WARPS * 32) attention_f32_kernel(
   for (int d = lane; d < hd; d += 32) q_s[warp][d] = qv[d];
   __syncwarp();
 
+  const float slope = slopes != nullptr ? slopes[h] : 0.0f;
   float m = -CUDART_INF_F, l = 0.0f;
   float acc[HDM / 32];
 #pragma unroll
@@ -77,6 +82,7 @@ __global__ void __launch_bounds__(WARPS * 32) attention_f32_kernel(
       }
       s = dot * scale;
       if (softcap > 0.0f) s = softcap * tanhf(s / softcap);
+      s = fmaf(slope, (float)(key - pos), s);
     }
     const float m_new = fmaxf(m, jb::warp_max(s));
     const float p = valid ? expf(s - m_new) : 0.0f;
@@ -94,7 +100,7 @@ __global__ void __launch_bounds__(WARPS * 32) attention_f32_kernel(
       for (int u = 0; u < U; ++u) {
         const int key2 = c0 + min(kk0 + u, n_keys - 1);
         const int page = pages[key2 / page_size], row = key2 % page_size;
-        const float* vr = v_cache + (((size_t)page * nkv + kvh) * page_size + row) * hd;
+        const float* vr = v_cache + (((size_t)page * nkv + kvh) * page_size + row) * ld_v;
 #pragma unroll
         for (int j = 0; j < HDM / 32; ++j) {
           const int d = lane + 32 * j;
@@ -114,11 +120,13 @@ __global__ void __launch_bounds__(WARPS * 32) attention_f32_kernel(
     m = m_new;
   }
   if (sink > 0.0f) l += sink * expf(m == -CUDART_INF_F ? 0.0f : -m);
+  if (sinks != nullptr) l += expf(sinks[h] - (m == -CUDART_INF_F ? 0.0f : m));
+  const float open = gate != nullptr ? 1.0f / (1.0f + expf(-gate[(size_t)t * ld_gate + h])) : 1.0f;
   float* o = out + ((size_t)t * nh + h) * vd;
 #pragma unroll
   for (int j = 0; j < HDM / 32; ++j) {
     const int d = lane + 32 * j;
-    if (d < vd) o[d] = acc[j] / l;
+    if (d < vd) o[d] = acc[j] / l * open;
   }
 }
 
@@ -127,10 +135,12 @@ __global__ void __launch_bounds__(WARPS * 32) attention_f32_kernel(
 JB_EXPORT int jb_attention_f32(const float* q, const float* k_cache, const float* v_cache, float* out,
                                const int* block_table, const int* token_slot, const int* positions, int T,
                                int nh, int nkv, int hd, int vd, int page_size, int max_pages, int window, float scale,
-                               int chunk, float softcap, float sink, cudaStream_t stream) {
+                               int chunk, float softcap, float sink, int ld_v, const float* slopes, const float* sinks,
+                               const float* gate, int ld_gate, cudaStream_t stream) {
   if (T <= 0) return 0;
-  JB_REFUSE(hd > MAX_HD || hd <= 0 || vd <= 0 || vd > hd, "attention_f32: head_dim %d is outside (0, %d], or its values (%d) are wider",
-            hd, MAX_HD, vd);
+  JB_REFUSE(hd > MAX_HD || hd <= 0 || vd <= 0 || vd > ld_v || vd > (hd <= SMALL_HD ? SMALL_HD : MAX_HD),
+            "attention_f32: head_dim %d is outside (0, %d], or its values (%d) are wider than their rows or the kernel", hd,
+            MAX_HD, vd);
   JB_REFUSE(nkv <= 0 || nh % nkv != 0, "attention_f32: %d heads are not a multiple of %d kv heads", nh, nkv);
   const long long items = (long long)T * nh;
   const unsigned blocks = (unsigned)((items + WARPS - 1) / WARPS);
@@ -139,7 +149,8 @@ JB_EXPORT int jb_attention_f32(const float* q, const float* k_cache, const float
   attention_f32_kernel<VEC, HDM, U><<<blocks, WARPS * 32, 0, stream>>>(q, k_cache, v_cache, out, block_table,      \
                                                                        token_slot, positions, T, nh, nkv, hd, vd,  \
                                                                        page_size, max_pages, window, scale, chunk, \
-                                                                       softcap, sink)
+                                                                       softcap, sink, ld_v, slopes, sinks, gate,   \
+                                                                       ld_gate)
   if (hd <= SMALL_HD) {
     if (vec) JB_GO(true, SMALL_HD, 8);
     else JB_GO(false, SMALL_HD, 8);

@@ -275,9 +275,18 @@ __device__ __forceinline__ void scale16(uint32_t* r, float f) {
 // [floor(pos / chunk) chunk, pos].  cap_s > 0: a raw score s becomes cap_s tanh(s inv_cap), with cap_s = cap / scale
 // and inv_cap = scale / cap, so that the scale applied afterwards gives cap tanh(s scale / cap).
 // sink = 1: the softmax's denominator has one more term, exp(0) (a key of score 0 that has no value).
+// slopes (one per query head, or null): slope (position - key position) is taken off the scaled score; inv_scale = 1 / scale.
+// sinks (one per query head, or null): the denominator has one more term, exp(sinks[head]).
+// gate (float32 rows of ld_gate numbers, a row per token, a number per query head, or null): a head's output is multiplied
+// by the number's sigmoid.
 struct Cap {
   int chunk;
   float cap_s, inv_cap, sink;
+  const float* slopes;
+  float inv_scale;
+  const float* sinks;
+  const float* gate;
+  int ld_gate;
 };
 // Where keys and values lie.  start null: in pages.  Else in a matrix: the key of position p of sequence s is row
 // start[s] + p, head h's key begins at column h hd of the keys' map and its value at column h vd of the values' map.
@@ -298,6 +307,37 @@ template <int N>
 __device__ __forceinline__ void cap_scores(uint32_t* sr, const Cap& cap) {
 #pragma unroll
   for (int c = 0; c < N; ++c) sr[c] = __float_as_uint(cap.cap_s * tanh_abs(__uint_as_float(sr[c]) * cap.inv_cap));
+}
+
+// sr[c] += slope (d0 + c): a bias that is linear in the distance (d0 <= 0 of the first key, in whole numbers, which float32
+// holds exactly), one rounding a score.
+template <int N>
+__device__ __forceinline__ void bias_scores(uint32_t* sr, float slope, float d0) {
+  const uint64_t s2 = pack2(slope, slope), step = pack2(8.0f, 8.0f);
+  uint64_t d[4];
+#pragma unroll
+  for (int k = 0; k < 4; ++k) d[k] = pack2(d0 + 2.0f * k, d0 + 2.0f * k + 1.0f);
+#pragma unroll
+  for (int c = 0; c < N / 2; ++c) {
+    float a, b;
+    unpack2(fma2(s2, d[c & 3], pack2(__uint_as_float(sr[2 * c]), __uint_as_float(sr[2 * c + 1]))), a, b);
+    d[c & 3] = add2(d[c & 3], step);
+    sr[2 * c] = __float_as_uint(a);
+    sr[2 * c + 1] = __float_as_uint(b);
+  }
+}
+// A row's softmax denominator l, relative to m_ref (in units of log2), with what a sink adds to it.
+__device__ __forceinline__ float with_sink(float l, float m_ref, const Cap& cap, int head) {
+  const float ref = m_ref == -CUDART_INF_F ? 0.0f : m_ref;
+  if (cap.sink > 0.0f) l += cap.sink * exp2f(-ref);
+  if (cap.sinks != nullptr) l += exp2f(cap.sinks[head] * LOG2E - ref);
+  return l;
+}
+// What a row's sums are multiplied by at the end: 1 / l, times the sigmoid of the head's gate.
+__device__ __forceinline__ float row_factor(float l, const Cap& cap, int token, int head) {
+  float f = 1.0f / l;
+  if (cap.gate != nullptr) f *= 1.0f / (1.0f + expf(-cap.gate[(size_t)token * cap.ld_gate + head]));
+  return f;
 }
 
 template <int NT>
@@ -453,6 +493,8 @@ __global__ void __launch_bounds__(threads_for(NT), 1) prefill_tc_kernel(
     const int row_lo = chunk_lo(window > 0 ? max(0, row_pos - window + 1) : 0, row_pos, cap.chunk);
     const uint32_t lane_addr = tmem + ((uint32_t)(quarter * 32) << 16);
     const uint32_t s_col = TMEM_S0 + w * 128, o_col = TMEM_O0 + w * HD;
+    const int head = kvh * G + row % G;
+    const float slope = cap.slopes != nullptr ? cap.slopes[head] * cap.inv_scale : 0.0f;
     float m_ref = -CUDART_INF_F, l = 0.0f;   // l is the row sum relative to m_ref
     bool ok = true;
     for (int j = 0; j < nb && ok; ++j) {
@@ -466,6 +508,7 @@ __global__ void __launch_bounds__(threads_for(NT), 1) prefill_tc_kernel(
       tmem_ld_wait();
       if (cap.cap_s > 0.0f) cap_scores<64>(sr, cap);
       const int key0 = (kb_start + j) * PAGE;
+      if (cap.slopes != nullptr) bias_scores<64>(sr, slope, (float)(key0 - row_pos));
       if (key0 + PAGE - 1 > row_pos || key0 < row_lo) {   // only blocks that touch the causal edge or the window
 #pragma unroll
         for (int c = 0; c < 64; ++c) {
@@ -509,9 +552,9 @@ __global__ void __launch_bounds__(threads_for(NT), 1) prefill_tc_kernel(
     if (ok && nb > 0) ok = mbar_wait(o_done(w), 0, status, 13);
     if (ok) {
       tc_fence_after();
-      if (cap.sink > 0.0f) l += cap.sink * exp2f(m_ref == -CUDART_INF_F ? 0.0f : -m_ref);
-      const float inv = 1.0f / l;
-      bf16* dst = out + ((size_t)(qs + tok_first + (valid ? tl : 0)) * nh + kvh * G + row % G) * keys.vd;
+      const int token = qs + tok_first + (valid ? tl : 0);
+      const float inv = row_factor(with_sink(l, m_ref, cap, head), cap, token, head);
+      bf16* dst = out + ((size_t)token * nh + head) * keys.vd;
 #pragma unroll
       for (int c0 = 0; c0 < HD; c0 += 16) {
         if (c0 >= keys.vd) break;
@@ -709,6 +752,8 @@ __global__ void __launch_bounds__(T2_THREADS, 1) prefill_tc128_kernel(
     const int row_lo = chunk_lo(window > 0 ? max(0, row_pos - window + 1) : 0, row_pos, cap.chunk);
     const uint32_t lane_addr = tmem + ((uint32_t)(quarter * 32) << 16);
     const uint32_t s_col = w * 128, o_col = 256 + w * 128;
+    const int head = kvh * G + row % G;
+    const float slope = cap.slopes != nullptr ? cap.slopes[head] * cap.inv_scale : 0.0f;
     float m_ref = -CUDART_INF_F, l = 0.0f;
     bool ok = true;
     for (int j = 0; j < nb && ok; ++j) {
@@ -721,6 +766,7 @@ __global__ void __launch_bounds__(T2_THREADS, 1) prefill_tc128_kernel(
       tmem_ld_wait();
       if (cap.cap_s > 0.0f) cap_scores<KB>(sr, cap);
       const int key0 = (kb_start + j) * KB;
+      if (cap.slopes != nullptr) bias_scores<KB>(sr, slope, (float)(key0 - row_pos));
       if (key0 + KB - 1 > row_pos || key0 < row_lo) {
 #pragma unroll
         for (int c = 0; c < KB; ++c) {
@@ -762,9 +808,9 @@ __global__ void __launch_bounds__(T2_THREADS, 1) prefill_tc128_kernel(
     if (ok && nb > 0) ok = mbar_wait(o_done(w), 0, status, 13);
     if (ok) {
       tc_fence_after();
-      if (cap.sink > 0.0f) l += cap.sink * exp2f(m_ref == -CUDART_INF_F ? 0.0f : -m_ref);
-      const float inv = 1.0f / l;
-      bf16* dst = out + ((size_t)(qs + tok_first + (valid ? tl : 0)) * nh + kvh * G + row % G) * keys.vd;
+      const int token = qs + tok_first + (valid ? tl : 0);
+      const float inv = row_factor(with_sink(l, m_ref, cap, head), cap, token, head);
+      bf16* dst = out + ((size_t)token * nh + head) * keys.vd;
 #pragma unroll
       for (int c0 = 0; c0 < HD; c0 += 16) {
         if (c0 >= keys.vd) break;
@@ -906,32 +952,43 @@ JB_EXPORT int jb_attention_tc_prefill(const void* q, const void* k_cache, const 
                                       int page_size, int max_pages, int window, float scale, int* status,
                                       cudaStream_t stream) {
   return tc_prefill_launch(q, k_cache, v_cache, out, block_table, q_start, kv_len, T, n_pages, n_seqs, max_q_len, nh,
-                           nkv, hd, page_size, max_pages, window, scale, Cap{0, 0.0f, 0.0f}, status, stream, Keys{nullptr, hd});
+                           nkv, hd, page_size, max_pages, window, scale, Cap{}, status, stream, Keys{nullptr, hd});
 }
 
 // As jb_attention_tc_prefill, with a chunked mask (chunk > 0: a query sees only the keys of its own chunk of
-// positions, counted from the sequence's first), capped scores (softcap > 0: s -> softcap tanh(s / softcap)) and a
-// sink (sink = 1: one more term exp(0) in the softmax's denominator).
+// positions, counted from the sequence's first), capped scores (softcap > 0: s -> softcap tanh(s / softcap)), a
+// sink (sink = 1: one more term exp(0) in the softmax's denominator; sinks [nh]: one more term exp(sinks[head])), a
+// distance bias (slopes [nh]: slopes[head] (position - key position) is taken off), an output gate (gate: float32 rows of
+// ld_gate numbers, column `head` for each; its sigmoid multiplies the head's output) and values of vd <= hd numbers (the
+// value pages [n_pages, nkv, 64, vd], out [T, nh vd]).  slopes, sinks, gate: device memory, or null.
 JB_EXPORT int jb_attention_tc_prefill_capped(const void* q, const void* k_cache, const void* v_cache, void* out,
                                              const int* block_table, const int* q_start, const int* kv_len, int T,
-                                             int n_pages, int n_seqs, int max_q_len, int nh, int nkv, int hd,
+                                             int n_pages, int n_seqs, int max_q_len, int nh, int nkv, int hd, int vd,
                                              int page_size, int max_pages, int window, float scale, int chunk,
-                                             float softcap, float sink, int* status, cudaStream_t stream) {
+                                             float softcap, float sink, const float* slopes, const float* sinks,
+                                             const float* gate, int ld_gate, int* status, cudaStream_t stream) {
   JB_REFUSE(chunk < 0 || softcap < 0.0f || scale <= 0.0f, "attention_tc: a chunk, a cap and a scale cannot be negative");
-  const Cap cap = softcap > 0.0f ? Cap{chunk, softcap / scale, scale / softcap, sink} : Cap{chunk, 0.0f, 0.0f, sink};
+  JB_REFUSE(vd <= 0 || vd > hd || vd % 8 != 0, "attention_tc: values of %d numbers beside keys of %d", vd, hd);
+  const bool capped = softcap > 0.0f;
+  const Cap cap{chunk, capped ? softcap / scale : 0.0f, capped ? scale / softcap : 0.0f, sink, slopes, 1.0f / scale, sinks,
+                gate, ld_gate};
   return tc_prefill_launch(q, k_cache, v_cache, out, block_table, q_start, kv_len, T, n_pages, n_seqs, max_q_len, nh,
-                           nkv, hd, page_size, max_pages, window, scale, cap, status, stream, Keys{nullptr, hd});
+                           nkv, hd, page_size, max_pages, window, scale, cap, status, stream, Keys{nullptr, vd});
 }
 
 // Causal attention with a key and a value head per query head, keys and values in one matrix kv [kv_rows][nh hd | nh vd]
 // (bfloat16): the key of position p of sequence s is row kv_start[s] + p.  q: [T, nh hd], out: [T, nh vd]; hd and vd are
 // multiples of 8, vd <= hd <= the build's row.  max_kv_len bounds a sequence's length (it picks the order of the blocks).
+// gate: as above, or null.
 JB_EXPORT int jb_attention_tc_matrix(const void* q, const void* kv, void* out, const int* kv_start, const int* q_start,
                                      const int* kv_len, int T, int kv_rows, int n_seqs, int max_q_len, int nh, int hd, int vd,
-                                     int max_kv_len, float scale, int* status, cudaStream_t stream) {
+                                     int max_kv_len, float scale, const float* gate, int ld_gate, int* status,
+                                     cudaStream_t stream) {
+  Cap cap{};
+  cap.gate = gate, cap.ld_gate = ld_gate;
   JB_REFUSE(vd <= 0 || vd > hd || vd % 8 != 0 || kv_rows <= 0 || kv_start == nullptr,
             "attention_tc: values of %d numbers beside keys of %d, in %d rows", vd, hd, kv_rows);
   return tc_prefill_launch(q, kv, (const bf16*)kv + (size_t)nh * hd, out, nullptr, q_start, kv_len, T, 0, n_seqs, max_q_len,
-                           nh, nh, hd, PAGE, (max_kv_len + PAGE - 1) / PAGE, 0, scale, Cap{0, 0.0f, 0.0f}, status, stream,
+                           nh, nh, hd, PAGE, (max_kv_len + PAGE - 1) / PAGE, 0, scale, cap, status, stream,
                            Keys{kv_start, vd}, kv_rows);
 }

@@ -93,9 +93,12 @@ template <> __device__ __forceinline__ __nv_bfloat16 from_f32<__nv_bfloat16>(flo
 // clamped form g * sigmoid(alpha g) * (u + 1) with g = min(gate, limit), u = clamp(up, -limit, limit).  limit < 0: the
 // tanh form of GELU, 0.5 g (1 + tanh(sqrt(2/pi) (g + 0.044715 g^3))) * up, written with
 // 0.5 (1 + tanh(a)) = 1 / (1 + exp(-2a)).
+// (`act` is the activation of a product without a gate, see `activated`.)
+enum Activation { ACT_GELU = 0, ACT_RELU2 = 1 };
 struct Gate {
   float limit;
   float alpha;
+  int act = ACT_GELU;
 };
 __device__ __forceinline__ float gated(float g, float u, const Gate& gate) {
   if (gate.limit > 0.0f) {
@@ -112,6 +115,14 @@ __device__ __forceinline__ float gated(float g, float u, const Gate& gate) {
 
 // GELU by the normal distribution's own integral, 0.5 z (1 + erf(z / sqrt(2))).
 __device__ __forceinline__ float gelu_erf(float z) { return 0.5f * z * (1.0f + erff(z * 0.70710678118654752f)); }
+
+// The square of what is above zero.
+__device__ __forceinline__ float relu2(float z) {
+  const float p = fmaxf(z, 0.0f);
+  return p * p;
+}
+// The activation of a product without a gate.
+__device__ __forceinline__ float activated(float z, int act) { return act == ACT_RELU2 ? relu2(z) : gelu_erf(z); }
 
 __device__ __forceinline__ float warp_sum(float v) {
 #pragma unroll

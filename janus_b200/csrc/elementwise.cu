@@ -393,9 +393,9 @@ JB_EXPORT int jb_clamped_glu(const float* gate_up, int ld, int up_col, void* out
 }
 
 namespace {
-// out = gelu(x): four numbers a thread (n4 groups), float32 in, the engine dtype out
+// out = act(x) (`jb::activated`): four numbers a thread (n4 groups), float32 in, the engine dtype out
 template <typename TO>
-__global__ void gelu_rows_kernel(const float* __restrict__ x, TO* __restrict__ out, size_t n, int vec) {
+__global__ void activate_rows_kernel(const float* __restrict__ x, TO* __restrict__ out, size_t n, int vec, int act) {
   jb::pdl_launch_dependents();
   jb::pdl_wait();
   const size_t step = (size_t)gridDim.x * blockDim.x;
@@ -403,25 +403,27 @@ __global__ void gelu_rows_kernel(const float* __restrict__ x, TO* __restrict__ o
   if (vec) {
     for (; i < n / 4; i += step) {
       const float4 v = reinterpret_cast<const float4*>(x)[i];
-      __align__(16) TO r[4] = {jb::from_f32<TO>(jb::gelu_erf(v.x)), jb::from_f32<TO>(jb::gelu_erf(v.y)),
-                 jb::from_f32<TO>(jb::gelu_erf(v.z)), jb::from_f32<TO>(jb::gelu_erf(v.w))};
+      __align__(16) TO r[4] = {jb::from_f32<TO>(jb::activated(v.x, act)), jb::from_f32<TO>(jb::activated(v.y, act)),
+                 jb::from_f32<TO>(jb::activated(v.z, act)), jb::from_f32<TO>(jb::activated(v.w, act))};
       if constexpr (sizeof(TO) == 2) reinterpret_cast<uint2*>(out)[i] = *reinterpret_cast<uint2*>(r);
       else reinterpret_cast<float4*>(out)[i] = *reinterpret_cast<float4*>(r);
     }
     return;
   }
-  for (; i < n; i += step) out[i] = jb::from_f32<TO>(jb::gelu_erf(x[i]));
+  for (; i < n; i += step) out[i] = jb::from_f32<TO>(jb::activated(x[i], act));
 }
 }  // namespace
 
-// The activation behind a plain product: out = gelu(x) (`jb::gelu_erf`) for n float32 numbers, out in out_dtype.
-JB_EXPORT int jb_gelu(const float* x, void* out, int out_dtype, long long n, cudaStream_t stream) {
+// The activation behind a plain product: out = act(x) for n float32 numbers, out in out_dtype; act: 0 `jb::gelu_erf`,
+// 1 `jb::relu2`.
+JB_EXPORT int jb_activate(const float* x, void* out, int out_dtype, long long n, int act, cudaStream_t stream) {
   if (n <= 0) return 0;
+  JB_REFUSE(act != jb::ACT_GELU && act != jb::ACT_RELU2, "activate: unknown activation %d", act);
   const int vec = n % 4 == 0 && (((uintptr_t)x | (uintptr_t)out) & 15) == 0;
   const long long want = (n / (vec ? 4 : 1) + 255) / 256;
   jb::Launch cfg(dim3((unsigned)(want < 148 * 16 ? want : 148 * 16)), dim3(256), 0, stream);
-  if (out_dtype == JB_F32) return (int)cudaLaunchKernelEx(&cfg.c, gelu_rows_kernel<float>, x, (float*)out, (size_t)n, vec);
-  if (out_dtype == JB_BF16) return (int)cudaLaunchKernelEx(&cfg.c, gelu_rows_kernel<bf16>, x, (bf16*)out, (size_t)n, vec);
+  if (out_dtype == JB_F32) return (int)cudaLaunchKernelEx(&cfg.c, activate_rows_kernel<float>, x, (float*)out, (size_t)n, vec, act);
+  if (out_dtype == JB_BF16) return (int)cudaLaunchKernelEx(&cfg.c, activate_rows_kernel<bf16>, x, (bf16*)out, (size_t)n, vec, act);
   return JB_ERR_BAD_DTYPE;
 }
 

@@ -61,7 +61,7 @@ constexpr int epi_warps(int bn) {
 static_assert(JB_EPI_WARPS == 0 || JB_EPI_WARPS == 4 || JB_EPI_WARPS == 8 || JB_EPI_WARPS == 16, "4, 8 or 16 epilogue warps");
 constexpr int threads_for(int bn) { return 64 + 32 * epi_warps(bn); }
 
-enum Mode { STORE_BF16 = 0, STORE_F32 = 1, ADD_F32 = 2, SWIGLU = 3, ADD_ORDERED = 4, STORE_GELU = 5 };   // 4: ADD_F32 with K cut, slices summed in order
+enum Mode { STORE_BF16 = 0, STORE_F32 = 1, ADD_F32 = 2, SWIGLU = 3, ADD_ORDERED = 4, STORE_ACT = 5 };   // 4: ADD_F32 with K cut, slices summed in order
 
 // How long a wait on an mbarrier may last before the kernel gives up (2 s; a test build sets a few ms).
 #ifndef JB_WAIT_LIMIT_NS
@@ -458,8 +458,8 @@ __global__ void __launch_bounds__(threads_for(BN)) gemm_tc_kernel(const __grid_c
                 const size_t o = (size_t)t * ldy + f;
                 if (MODE == STORE_BF16) {
                   ((__nv_bfloat16*)Y)[o] = __float2bfloat16_rn(v);
-                } else if (MODE == STORE_GELU) {
-                  ((__nv_bfloat16*)Y)[o] = __float2bfloat16_rn(jb::gelu_erf(v));
+                } else if (MODE == STORE_ACT) {
+                  ((__nv_bfloat16*)Y)[o] = __float2bfloat16_rn(jb::activated(v, gate.act));
                 } else if (MODE == STORE_F32) {
                   ((float*)Y)[o] = v;
                 } else if (MODE == ADD_F32) {
@@ -625,7 +625,8 @@ int dispatch(const CUtensorMap& mw, const void* X, void* Y, int T, int N_out, in
 // (`w_tiles` tiles of 16 KB in all; for mode SWIGLU the gate rows' tiles first and the up rows' tiles from row
 // tile `up_tile_offset` on); Y: [T, ldy] with N_out columns used.
 // mode: 0 store bf16, 1 store f32, 2 add into f32, 3 act(gate)*up -> bf16 (`jb::gated` with gate_limit, gate_alpha:
-// limit 0 is SiLU, limit < 0 the tanh form of GELU), 5 store gelu(result) -> bf16 (`jb::gelu_erf`).
+// limit 0 is SiLU, limit < 0 the tanh form of GELU), 5 store gelu(result) -> bf16 (`jb::gelu_erf`),
+// 6 store relu(result)^2 -> bf16 (`jb::relu2`).
 // split_k > 1 only with mode 2: partial sums meet in Y through atomic adds, or, if `partials` (room for
 // `partial_floats` floats) and `tickets` (`n_tickets` ints, zero) are given, in the fixed order of the slices:
 // tiles x slices x 128 x token tile floats and one ticket per output tile are needed (token tile: 16, 32, 64,
@@ -639,7 +640,7 @@ JB_EXPORT int jb_gemm_bf16(const void* X, const void* W, long long w_tiles, int 
   if (T <= 0 || N_out <= 0) return 0;
   JB_REFUSE(K <= 0 || K % 8 != 0, "gemm_bf16: K = %d must be a positive multiple of 8 (16-byte rows for TMA)", K);
   JB_REFUSE(((uintptr_t)X | (uintptr_t)W) & 15, "gemm_bf16: operands must be 16-byte aligned");
-  JB_REFUSE(mode < 0 || mode > 5 || mode == ADD_ORDERED, "gemm_bf16: unknown mode %d", mode);
+  JB_REFUSE(mode < 0 || mode > 6 || mode == ADD_ORDERED, "gemm_bf16: unknown mode %d", mode);
   JB_REFUSE(split_k < 1 || (split_k > 1 && mode != ADD_F32), "gemm_bf16: K can be split only in mode 2");
   const long long k_tiles = (K + BK - 1) / BK, row_tiles = (N_out + BM - 1) / BM;
   const long long need = mode == SWIGLU ? (up_tile_offset + row_tiles) * k_tiles : row_tiles * k_tiles;
@@ -649,7 +650,10 @@ JB_EXPORT int jb_gemm_bf16(const void* X, const void* W, long long w_tiles, int 
   if (!make_packed_map(&mw, W, (uint64_t)w_tiles)) return JB_ERR_TENSORMAP;
   switch (mode) {
     case STORE_BF16: return dispatch<STORE_BF16>(mw, X, Y, T, N_out, K, ldy, 1, 0, none, status, stream);
-    case STORE_GELU: return dispatch<STORE_GELU>(mw, X, Y, T, N_out, K, ldy, 1, 0, none, status, stream);
+    case STORE_ACT:
+    case STORE_ACT + 1:
+      return dispatch<STORE_ACT>(mw, X, Y, T, N_out, K, ldy, 1, 0, none, status, stream,
+                                 jb::Gate{0.0f, 1.0f, mode == STORE_ACT ? jb::ACT_GELU : jb::ACT_RELU2});
     case STORE_F32: return dispatch<STORE_F32>(mw, X, Y, T, N_out, K, ldy, 1, 0, none, status, stream);
     case ADD_F32:
       if (split_k > 1 && partials != nullptr)

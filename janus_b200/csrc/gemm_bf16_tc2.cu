@@ -44,7 +44,7 @@ constexpr int EPI_PARTS = EPI_WARPS / 4;
 constexpr int THREADS = 64 + 32 * EPI_WARPS;
 constexpr uint32_t PEER_MASK = 0xFEFFFFFFu;  // clears the CTA-rank bit of a shared::cluster address: the pair's first CTA
 
-enum Mode { STORE_BF16 = 0, STORE_F32 = 1, ADD_F32 = 2, SWIGLU = 3, QKV_ROPE = 4, STORE_GELU = 5 };
+enum Mode { STORE_BF16 = 0, STORE_F32 = 1, ADD_F32 = 2, SWIGLU = 3, QKV_ROPE = 4, STORE_ACT = 5 };
 
 constexpr unsigned long long WAIT_LIMIT_NS = 2000000000ull;
 
@@ -466,8 +466,8 @@ __global__ void __launch_bounds__(THREADS) gemm_tc2_kernel(const __grid_constant
                 const size_t o = (size_t)t * ldy + f;
                 if (MODE == STORE_BF16) {
                   ((__nv_bfloat16*)Y)[o] = __float2bfloat16_rn(v);
-                } else if (MODE == STORE_GELU) {
-                  ((__nv_bfloat16*)Y)[o] = __float2bfloat16_rn(jb::gelu_erf(v));
+                } else if (MODE == STORE_ACT) {
+                  ((__nv_bfloat16*)Y)[o] = __float2bfloat16_rn(jb::activated(v, gate.act));
                 } else if (MODE == STORE_F32) {
                   ((float*)Y)[o] = v;
                 } else {
@@ -612,7 +612,7 @@ int launch(const void* X, const void* W, long long w_tiles, int up_tile_offset, 
 // `whole_tiles` output tiles (256 x 256, token tile fastest) stay uncut: the tiles that fill whole waves of CTA
 // pairs, so that only the last, partial wave is cut.
 // Mode SWIGLU applies `jb::gated` with (gate_limit, gate_alpha): limit 0 is SiLU, limit < 0 the tanh form of GELU;
-// mode STORE_GELU stores `jb::gelu_erf` of the results in bf16.
+// mode 5 stores `jb::gelu_erf` of the results in bf16, mode 6 `jb::relu2`.
 // Meant for prompt-sized T.  status codes of a timed-out wait: 21 producer, 22 MMA, 23 epilogue.
 JB_EXPORT int jb_gemm_bf16_pair(const void* X, const void* W, long long w_tiles, int up_tile_offset, void* Y, int T,
                                 int N_out, int K, int ldy, int mode, int split_k, int whole_tiles, float gate_limit,
@@ -622,7 +622,10 @@ JB_EXPORT int jb_gemm_bf16_pair(const void* X, const void* W, long long w_tiles,
   JB_REFUSE(((uintptr_t)X | (uintptr_t)W) & 15, "gemm_bf16_pair: operands must be 16-byte aligned");
   switch (mode) {
     case STORE_BF16: return launch<STORE_BF16>(X, W, w_tiles, up_tile_offset, Y, T, N_out, K, ldy, RopeOut{}, status, stream);
-    case STORE_GELU: return launch<STORE_GELU>(X, W, w_tiles, up_tile_offset, Y, T, N_out, K, ldy, RopeOut{}, status, stream);
+    case STORE_ACT:
+    case STORE_ACT + 1:
+      return launch<STORE_ACT>(X, W, w_tiles, up_tile_offset, Y, T, N_out, K, ldy, RopeOut{}, status, stream, 1, 0,
+                               jb::Gate{0.0f, 1.0f, mode == STORE_ACT ? jb::ACT_GELU : jb::ACT_RELU2});
     case STORE_F32: return launch<STORE_F32>(X, W, w_tiles, up_tile_offset, Y, T, N_out, K, ldy, RopeOut{}, status, stream);
     case ADD_F32: return launch<ADD_F32>(X, W, w_tiles, up_tile_offset, Y, T, N_out, K, ldy, RopeOut{}, status, stream, split_k, whole_tiles);
     case SWIGLU:

@@ -8,9 +8,11 @@
 //                    the token's row is normed, turned and appended to the pages (and to `rows` [T, stored], if given)
 //   latent_queries   queries in the latents' space: q_out[t, h] = [Wuk_h^T q | turned q], so that the score with the
 //                    cached row itself is the head's score; the token's row as above
+//   latent_down      where the queries have a latent of their own (m numbers at column 0): it is normed and written for the
+//                    product that makes the queries from it; the token's row as above
 //   latent_values    out[t, h] = Wuv_h o, o = sum_j p_j c_j the attention's output in the latents' space, from rows
 //                    [T, H, n] or straight from the partial sums that the splits of the keys left; times the sigmoid
-//                    of an output gate, if there is one
+//                    of an output gate, if there is one (a number for every value, or one per head)
 //   gather_rows      the cached rows of a step's sequences, sequence after sequence, in one matrix
 //
 // The rotation turns the pair (i, i + r/2) by the position's angle; cos and sin come from a table [positions][r/2][2].
@@ -131,6 +133,33 @@ __global__ void __launch_bounds__(256) latent_prep_kernel(const float* __restric
       q[i] = jb::from_f32<TO>(v);
     }
   }
+}
+
+// a_out[t] = x / rms(x) * w with x = proj[t, 0 : m], a block per token (blockIdx.y == 0); the token's row, another one
+// (blockIdx.y == 1).  All blocks together set the n_clear float4 at `clear` to zero.
+template <typename TO>
+__global__ void __launch_bounds__(256) latent_down_kernel(const float* __restrict__ proj, int ld, int m,
+                                                          const float* __restrict__ w, float eps, TO* __restrict__ a_out,
+                                                          const float* __restrict__ table, const int* __restrict__ positions,
+                                                          float4* __restrict__ clear, long long n_clear, Row row) {
+  __shared__ float scratch[33];
+  jb::pdl_launch_dependents();
+  jb::pdl_wait();
+  const int t = blockIdx.x;
+  const float* x = proj + (size_t)t * ld;
+  const long long blocks = (long long)gridDim.x * gridDim.y, block = (long long)blockIdx.y * gridDim.x + t;
+  for (long long i = block * blockDim.x + threadIdx.x; i < n_clear; i += blocks * blockDim.x)
+    clear[i] = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+  if (blockIdx.y == 1) {
+    const float* cs = table != nullptr && row.r > 0 ? table + (size_t)positions[t] * (row.r >> 1) * 2 : nullptr;
+    write_row<TO>(x, row, cs, t, scratch);
+    return;
+  }
+  float ss = 0.0f;
+  for (int i = threadIdx.x; i < m; i += blockDim.x) ss = fmaf(x[i], x[i], ss);
+  ss = jb::block_sum(ss, scratch);
+  const float inv = 1.0f / sqrtf(ss / (float)m + eps);
+  for (int i = threadIdx.x; i < m; i += blockDim.x) a_out[(size_t)t * m + i] = jb::from_f32<TO>((x[i] * inv) * w[i]);
 }
 
 // V numbers of a weight row (16 bytes, or one number): the bits are loaded early and unpacked late.
@@ -258,7 +287,8 @@ __global__ void __launch_bounds__(Q_THREADS) latent_queries_kernel(
 constexpr int VT = 4;              // tokens of a block of latent_values
 constexpr int V_WARPS = 8, V_ROWS = 4;
 
-// out[t, h, c] = (uv[h e + c, :] . o[t, h]) * sigmoid(gate[t, h e + c]) for c < e, zero for e <= c < ep.  o comes from
+// out[t, h, c] = (uv[h e + c, :] . o[t, h]) * sigmoid(gate[t, h e + c]) for c < e, zero for e <= c < ep (gate_per_head:
+// the gate's column is h).  o comes from
 // `o_rows` [T, H, n] (splits == 0), or from the key splits' partial sums: part_o [T, H, splits, n] and part_ml
 // [T, H, splits, 2] (maximum in units of log2, sum), o = sum_s f_s part_o[s] / sum_s f_s l_s with f_s = 2^(m_s - max).
 // A block owns (a chunk of V_WARPS * V_ROWS value rows, head, VT tokens); a warp takes V_ROWS rows, whose first columns
@@ -267,8 +297,8 @@ constexpr int V_WARPS = 8, V_ROWS = 4;
 template <typename T, int V>
 __global__ void __launch_bounds__(V_WARPS * 32) latent_values_kernel(
     const T* __restrict__ o_rows, const float* __restrict__ part_o, const float* __restrict__ part_ml, int splits,
-    const T* __restrict__ uv, const float* __restrict__ gate, int ld_gate, T* __restrict__ out, int n_tokens, int H, int n,
-    int e, int ep) {
+    const T* __restrict__ uv, const float* __restrict__ gate, int ld_gate, int gate_per_head, T* __restrict__ out,
+    int n_tokens, int H, int n, int e, int ep) {
   extern __shared__ __align__(16) float o_s[];   // [VT][n padded to 8], then the splits' factors [VT][splits]
   jb::pdl_launch_dependents();
   cg::cluster_group cluster = cg::this_cluster();
@@ -292,7 +322,7 @@ __global__ void __launch_bounds__(V_WARPS * 32) latent_values_kernel(
   // the sum this lane will write: row my_c of token my_k; its gate is asked for early (no gate: z -> infinity, sigmoid 1)
   const int my_c = c0 + (lane >> 1) / VT, my_k = (lane >> 1) % VT;
   float z = CUDART_INF_F;
-  if (gate != nullptr && my_k < nt && my_c < e) z = gate[(size_t)(t0 + my_k) * ld_gate + (size_t)h * e + my_c];
+  if (gate != nullptr && my_k < nt && my_c < e) z = gate[(size_t)(t0 + my_k) * ld_gate + (gate_per_head ? (size_t)h : (size_t)h * e + my_c)];
   if (splits > 0) {
     float* f_s = o_s + VT * np;
     if (warp < nt) {                             // a warp per token: lanes over the splits
@@ -411,14 +441,18 @@ __global__ void __launch_bounds__(256) gather_rows_kernel(const uint4* __restric
 
 bool aligned16(const void* p) { return ((uintptr_t)p & 15) == 0; }
 
-int check_row(int ld, int q_col, int H, int d, int r, const Row& row) {
-  JB_REFUSE(H < 1 || d < 0 || r < 0 || (r & 1) || d + r < 1, "latent: %d heads of %d + %d numbers", H, d, r);
-  JB_REFUSE(ld < q_col + H * (d + r), "latent: rows of %d floats do not hold the queries", ld);
+int check_row(int ld, int r, const Row& row) {
+  JB_REFUSE(r < 0 || (r & 1), "latent: %d rotated numbers", r);
   JB_REFUSE(row.c_cache != nullptr && (ld < row.c_col + row.n + row.r || row.stored < row.n + row.r || row.n < 1 ||
                                        row.r != r || row.w == nullptr || row.dest == nullptr),
             "latent: rows of %d floats do not hold a row of %d + %d numbers, or %d columns do not store it", ld, row.n,
             row.r, row.stored);
   return 0;
+}
+int check_queries(int ld, int q_col, int H, int d, int r, const Row& row) {
+  JB_REFUSE(H < 1 || d < 0 || d + r < 1, "latent: %d heads of %d + %d numbers", H, d, r);
+  JB_REFUSE(ld < q_col + H * (d + r), "latent: rows of %d floats do not hold the queries", ld);
+  return check_row(ld, r, row);
 }
 
 }  // namespace
@@ -431,7 +465,7 @@ JB_EXPORT int jb_latent_heads(const float* proj, int ld, int q_col, int H, int d
                               cudaStream_t stream) {
   if (T <= 0) return 0;
   const Row row{c_col, n, r, stored, w, eps, dest, c_cache, rows};
-  if (const int bad = check_row(ld, q_col, H, d, r, row)) return bad;
+  if (const int bad = check_queries(ld, q_col, H, d, r, row)) return bad;
   JB_REFUSE(dp < d + r, "latent_heads: heads of %d numbers cannot be stored in %d columns", d + r, dp);
   const bool vec = ld % 4 == 0 && q_col % 4 == 0 && d % 4 == 0 && r % 8 == 0 && dp % 4 == 0 && aligned16(proj) &&
                    aligned16(q_out) && (table == nullptr || aligned16(table));
@@ -452,6 +486,28 @@ JB_EXPORT int jb_latent_heads(const float* proj, int ld, int q_col, int H, int d
   return (int)e;
 }
 
+// proj: float32 [T, ld] with the queries' latent in columns [0, m); w [m] float32; a_out [T, m], the pages and `rows` in
+// out_dtype; the row's arguments as in jb_latent_heads.  clear: n_clear floats (whole 16-byte vectors) set to zero, or null.
+JB_EXPORT int jb_latent_down(const float* proj, int ld, int m, const float* w, float eps, void* a_out, int out_dtype, int r,
+                             const float* table, const int* positions, int c_col, int n, int stored, const float* row_w,
+                             const int* dest, void* c_cache, void* rows, float* clear, long long n_clear, int T,
+                             cudaStream_t stream) {
+  if (T <= 0) return 0;
+  const Row row{c_col, n, r, stored, row_w, eps, dest, c_cache, rows};
+  JB_REFUSE(m < 1 || ld < m, "latent_down: rows of %d floats do not hold %d numbers", ld, m);
+  if (const int bad = check_row(ld, r, row)) return bad;
+  JB_REFUSE(clear != nullptr && (n_clear % 4 != 0 || !aligned16(clear)), "latent_down: %lld floats to clear", n_clear);
+  const long long vecs = clear != nullptr ? n_clear / 4 : 0;
+  jb::Launch cfg(dim3(T, c_cache != nullptr ? 2 : 1), dim3(256), 0, stream);
+  if (out_dtype == JB_F32)
+    return (int)cudaLaunchKernelEx(&cfg.c, latent_down_kernel<float>, proj, ld, m, w, eps, (float*)a_out, table, positions,
+                                   (float4*)clear, vecs, row);
+  if (out_dtype == JB_BF16)
+    return (int)cudaLaunchKernelEx(&cfg.c, latent_down_kernel<bf16>, proj, ld, m, w, eps, (bf16*)a_out, table, positions,
+                                   (float4*)clear, vecs, row);
+  return JB_ERR_BAD_DTYPE;
+}
+
 // As jb_latent_heads, the queries multiplied into the latents' space: q_out [T, H dp], dp >= n + r; uk: [H d, n]
 // row-major in dtype.
 JB_EXPORT int jb_latent_queries(const float* proj, int ld, int q_col, int H, int d, int r, int n, int dp, const void* uk,
@@ -459,7 +515,7 @@ JB_EXPORT int jb_latent_queries(const float* proj, int ld, int q_col, int H, int
                                 const float* w, float eps, const int* dest, void* c_cache, int T, cudaStream_t stream) {
   if (T <= 0) return 0;
   const Row row{c_col, n, r, stored, w, eps, dest, c_cache, nullptr};
-  if (const int bad = check_row(ld, q_col, H, d, r, row)) return bad;
+  if (const int bad = check_queries(ld, q_col, H, d, r, row)) return bad;
   JB_REFUSE(dp < n + r || n < 1 || d < 1, "latent_queries: %d + %d numbers cannot be stored in %d columns", n, r, dp);
   const int vw = dtype == JB_BF16 ? 8 : 4;
   const bool vec = n % vw == 0 && aligned16(uk);
@@ -490,10 +546,10 @@ JB_EXPORT int jb_latent_queries(const float* proj, int ld, int q_col, int H, int
 }
 
 // uv: [H e, n] row-major; o_rows [T, H n] and out [T, H ep] in dtype; gate: float32 rows of ld_gate numbers, column
-// h e + c for number c of head h (null: no gate).  splits > 0: from part_o and part_ml instead of o_rows.
+// h e + c for number c of head h, or h with gate_per_head (null: no gate).  splits > 0: from part_o and part_ml instead of o_rows.
 JB_EXPORT int jb_latent_values(const void* o_rows, const float* part_o, const float* part_ml, int splits, const void* uv,
-                               const float* gate, int ld_gate, void* out, int dtype, int T, int H, int n, int e, int ep,
-                               cudaStream_t stream) {
+                               const float* gate, int ld_gate, int gate_per_head, void* out, int dtype, int T, int H, int n,
+                               int e, int ep, cudaStream_t stream) {
   if (T <= 0) return 0;
   JB_REFUSE(e < 1 || ep < e || n < 1 || H < 1 || splits < 0, "latent_values: %d values in %d columns from %d numbers", e, ep, n);
   JB_REFUSE(splits > 0 ? (part_o == nullptr || part_ml == nullptr) : o_rows == nullptr, "latent_values: no input");
@@ -518,7 +574,7 @@ JB_EXPORT int jb_latent_values(const void* o_rows, const float* part_o, const fl
     if (smem > 48 * 1024) err = cudaFuncSetAttribute(k, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);    \
     if (err == cudaSuccess)                                                                                         \
       err = cudaLaunchKernelEx(&cfg.c, k, (const T_*)o_rows, part_o, part_ml, splits, (const T_*)uv, gate, ld_gate, \
-                               (T_*)out, T, H, n, e, ep);                                                           \
+                               gate_per_head, (T_*)out, T, H, n, e, ep);                                            \
   } while (0)
   if (dtype == JB_F32) {
     if (vec) JB_GO(float, 4);

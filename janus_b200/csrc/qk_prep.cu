@@ -121,15 +121,18 @@ __global__ void latent_prep_kernel(const float* __restrict__ proj, int ld, int Q
 //   wq (or wk), a weight of size d that all heads share (null: no norm, or with `unit` the division alone, which a
 //   rotation commutes with: it keeps every pair's sum of squares); then the first `rot` dimensions are turned as
 //   above, and q is multiplied by the query temperature 1 + temp_coef ln(floor((p + 1) / temp_every) + 1) of the
-//   token's position p (temp_every 0: none).  q is written [T, H dp], k and v are appended to pages whose rows hold dp numbers (dp >= d, dp >= e; the
-//   extra columns of q are zero, those of the pages are never written).  One block per token, a warp per head.
+//   token's position p (temp_every 0: none).  With `first` (the value heads of the same tokens in another layer) the value
+//   is (1 - mix) v + mix first.  q is written [T, H dp], k is appended to pages whose rows hold dp numbers, v to pages
+//   whose rows hold ep (dp >= d, ep >= e; the extra columns of q are zero, those of the pages are never written).  One
+//   block per token, a warp per head.
 template <typename TO>
 __global__ void head_norm_rope_cache_kernel(const float* __restrict__ proj, int ld, const float* __restrict__ wq,
                                             const float* __restrict__ wk, float eps, const float* __restrict__ table,
                                             int rot, const int* __restrict__ positions, TO* __restrict__ q_out,
                                             const int* __restrict__ dest, TO* __restrict__ k_cache,
-                                            TO* __restrict__ v_cache, int H, int G, int d, int e, int dp, int page_size,
-                                            int write_kv, int unit, float temp_coef, int temp_every) {
+                                            TO* __restrict__ v_cache, int H, int G, int d, int e, int dp, int ep,
+                                            int page_size, int write_kv, int unit, float temp_coef, int temp_every,
+                                            const float* __restrict__ first, int ld_first, float mix) {
   jb::pdl_launch_dependents();
   jb::pdl_wait();
   const int t = blockIdx.x;
@@ -146,11 +149,16 @@ __global__ void head_norm_rope_cache_kernel(const float* __restrict__ proj, int 
   const int n_heads = H + (write_kv ? 2 * G : 0);
   const float temp = temp_every > 0 ? 1.0f + temp_coef * logf((float)((positions[t] + 1) / temp_every) + 1.0f) : 1.0f;
   for (int head = warp; head < n_heads; head += warps) {
-    if (head >= H + G) {                                // a value head: appended as projected
+    if (head >= H + G) {                                // a value head: appended as projected, or mixed
       const int g = head - H - G;
       const float* x = pr + (size_t)(H + G) * d + (size_t)g * e;
-      TO* out = v_cache + ((page * G + g) * page_size + prow) * dp;
-      for (int j = lane; j < e; j += 32) out[j] = jb::from_f32<TO>(x[j]);
+      TO* out = v_cache + ((page * G + g) * page_size + prow) * ep;
+      if (first != nullptr) {
+        const float* y = first + (size_t)t * ld_first + (size_t)g * e;
+        for (int j = lane; j < e; j += 32) out[j] = jb::from_f32<TO>((1.0f - mix) * x[j] + mix * y[j]);
+      } else {
+        for (int j = lane; j < e; j += 32) out[j] = jb::from_f32<TO>(x[j]);
+      }
       continue;
     }
     const bool is_q = head < H;
@@ -236,15 +244,16 @@ JB_EXPORT int jb_latent_prep(const float* proj, int ld, int Q, int r, int rp, co
 }
 
 // proj: float32 [T, ld] = [q: H d | k: G d | v: G e]; wq, wk: float32 [d] or null; table: float32 [positions][rot/2][2]
-// or null; q_out [T, H dp] and the pages (rows of dp) in out_dtype.  write_kv = 0: q only.  unit = 1: heads are divided by
-// their root mean square also without a weight.  temp_every > 0: the query temperature.
+// or null; q_out [T, H dp] and the pages (rows of dp for keys, ep for values) in out_dtype.  write_kv = 0: q only.  unit = 1:
+// heads are divided by their root mean square also without a weight.  temp_every > 0: the query temperature.  first
+// (float32 rows of ld_first numbers, [G e] of each token, or null): values are mixed with it.
 JB_EXPORT int jb_head_norm_rope_cache(const float* proj, int ld, const float* wq, const float* wk, float eps,
                                       const float* table, int rot, const int* positions, void* q_out, int out_dtype,
                                       const int* dest, void* k_cache, void* v_cache, int T, int H, int G, int d, int e,
-                                      int dp, int page_size, int write_kv, int unit, float temp_coef, int temp_every,
-                                      cudaStream_t stream) {
+                                      int dp, int ep, int page_size, int write_kv, int unit, float temp_coef,
+                                      int temp_every, const float* first, int ld_first, float mix, cudaStream_t stream) {
   if (T <= 0) return 0;
-  JB_REFUSE(dp < d || dp < e, "head_norm_rope_cache: heads of %d and %d cannot be stored in %d columns", d, e, dp);
+  JB_REFUSE(dp < d || ep < e, "head_norm_rope_cache: heads of %d and %d cannot be stored in %d and %d columns", d, e, dp, ep);
   JB_REFUSE(rot < 0 || rot > d || (rot & 1), "head_norm_rope_cache: %d rotated dimensions do not fit a head of %d", rot, d);
   JB_REFUSE(ld < H * d + (write_kv ? G * (d + e) : 0), "head_norm_rope_cache: rows of %d floats do not hold the projections", ld);
   const int heads = H + (write_kv ? 2 * G : 0);
@@ -252,12 +261,12 @@ JB_EXPORT int jb_head_norm_rope_cache(const float* proj, int ld, const float* wq
   cudaError_t err;
   if (out_dtype == JB_F32)
     err = cudaLaunchKernelEx(&cfg.c, head_norm_rope_cache_kernel<float>, proj, ld, wq, wk, eps, table, rot, positions,
-                             (float*)q_out, dest, (float*)k_cache, (float*)v_cache, H, G, d, e, dp, page_size, write_kv,
-                             unit, temp_coef, temp_every);
+                             (float*)q_out, dest, (float*)k_cache, (float*)v_cache, H, G, d, e, dp, ep, page_size,
+                             write_kv, unit, temp_coef, temp_every, first, ld_first, mix);
   else if (out_dtype == JB_BF16)
     err = cudaLaunchKernelEx(&cfg.c, head_norm_rope_cache_kernel<bf16>, proj, ld, wq, wk, eps, table, rot, positions,
-                             (bf16*)q_out, dest, (bf16*)k_cache, (bf16*)v_cache, H, G, d, e, dp, page_size, write_kv,
-                             unit, temp_coef, temp_every);
+                             (bf16*)q_out, dest, (bf16*)k_cache, (bf16*)v_cache, H, G, d, e, dp, ep, page_size,
+                             write_kv, unit, temp_coef, temp_every, first, ld_first, mix);
   else
     return JB_ERR_BAD_DTYPE;
   return (int)err;

@@ -8,7 +8,8 @@
 //   out[t] += sum over the chosen e of  Wd_e ( act(Wg_e x) * (Wu_e x) ),  x = s_e h[t]        (the weight is on the input)
 //   or, with the weight on the output,  out[t] += sum over the chosen e of  s_e Wd_e ( act(Wg_e h[t]) * (Wu_e h[t]) ).
 //   Scores may also be the softmax over all experts, and the choice may be limited to the best groups of neighbours; the
-//   choice may rest on scores with a correction per expert added, and the weights may be multiplied by a constant.
+//   choice may rest on scores with a correction per expert added; the weights may be divided by their sum over the token's
+//   experts, and multiplied by a constant.
 //
 // Experts' weights: gate and up [E][F][W], down [E][W][F], row-major, float32 or bfloat16.
 #include <math_constants.h>
@@ -24,10 +25,11 @@ constexpr int MAX_TOP = 16;
 // one warp per token.  softmax = 0: a score is the logit's sigmoid; 1: the softmax over all experts.  groups > 0: the
 // experts form `groups` equal groups of neighbours, a group's score is its largest score, and only experts of the
 // `keep` groups with the largest scores can be chosen (the lower group wins a tie).  correction (per expert, or null):
-// the choice is made by score + correction, the weight stays the score.  Weights are multiplied by `scale`.
+// the choice is made by score + correction, the weight stays the score.  shares = 1: a token's weights are divided by
+// their sum + 1e-20.  Weights are multiplied by `scale`.
 __global__ void route_topk_kernel(const float* __restrict__ logits, int ld, int E, int top, int* __restrict__ sel_e,
                                   float* __restrict__ sel_w, int T, int softmax, int groups, int keep,
-                                  const float* __restrict__ correction, float scale) {
+                                  const float* __restrict__ correction, float scale, int shares) {
   jb::pdl_launch_dependents();
   jb::pdl_wait();
   const int t = blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5), lane = threadIdx.x & 31;
@@ -98,8 +100,13 @@ __global__ void route_topk_kernel(const float* __restrict__ logits, int ld, int 
     picked[k] = arg;
     if (lane == 0) {
       sel_e[(size_t)t * top + k] = arg;
-      sel_w[(size_t)t * top + k] = score(z[arg]) * scale;
+      if (!shares) sel_w[(size_t)t * top + k] = score(z[arg]) * scale;
     }
+  }
+  if (shares && lane == 0) {
+    float sum = 0.0f;
+    for (int k = 0; k < top; ++k) sum += score(z[picked[k]]);
+    for (int k = 0; k < top; ++k) sel_w[(size_t)t * top + k] = score(z[picked[k]]) / (sum + 1e-20f) * scale;
   }
 }
 
@@ -578,7 +585,8 @@ __global__ void expert_scatter_kernel(const float* __restrict__ results, const i
 }  // namespace
 
 JB_EXPORT int jb_route_topk(const float* logits, int ld, int E, int top, int* sel_e, float* sel_w, int T, int softmax,
-                            int groups, int keep, const float* correction, float scale, cudaStream_t stream) {
+                            int groups, int keep, const float* correction, float scale, int shares,
+                            cudaStream_t stream) {
   if (T <= 0) return 0;
   JB_REFUSE(top < 1 || top > MAX_TOP || top > E, "route_topk: %d of %d experts (at most %d a token)", top, E, MAX_TOP);
   JB_REFUSE(groups < 0 || groups > 64 || (groups > 0 && (E % groups != 0 || keep < 1 || keep > groups ||
@@ -586,7 +594,7 @@ JB_EXPORT int jb_route_topk(const float* logits, int ld, int E, int top, int* se
             "route_topk: %d groups of which %d are kept do not fit %d experts and %d a token", groups, keep, E, top);
   jb::Launch cfg(dim3((T + 3) / 4), dim3(128), 0, stream);
   return (int)cudaLaunchKernelEx(&cfg.c, route_topk_kernel, logits, ld, E, top, sel_e, sel_w, T, softmax, groups, keep,
-                                 correction, scale);
+                                 correction, scale, shares);
 }
 
 // h: [T, W] in x_dtype; the experts' weights ([E] of them) in w_dtype; act: float32 scratch [T top, F]; out: float32

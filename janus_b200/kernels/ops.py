@@ -56,22 +56,23 @@ _SIGNATURES = {
     "jb_embed_gather": "pippiippfp", "jb_rmsnorm": "pppifpiiiplp", "jb_residual_add": "ppilp",
     "jb_swiglu": "ppiiip", "jb_swiglu_f32_to_bf16": "piipiip", "jb_zero_f32": "plp",
     "jb_pack_weight_bf16": "piipp", "jb_rope_cache_write": "piipipppppiiiiiiip",
-    "jb_gemm_f32": "pppiiiiiip", "jb_attention_f32": "pppppppiiiiiiiififfp",
+    "jb_gemm_f32": "pppiiiiiip", "jb_attention_f32": "pppppppiiiiiiiififfipppip",
     "jb_gemm_bf16": "pplipiiiiiiplpiffpp", "jb_gemm_bf16_pair": "pplipiiiiiiiffpp",
     "jb_gemm_bf16_pair_grouped": "pplipiiiiipiffpp", "jb_expert_plan": "piiiippppp",
     "jb_gemm_bf16_pair_qkv_rope": "ppliippppppiiiipp",
     "jb_sample": "piipfiffppupppp",
     "jb_attention_bf16_prefill": "pppppppiiiiiiiifp", "jb_attention_bf16_decode": "ppppppppiiiiiiifip",
-    "jb_attention_bf16_decode_fused": "pipppppppppiiiiiiifiip",
-    "jb_attention_bf16_prefill_capped": "pppppppiiiiiiiififfp", "jb_attention_bf16_decode_capped": "ppppppppiiiiiiifiiffp",
+    "jb_attention_bf16_decode_fused": "pipppppppppiiiiiiifiiiffpppipifp",
+    "jb_attention_bf16_prefill_capped": "pppppppiiiiiiiififfpppip",
+    "jb_attention_bf16_decode_capped": "ppppppppiiiiiiifiiffpppip",
     "jb_join_norm": "pppppffpppfipipiiplplp", "jb_head_norm_gate": "ppipipfipiiiip", "jb_sigmoid_gate": "pipiiiiip",
-    "jb_head_norm_rope_cache": "pippfpippipppiiiiiiiiifip",
+    "jb_head_norm_rope_cache": "pippfpippipppiiiiiiiiiifipifp",
     "jb_delta_rule": "piiiipiiippfppllppiiiiip",
-    "jb_route_topk": "piiippiiiipfp", "jb_experts_few_tokens": "pippipppippiiiiffip", "jb_expert_gather": "pippipiip", "jb_experts_few_tokens_tc": "pppipppppiiiiffip",
+    "jb_route_topk": "piiippiiiipfip", "jb_experts_few_tokens": "pippipppippiiiiffip", "jb_expert_gather": "pippipiip", "jb_experts_few_tokens_tc": "pppipppppiiiiffip",
     "jb_expert_scatter": "pppipiip",
     "jb_gla_decay": "piiippfpiip", "jb_exp_gates": "piiippfppllppiip",
     "jb_gated_linear_scan": "piiiifpiippplppiiiiiippp", "jb_scale_rows_sigmoid": "pipiiip",
-    "jb_attention_tc_prefill": "pppppppiiiiiiiiiifpp", "jb_attention_tc_prefill_capped": "pppppppiiiiiiiiiififfpp",
+    "jb_attention_tc_prefill": "pppppppiiiiiiiiiifpp", "jb_attention_tc_prefill_capped": "pppppppiiiiiiiiiiififfpppipp",
     "jb_streams_rmsnorm": "pppipifpiiipplp", "jb_streams_mix": "ppppiiip", "jb_streams_mix_rmsnorm": "pppppipifpiiiplp", "jb_embed_streams": "pippiiippp",
     "jb_lightning_scan": "piiiipppppiiiiiipp", "jb_gated_rmsnorm": "ppipifpiiip",
     "jb_conv_rope_cache": "pipipipppppippppiiiiiiip", "jb_conv_state_update": "pipippiip",
@@ -81,9 +82,10 @@ _SIGNATURES = {
     "jb_sublayer_norm_add": "ppiffppiiiplplp", "jb_qk_norm_rope_cache": "pippppfpippipppiiiiiiip",
     "jb_latent_prep": "piiiipfpippiip", "jb_causal_conv_silu": "piiippipllppppiiiip",
     "jb_mamba2_scan": "piiipipppppllppiiiiiiippp", "jb_gated_group_rmsnorm": "ppipfpiiiip", "jb_pad_rows_bf16": "pipiip", "jb_scale_softcap": "plffp",
-    "jb_gelu": "ppilp", "jb_tanh_norm": "ppppffippfpipiiplplp",
-    "jb_latent_heads": "piiiiiipppiiiipfpppip", "jb_latent_queries": "piiiiiiippppiiipfppip", "jb_latent_values": "pppippipiiiiiip",
-    "jb_gather_rows": "ppiipppiiip", "jb_latent_attention": "ppppppppiiiiiiifiipp", "jb_attention_tc_matrix": "ppppppiiiiiiiifpp",
+    "jb_activate": "ppilip", "jb_tanh_norm": "ppppffippfpipiiplplp",
+    "jb_latent_heads": "piiiiiipppiiiipfpppip", "jb_latent_queries": "piiiiiiippppiiipfppip", "jb_latent_values": "pppippiipiiiiiip",
+    "jb_latent_down": "piipfpiippiiippppplip",
+    "jb_gather_rows": "ppiipppiiip", "jb_latent_attention": "ppppppppiiiiiiifiipp", "jb_attention_tc_matrix": "ppppppiiiiiiiifpipp",
 }
 _CTYPES = {"p": ctypes.c_void_p, "i": ctypes.c_int, "l": ctypes.c_longlong, "u": ctypes.c_ulonglong,
            "f": ctypes.c_float}
@@ -294,13 +296,31 @@ def gemm_f32(x: torch.Tensor, w: torch.Tensor, y: torch.Tensor, accumulate: bool
            "gemm_f32 " + label if label else "gemm_f32")
 
 
+def _head_extras(slopes: Optional[torch.Tensor], sinks: Optional[torch.Tensor], gate: Optional[torch.Tensor], T: int, nh: int):
+    """What the attention kernels take per query head, as their C arguments: `slopes` float32 [nh], a bias that is linear in
+    the distance (slopes[h] (position - key position) is taken off a score); `sinks` float32 [nh], one more term
+    exp(sinks[h]) of the softmax's denominator; `gate` float32 [T, nh] (a view whose rows may be wider), whose sigmoid
+    multiplies a head's output."""
+    if _checks[0]:
+        for t, name in ((slopes, "distance slopes"), (sinks, "sinks")):
+            if t is not None:
+                _need(t, name, torch.float32, (nh,))
+        if gate is not None and (not gate.is_cuda or gate.dtype != torch.float32 or gate.stride(1) != 1
+                                 or tuple(gate.shape) != (T, nh)):
+            raise KernelError("attention: the gate must be float32 columns, one for each head")
+    return _ptr(slopes), _ptr(sinks), _ptr(gate), 0 if gate is None else gate.stride(0)
+
+
 def attention_f32(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor, out: torch.Tensor,
                   block_table: torch.Tensor, token_slot: torch.Tensor, positions: torch.Tensor,
                   nh: int, nkv: int, hd: int, page_size: int, window: int, scale: float, chunk: int = 0,
-                  softcap: float = 0.0, sink: bool = False, vd: Optional[int] = None) -> None:
-    """`vd`: the values are the first vd numbers of the value rows (None: all hd), out is [T, nh vd].  `chunk` > 0: a query sees only the keys of its own chunk of positions, [floor(pos / chunk) chunk, pos];
-    `softcap` > 0: a score s becomes softcap tanh(s / softcap); `sink`: the softmax's denominator has one more
-    term, exp(0), a key of score 0 that has no value."""
+                  softcap: float = 0.0, sink: bool = False, vd: Optional[int] = None,
+                  slopes: Optional[torch.Tensor] = None, sinks: Optional[torch.Tensor] = None,
+                  gate: Optional[torch.Tensor] = None) -> None:
+    """`vd`: the values are the first vd numbers of the value rows (None: all hd), out is [T, nh vd].  `chunk` > 0: a query
+    sees only the keys of its own chunk of positions, [floor(pos / chunk) chunk, pos]; `softcap` > 0: a score s becomes
+    softcap tanh(s / softcap); `sink`: the softmax's denominator has one more term, exp(0), a key of score 0 that has no
+    value.  `slopes`, `sinks`, `gate`: see `_head_extras`."""
     T = q.shape[0]
     vd = hd if vd is None else int(vd)
     _need(q, "attention q", torch.float32, (T, nh * hd))
@@ -313,7 +333,7 @@ def attention_f32(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor,
     _check(_lib("attention_f32").jb_attention_f32(
         _ptr(q), _ptr(k_cache), _ptr(v_cache), _ptr(out), _ptr(block_table), _ptr(token_slot), _ptr(positions),
         T, nh, nkv, hd, vd, page_size, block_table.shape[1], int(window), scale, int(chunk), float(softcap),
-        1.0 if sink else 0.0, _stream()), "attention_f32")
+        1.0 if sink else 0.0, v_cache.shape[-1], *_head_extras(slopes, sinks, gate, T, nh), _stream()), "attention_f32")
 
 
 # -- bfloat16 tensor-core matrix product --------------------------------------------
@@ -603,6 +623,9 @@ _LATENT_DEFINES = _defines_from_env("JANUS_LATENT_DEFINES")
 _ATTN_TC = os.environ.get("JANUS_ATTN_TC", "1") != "0"     # 0: prompts attend on the mma.sync kernel
 
 
+ACTIVATIONS = {"gelu": 0, "relu2": 1}       # of products without a gate, as the kernels number them
+
+
 def gemm_bf16(x: torch.Tensor, w: PackedWeight, y: torch.Tensor, mode: str = "store",
               split_k: Optional[int] = None, pair: Optional[bool] = None, whole_tiles: int = 0,
               label: str = "", gate_limit: float = 0.0, gate_alpha: float = 1.0) -> None:
@@ -611,7 +634,8 @@ def gemm_bf16(x: torch.Tensor, w: PackedWeight, y: torch.Tensor, mode: str = "st
     mode "add":   y[T, N] += result, y float32 (K may be split, sums meet by atomic adds);
     mode "swiglu": w a gated pair (`pack_gated`), y[T, N] = silu(gate) * up in bf16; with gate_limit > 0 the
                    clamped form g sigmoid(gate_alpha g) (u + 1), g = min(gate, limit), u = clamp(up, +-limit);
-    mode "gelu":  y[T, N] = gelu(result) in bf16, gelu(z) = z (1 + erf(z / sqrt 2)) / 2.
+    mode "gelu":  y[T, N] = gelu(result) in bf16, gelu(z) = z (1 + erf(z / sqrt 2)) / 2;
+    mode "relu2": y[T, N] = relu(result)^2 in bf16.
     `split_k`, `pair`, `whole_tiles`: as `gemm_plan_whole` picks them unless given (`whole_tiles`: CTA pairs
     only, the first so many 256 x 256 output tiles of an adding product stay uncut)."""
     T, K = x.shape
@@ -631,8 +655,8 @@ def gemm_bf16(x: torch.Tensor, w: PackedWeight, y: torch.Tensor, mode: str = "st
             raise KernelError(f"gemm {mode}: the weight is a gated pair")
         if mode == "add":
             code, want = 2, torch.float32
-        elif mode == "gelu":
-            code, want = 5, torch.bfloat16
+        elif mode in ACTIVATIONS:
+            code, want = 5 + ACTIVATIONS[mode], torch.bfloat16
         elif mode == "store":
             code, want = (1, torch.float32) if y.dtype == torch.float32 else (0, torch.bfloat16)
         else:
@@ -778,32 +802,42 @@ ATTENTION_MAX_HEAD_DIM = 256      # every attention kernel, float32 and bfloat16
 ATTENTION_BF16_MAX_GROUP = 64     # query heads per kv head of the mma.sync prompt kernel (a row tile holds 64 rows)
 
 
-def _attention_lib(hd: int):
-    if hd % 8 or not 8 <= hd <= 256:
-        raise KernelError(f"attention_bf16: head_dim {hd} is not a multiple of 8 in [8, 256]")
-    return _lib("attention_bf16", int(hd), lambda h: dict({"JB_HEAD_DIM": h}, **_ATTN_DEFINES))
+def _attention_lib(hd: int, vd: Optional[int] = None):
+    """The build for head size `hd` and value size `vd` (None: the same)."""
+    vd = hd if vd is None else vd
+    for size in (hd, vd):
+        if size % 8 or not 8 <= size <= 256:
+            raise KernelError(f"attention_bf16: head_dim {size} is not a multiple of 8 in [8, 256]")
+    if vd == hd:
+        return _lib("attention_bf16", int(hd), lambda h: dict({"JB_HEAD_DIM": h}, **_ATTN_DEFINES))
+    return _lib("attention_bf16", (int(hd), int(vd)),
+                lambda k: dict({"JB_HEAD_DIM": k[0], "JB_VALUE_DIM": k[1]}, **_ATTN_DEFINES))
 
 
 def attention_bf16_prefill(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor, out: torch.Tensor,
                            block_table: torch.Tensor, q_start: torch.Tensor, kv_len: torch.Tensor,
                            n_seqs: int, max_q_len: int, nh: int, nkv: int, hd: int, page_size: int,
                            window: int, scale: float, chunk: int = 0, softcap: float = 0.0,
-                           sink: bool = False) -> None:
+                           sink: bool = False, vd: Optional[int] = None, slopes: Optional[torch.Tensor] = None,
+                           sinks: Optional[torch.Tensor] = None, gate: Optional[torch.Tensor] = None) -> None:
     """Causal attention of each sequence's new tokens (the last q_len positions of
-    its kv_len) over its cached keys.  `chunk`, `softcap`, `sink`: as in `attention_f32`."""
+    its kv_len) over its cached keys.  `chunk`, `softcap`, `sink`, `slopes`, `sinks`, `gate`: as in `attention_f32`; `vd`:
+    the size of a value (None: hd), out is [T, nh vd]."""
     T = q.shape[0]
+    vd = hd if vd is None else int(vd)
     _need(q, "attention q", torch.bfloat16, (T, nh * hd))
-    _need(out, "attention out", torch.bfloat16, (T, nh * hd))
+    _need(out, "attention out", torch.bfloat16, (T, nh * vd))
     _need(k_cache, "k cache", torch.bfloat16)
     _need(v_cache, "v cache", torch.bfloat16)
     _need(block_table, "block table", torch.int32)
     _need(q_start, "q_start", torch.int32, (n_seqs + 1,))
     _need(kv_len, "kv_len", torch.int32, (n_seqs,))
-    if chunk or softcap or sink:
-        _check(_attention_lib(hd).jb_attention_bf16_prefill_capped(
+    if chunk or softcap or sink or vd != hd or slopes is not None or sinks is not None or gate is not None:
+        _check(_attention_lib(hd, vd).jb_attention_bf16_prefill_capped(
             _ptr(q), _ptr(k_cache), _ptr(v_cache), _ptr(out), _ptr(block_table), _ptr(q_start), _ptr(kv_len),
             n_seqs, max_q_len, nh, nkv, hd, page_size, block_table.shape[1], int(window), scale, int(chunk),
-            float(softcap), 1.0 if sink else 0.0, _stream()), "attention_bf16_prefill")
+            float(softcap), 1.0 if sink else 0.0, *_head_extras(slopes, sinks, gate, T, nh), _stream()),
+            "attention_bf16_prefill")
         return
     _check(_attention_lib(hd).jb_attention_bf16_prefill(
         _ptr(q), _ptr(k_cache), _ptr(v_cache), _ptr(out), _ptr(block_table), _ptr(q_start), _ptr(kv_len),
@@ -822,15 +856,16 @@ _SPLIT_SHARED_SM = 0.2              # a CTA that shares its SM with another walk
 _SPLIT_CHOICES = (1, 2, 3, 4, 6, 8, 12, 16, 24, 32)
 
 
-def _decode_ctas_per_sm(head_dim: int, ctas: int, pages_per_cta: int) -> int:
+def _decode_ctas_per_sm(head_dim: int, ctas: int, pages_per_cta: int, value_dim: Optional[int] = None) -> int:
     """CTAs of the decode kernel that share an SM: its ring of pages is picked at the launch (in step with
     `decode_stages_for` of csrc/attention_bf16.cu): three pages for large heads (two CTAs an SM at head size
     128); small heads take two pages when there are more CTAs than fit at once (five an SM at head size 64),
     five pages for few CTAs of many pages (two an SM), else three (three an SM)."""
-    ld = (head_dim + 15) // 16 * 16 + 8
+    value_dim = head_dim if value_dim is None else value_dim
+    ld, ld_v = ((d + 15) // 16 * 16 + 8 for d in (head_dim, value_dim))
 
     def fit(stages: int) -> int:
-        smem = 18 * ld * 2 + max(2 * stages * 64 * ld * 2, (4 * 16 * (head_dim + 8) + 128) * 4)
+        smem = (17 * ld + ld_v) * 2 + max(stages * 64 * (ld + ld_v) * 2, (4 * 16 * (value_dim + 8) + 128) * 4)
         return max(1, min(16, 228 * 1024 // (smem + 1024)))
 
     if head_dim > 64:
@@ -844,7 +879,8 @@ def _decode_ctas_per_sm(head_dim: int, ctas: int, pages_per_cta: int) -> int:
 
 
 @functools.lru_cache(maxsize=4096)
-def decode_splits_for(n_seqs: int, nkv_blocks: int, max_kv_len: int, page_size: int, head_dim: int = 128) -> int:
+def decode_splits_for(n_seqs: int, nkv_blocks: int, max_kv_len: int, page_size: int, head_dim: int = 128,
+                      value_dim: Optional[int] = None) -> int:
     """Splits of the key range per (sequence, kv head), from an estimate of the kernel's time for each count.
 
     A launch is `n_seqs * nkv_blocks * splits` CTAs of about `pages / splits` pages each; as many CTAs as fit the
@@ -860,14 +896,14 @@ def decode_splits_for(n_seqs: int, nkv_blocks: int, max_kv_len: int, page_size: 
     base = max(1, n_seqs * nkv_blocks)
     sms = SM_COUNT_TARGET // 2
     page_us = _SPLIT_PAGE_US[64 if head_dim <= 64 else 128]
-    page_bytes = page_size * head_dim * 2 * 2
+    page_bytes = page_size * (head_dim + (head_dim if value_dim is None else value_dim)) * 2
     best = (float("inf"), 1)
     for splits in _SPLIT_CHOICES:
         if splits > 1 and splits > max(1, cap_pages // 2):
             break
         per = (pages + splits - 1) // splits
         ctas = base * splits
-        places = sms * _decode_ctas_per_sm(head_dim, ctas, per)
+        places = sms * _decode_ctas_per_sm(head_dim, ctas, per, value_dim)
         alone = _SPLIT_CTA_US + per * page_us
 
         def wave(n: int) -> float:      # n CTAs at once: on how many SMs, at the memory's rate or a CTA's own pace
@@ -888,35 +924,41 @@ def attention_bf16_decode(q: Optional[torch.Tensor], k_cache: torch.Tensor, v_ca
                           page_size: int, window: int, scale: float, workspace, max_kv_len: int,
                           n_splits: Optional[int] = None, qkv: Optional[torch.Tensor] = None,
                           cos_sin: Optional[torch.Tensor] = None, dest: Optional[torch.Tensor] = None,
-                          write_kv: bool = True, chunk: int = 0, softcap: float = 0.0, sink: bool = False) -> None:
-    """One new token per sequence (its last position) over its cached keys.  `chunk`, `softcap`, `sink` (with `q`
-    only): as in `attention_f32`.
+                          write_kv: bool = True, chunk: int = 0, softcap: float = 0.0, sink: bool = False,
+                          vd: Optional[int] = None, slopes: Optional[torch.Tensor] = None,
+                          sinks: Optional[torch.Tensor] = None, gate: Optional[torch.Tensor] = None,
+                          first: Optional[torch.Tensor] = None, mix: float = 0.0) -> None:
+    """One new token per sequence (its last position) over its cached keys.  `chunk`, `softcap`, `sink`, `slopes`, `sinks`,
+    `gate`: as in `attention_f32`; `vd`: the size of a value (None: hd), out is [B, nh vd].
 
     Either `q` (rotated bf16 queries; the cache already holds the new token), or `qkv`: the
-    projection's float32 output [B, (nh + 2 nkv) hd] (or [B, nh hd] with write_kv False), which the
-    kernel rotates with `cos_sin` (None: no rotation), appends to the cache at rows `dest` and uses."""
+    projection's float32 output [B, nh hd + nkv (hd + vd)] (or [B, nh hd] with write_kv False; rows may be wider), which the
+    kernel rotates with `cos_sin` (None: no rotation), appends to the cache at rows `dest` and uses.  With `first`
+    (float32 [B, nkv vd], rows may be wider) the values are (1 - mix) v + mix first."""
     B = out.shape[0]
-    _need(out, "attention out", torch.bfloat16, (B, nh * hd))
+    vd = hd if vd is None else int(vd)
+    _need(out, "attention out", torch.bfloat16, (B, nh * vd))
     _need(k_cache, "k cache", torch.bfloat16)
     _need(v_cache, "v cache", torch.bfloat16)
     _need(block_table, "block table", torch.int32)
     _need(kv_len, "kv_len", torch.int32, (B,))
     n_rb = (nh // nkv + 15) // 16
     if n_splits is None:
-        n_splits = decode_splits_for(B, nkv * n_rb, max_kv_len, page_size, hd)
+        n_splits = decode_splits_for(B, nkv * n_rb, max_kv_len, page_size, hd, None if vd == hd else vd)
     part_o = part_ml = None
     if n_splits > 1:
-        part_o = workspace.get("attn_part_o", (B * nh * n_splits * hd,), torch.float32)
+        part_o = workspace.get("attn_part_o", (B * nh * n_splits * vd,), torch.float32)
         part_ml = workspace.get("attn_part_ml", (B * nh * n_splits * 2,), torch.float32)
-    lib = _attention_lib(hd)
+    lib = _attention_lib(hd, vd)
     kernels = 2 if n_splits > 1 else 1
+    extras = _head_extras(slopes, sinks, gate, B, nh)
     if qkv is None:
         _need(q, "attention q", torch.bfloat16, (B, nh * hd))
-        if chunk or softcap or sink:
+        if chunk or softcap or sink or slopes is not None or sinks is not None or gate is not None:
             _check(lib.jb_attention_bf16_decode_capped(
                 _ptr(q), _ptr(k_cache), _ptr(v_cache), _ptr(out), _ptr(part_o), _ptr(part_ml), _ptr(block_table),
                 _ptr(kv_len), B, nh, nkv, hd, page_size, block_table.shape[1], int(window), scale,
-                int(n_splits), int(chunk), float(softcap), 1.0 if sink else 0.0, _stream()),
+                int(n_splits), int(chunk), float(softcap), 1.0 if sink else 0.0, *extras, _stream()),
                 "attention_bf16_decode", kernels=kernels)
             return
         _check(lib.jb_attention_bf16_decode(
@@ -924,10 +966,8 @@ def attention_bf16_decode(q: Optional[torch.Tensor], k_cache: torch.Tensor, v_ca
             _ptr(kv_len), B, nh, nkv, hd, page_size, block_table.shape[1], int(window), scale,
             int(n_splits), _stream()), "attention_bf16_decode", kernels=kernels)
         return
-    if chunk or softcap or sink:
-        raise KernelError("attention decode: the kernel that rotates and appends takes no chunked mask, cap or sink")
     _need(qkv, "qkv", torch.float32)
-    width = (nh + 2 * nkv) * hd if write_kv else nh * hd
+    width = nh * hd + nkv * (hd + vd) if write_kv else nh * hd
     if qkv.shape[0] != B or qkv.shape[1] < width:
         raise KernelError(f"attention decode: qkv shape {tuple(qkv.shape)} does not hold {B} rows of width {width}")
     if cos_sin is not None:
@@ -936,10 +976,13 @@ def attention_bf16_decode(q: Optional[torch.Tensor], k_cache: torch.Tensor, v_ca
             raise KernelError(f"attention decode: table shape {tuple(cos_sin.shape)} does not fit head_dim {hd}")
     if write_kv:
         _need(dest, "cache rows", torch.int32, (B,))
+    if first is not None and (first.dtype != torch.float32 or first.stride(1) != 1 or tuple(first.shape) != (B, nkv * vd)):
+        raise KernelError("attention decode: the values to mix in must be float32 columns, a value a kv head")
     _check(lib.jb_attention_bf16_decode_fused(
         _ptr(qkv), qkv.shape[1], _ptr(cos_sin), _ptr(dest), _ptr(k_cache), _ptr(v_cache), _ptr(out), _ptr(part_o),
         _ptr(part_ml), _ptr(block_table), _ptr(kv_len), B, nh, nkv, hd, page_size, block_table.shape[1], int(window),
-        scale, int(n_splits), int(write_kv), _stream()), "attention_bf16_decode_fused", kernels=kernels)
+        scale, int(n_splits), int(write_kv), int(chunk), float(softcap), 1.0 if sink else 0.0, *extras, _ptr(first),
+        0 if first is None else first.stride(0), float(mix), _stream()), "attention_bf16_decode_fused", kernels=kernels)
 
 
 # -- tcgen05 prefill attention (head sizes up to 256 in steps of 8, up to 128 query heads per kv head) -----
@@ -961,25 +1004,28 @@ def attention_tc_prefill(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.
                          block_table: torch.Tensor, q_start: torch.Tensor, kv_len: torch.Tensor,
                          n_seqs: int, max_q_len: int, nh: int, nkv: int, hd: int, page_size: int,
                          window: int, scale: float, chunk: int = 0, softcap: float = 0.0,
-                         sink: bool = False) -> None:
-    """As attention_bf16_prefill, on the tcgen05 tensor cores.  `chunk`, `softcap`, `sink`: as in `attention_f32`."""
+                         sink: bool = False, vd: Optional[int] = None, slopes: Optional[torch.Tensor] = None,
+                         sinks: Optional[torch.Tensor] = None, gate: Optional[torch.Tensor] = None) -> None:
+    """As attention_bf16_prefill, on the tcgen05 tensor cores (a value holds at most hd numbers)."""
     T = q.shape[0]
+    vd = hd if vd is None else int(vd)
     _need(q, "attention q", torch.bfloat16, (T, nh * hd))
-    _need(out, "attention out", torch.bfloat16, (T, nh * hd))
+    _need(out, "attention out", torch.bfloat16, (T, nh * vd))
     _need(k_cache, "k cache", torch.bfloat16)
     _need(v_cache, "v cache", torch.bfloat16)
     _need(block_table, "block table", torch.int32)
     _need(q_start, "q_start", torch.int32, (n_seqs + 1,))
     _need(kv_len, "kv_len", torch.int32, (n_seqs,))
-    if tuple(k_cache.shape[1:]) != (nkv, page_size, hd) or k_cache.shape != v_cache.shape:
-        raise KernelError(f"attention_tc: cache shape {tuple(k_cache.shape)} does not fit [pages, {nkv}, {page_size}, {hd}]")
+    if tuple(k_cache.shape[1:]) != (nkv, page_size, hd) or tuple(v_cache.shape) != (*k_cache.shape[:3], vd):
+        raise KernelError(f"attention_tc: cache shapes {tuple(k_cache.shape)}, {tuple(v_cache.shape)} do not fit "
+                          f"[pages, {nkv}, {page_size}, {hd}] and values of {vd}")
     lib = _lib("attention_tc", _attention_tc_row(hd), lambda h: dict({"JB_HEAD_DIM": h}, **_ATTN_TC_DEFINES))
-    if chunk or softcap or sink:
+    if chunk or softcap or sink or vd != hd or slopes is not None or sinks is not None or gate is not None:
         _check(lib.jb_attention_tc_prefill_capped(
             _ptr(q), _ptr(k_cache), _ptr(v_cache), _ptr(out), _ptr(block_table), _ptr(q_start), _ptr(kv_len),
-            T, k_cache.shape[0], n_seqs, max_q_len, nh, nkv, hd, page_size, block_table.shape[1], int(window),
-            scale, int(chunk), float(softcap), 1.0 if sink else 0.0, _ptr(kernel_status(q.device)), _stream()),
-            "attention_tc_prefill")
+            T, k_cache.shape[0], n_seqs, max_q_len, nh, nkv, hd, vd, page_size, block_table.shape[1], int(window),
+            scale, int(chunk), float(softcap), 1.0 if sink else 0.0, *_head_extras(slopes, sinks, gate, T, nh),
+            _ptr(kernel_status(q.device)), _stream()), "attention_tc_prefill")
         return
     _check(lib.jb_attention_tc_prefill(
         _ptr(q), _ptr(k_cache), _ptr(v_cache), _ptr(out), _ptr(block_table), _ptr(q_start), _ptr(kv_len),
@@ -989,10 +1035,11 @@ def attention_tc_prefill(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.
 
 def attention_tc_matrix(q: torch.Tensor, kv: torch.Tensor, out: torch.Tensor, kv_start: torch.Tensor,
                         q_start: torch.Tensor, kv_len: torch.Tensor, n_seqs: int, max_q_len: int, nh: int, hd: int,
-                        vd: int, max_kv_len: int, scale: float) -> None:
+                        vd: int, max_kv_len: int, scale: float, gate: Optional[torch.Tensor] = None) -> None:
     """Causal attention on the tcgen05 tensor cores of each sequence's new tokens (the last q_len positions of its
     kv_len) over keys and values that lie in one matrix, kv [rows, nh hd + nh vd] bfloat16: a key and a value per query
-    head, the key of position p of sequence s in row kv_start[s] + p.  q [T, nh hd], out [T, nh vd]."""
+    head, the key of position p of sequence s in row kv_start[s] + p.  q [T, nh hd], out [T, nh vd].  `gate`: as in
+    `attention_f32`."""
     T = q.shape[0]
     _need(q, "attention q", torch.bfloat16, (T, nh * hd))
     _need(out, "attention out", torch.bfloat16, (T, nh * vd))
@@ -1006,7 +1053,8 @@ def attention_tc_matrix(q: torch.Tensor, kv: torch.Tensor, out: torch.Tensor, kv
     lib = _lib("attention_tc", _attention_tc_row(hd), lambda h: dict({"JB_HEAD_DIM": h}, **_ATTN_TC_DEFINES))
     _check(lib.jb_attention_tc_matrix(
         _ptr(q), _ptr(kv), _ptr(out), _ptr(kv_start), _ptr(q_start), _ptr(kv_len), T, kv.shape[0], n_seqs, max_q_len, nh,
-        hd, vd, int(max_kv_len), float(scale), _ptr(kernel_status(q.device)), _stream()), "attention_tc_matrix")
+        hd, vd, int(max_kv_len), float(scale), *_head_extras(None, None, gate, T, nh)[2:], _ptr(kernel_status(q.device)),
+        _stream()), "attention_tc_matrix")
 
 
 # -- several residual streams per token -------------------------------------------------
@@ -1228,11 +1276,12 @@ def diff_attention_prefill(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torc
         eps, out_scale, _stream()), "diff_attention_prefill")
 
 
-def gelu(x: torch.Tensor, out: torch.Tensor) -> None:
-    """out = gelu(x) elementwise, gelu(z) = z (1 + erf(z / sqrt 2)) / 2; float32 in, out's dtype out."""
-    _need(x, "activation in", torch.float32)
+def activate(x: torch.Tensor, out: torch.Tensor, activation: str) -> None:
+    """out = act(x) for a float32 x, out in its dtype: "gelu", z (1 + erf(z / sqrt 2)) / 2, or "relu2", relu(z)^2."""
+    _need(x, "activation input", torch.float32)
     _need(out, "activation out", None, tuple(x.shape))
-    _check(_lib("elementwise").jb_gelu(_ptr(x), _ptr(out), dtype_code(out.dtype), x.numel(), _stream()), "gelu")
+    _check(_lib("elementwise").jb_activate(_ptr(x), _ptr(out), dtype_code(out.dtype), x.numel(), ACTIVATIONS[activation],
+                                           _stream()), activation)
 
 
 # -- a gated activation with clamped branches; scale and soft cap -------------------------------
@@ -1535,13 +1584,15 @@ def head_norm_rope_cache(proj: torch.Tensor, wq: Optional[torch.Tensor], wk: Opt
                          dest: Optional[torch.Tensor], k_cache: Optional[torch.Tensor], v_cache: Optional[torch.Tensor],
                          heads: int, kv_heads: int, dim: int, vdim: int, stored_dim: int, page_size: int,
                          write_kv: bool = True, unit_norm: bool = False, temp_coef: float = 0.0,
-                         temp_every: int = 0) -> None:
+                         temp_every: int = 0, stored_vdim: Optional[int] = None, first: Optional[torch.Tensor] = None,
+                         mix: float = 0.0) -> None:
     """proj float32 [T, >= heads dim + kv_heads (dim + vdim)]: q, k and v as projected.  Every head of q and k is
     divided by its own root mean square and multiplied by the weight [dim] that the heads share (None: no norm), its
     first `rot` dimensions are turned by the table's cos and sin at the token's position; q is written
-    [T, heads stored_dim], k and v are appended to pages whose rows hold stored_dim numbers.  `unit_norm`: without
-    weights the heads are still divided by their root mean square.  `temp_every` > 0: q is multiplied by
-    1 + temp_coef ln(floor((position + 1) / temp_every) + 1)."""
+    [T, heads stored_dim], k and v are appended to pages whose rows hold stored_dim (v: stored_vdim, None: the same)
+    numbers.  `unit_norm`: without weights the heads are still divided by their root mean square.  `temp_every` > 0: q is
+    multiplied by 1 + temp_coef ln(floor((position + 1) / temp_every) + 1).  With `first` (float32 [T, kv_heads vdim],
+    rows may be wider) the values are (1 - mix) v + mix first."""
     T = q_out.shape[0]
     _need(proj, "projections", torch.float32)
     if proj.shape[0] != T:
@@ -1559,11 +1610,14 @@ def head_norm_rope_cache(proj: torch.Tensor, wq: Optional[torch.Tensor], wk: Opt
         _need(dest, "cache rows", torch.int32, (T,))
         _need(k_cache, "key pages", q_out.dtype)
         _need(v_cache, "value pages", q_out.dtype)
+    if first is not None and (first.dtype != torch.float32 or first.stride(1) != 1 or tuple(first.shape) != (T, kv_heads * vdim)):
+        raise KernelError("head_norm_rope_cache: the values to mix in must be float32 columns, a value a kv head")
     _check(_lib("qk_prep").jb_head_norm_rope_cache(
         _ptr(proj), proj.shape[1], _ptr(wq), _ptr(wk), float(eps), _ptr(table) if rot > 0 else None, int(rot),
         _ptr(positions), _ptr(q_out), dtype_code(q_out.dtype), _ptr(dest) if write_kv else None,
         _ptr(k_cache) if write_kv else None, _ptr(v_cache) if write_kv else None, T, heads, kv_heads, dim, vdim,
-        stored_dim, page_size, int(write_kv), int(bool(unit_norm)), float(temp_coef), int(temp_every), _stream()),
+        stored_dim, stored_dim if stored_vdim is None else int(stored_vdim), page_size, int(write_kv), int(bool(unit_norm)),
+        float(temp_coef), int(temp_every), _ptr(first), 0 if first is None else first.stride(0), float(mix), _stream()),
         "head_norm_rope_cache")
 
 
@@ -1596,13 +1650,13 @@ def delta_rule(conv: torch.Tensor, q_col: int, k_col: int, v_col: int, raw: torc
 # -- experts of which a token uses a few ---------------------------------------------------------------------------
 def route_topk(logits: torch.Tensor, top: int, sel_e: torch.Tensor, sel_w: torch.Tensor, softmax: bool = False,
                groups: int = 0, keep: int = 0, experts: Optional[int] = None,
-               correction: Optional[torch.Tensor] = None, scale: float = 1.0) -> None:
+               correction: Optional[torch.Tensor] = None, scale: float = 1.0, shares: bool = False) -> None:
     """Per row of the float32 logits [T, >= E] (the first `experts` columns; None: all): the `top` largest (the lower
     index wins a tie) as indices (int32 [T, top]) and their scores as weights (float32 [T, top]): the logits' sigmoids,
     or with `softmax` the softmax over all experts.  `groups` > 0: the experts form that many equal groups of
     neighbours, and only experts of the `keep` groups whose best expert scores highest can be chosen.  `correction`
-    (float32 [experts]): the choice goes by score + correction, the weights stay the scores.  The weights are multiplied
-    by `scale`."""
+    (float32 [experts]): the choice goes by score + correction, the weights stay the scores.  `shares`: a token's weights
+    are divided by their sum + 1e-20.  The weights are multiplied by `scale`."""
     T, ld = logits.shape
     E = ld if experts is None else int(experts)
     _need(logits, "router logits", torch.float32)
@@ -1613,8 +1667,8 @@ def route_topk(logits: torch.Tensor, top: int, sel_e: torch.Tensor, sel_w: torch
     if E > ld:
         raise KernelError(f"route_topk: {E} experts in rows of {ld} logits")
     _check(_lib("routed").jb_route_topk(_ptr(logits), ld, E, int(top), _ptr(sel_e), _ptr(sel_w), T,
-                                        int(bool(softmax)), int(groups), int(keep), _ptr(correction), float(scale), _stream()),
-           "route_topk")
+                                        int(bool(softmax)), int(groups), int(keep), _ptr(correction), float(scale), int(bool(shares)),
+                                        _stream()), "route_topk")
 
 
 def experts_few_tokens(h: torch.Tensor, sel_e: torch.Tensor, sel_w: torch.Tensor, w_gate: torch.Tensor,
@@ -1880,6 +1934,27 @@ def latent_heads(proj: torch.Tensor, q_col: int, heads: int, d: int, r: int, sto
         _ptr(rows), T, _stream()), "latent_heads")
 
 
+def latent_down(proj: torch.Tensor, m: int, weight: torch.Tensor, eps: float, a_out: torch.Tensor, r: int,
+                table: Optional[torch.Tensor], positions: torch.Tensor, row: Optional[tuple] = None,
+                rows: Optional[torch.Tensor] = None, clear: Optional[torch.Tensor] = None) -> None:
+    """a_out [T, m] = x / rms(x) * weight with x the first m columns of proj (eps inside the root): the queries' latent, for
+    the product that makes the queries.  `row`, `rows`: the token's own row, as in `latent_heads`.  `clear`: a float32
+    scratch tensor (whole 16-byte vectors) that the same launch sets to zero."""
+    T = a_out.shape[0]
+    _latent_row(proj, a_out, 0, r, table, positions, row)
+    _need(a_out, "queries' latent", None, (T, m))
+    _need(weight, "queries' latent norm weight", torch.float32, (m,))
+    col, n, stored, row_weight, _, dest, pages = row if row is not None else (0, 0, 0, None, 0.0, None, None)
+    if rows is not None:
+        _need(rows, "rows", a_out.dtype, (T, stored))
+    if clear is not None:
+        _need(clear, "buffer to clear", torch.float32)
+    _check(_lib("latent").jb_latent_down(
+        _ptr(proj), proj.shape[1], int(m), _ptr(weight), float(eps), _ptr(a_out), dtype_code(a_out.dtype), int(r),
+        _ptr(table) if r else None, _ptr(positions), int(col), n, stored, _ptr(row_weight), _ptr(dest), _ptr(pages),
+        _ptr(rows), _ptr(clear), 0 if clear is None else clear.numel(), T, _stream()), "latent_down")
+
+
 def latent_queries(proj: torch.Tensor, q_col: int, heads: int, d: int, r: int, n: int, stored: int, uk: torch.Tensor,
                    table: Optional[torch.Tensor], positions: torch.Tensor, q_out: torch.Tensor,
                    row: Optional[tuple] = None) -> None:
@@ -1898,8 +1973,8 @@ def latent_queries(proj: torch.Tensor, q_col: int, heads: int, d: int, r: int, n
 
 def latent_values(o: Optional[torch.Tensor], partial: Optional[tuple], uv: torch.Tensor, gate: Optional[torch.Tensor],
                   out: torch.Tensor, heads: int, n: int, e: int, stored: int) -> None:
-    """out[t, h, :e] = uv_h o[t, h] (times sigmoid(gate[t, h, :]), float32 columns), zeros up to `stored`; uv
-    [heads e, n].  o [T, heads n], or `partial` = (sums, maxima, splits): what the splits of `latent_attention` left."""
+    """out[t, h, :e] = uv_h o[t, h] (times the sigmoid of the gate, float32 columns: one for each value number,
+    [T, heads e], or one per head, [T, heads]), zeros up to `stored`; uv [heads e, n].  o [T, heads n], or `partial` = (sums, maxima, splits): what the splits of `latent_attention` left."""
     T = out.shape[0]
     _need(out, "head outputs", None, (T, heads * stored))
     _need(uv, "values' matrix", out.dtype, (heads * e, n))
@@ -1911,11 +1986,13 @@ def latent_values(o: Optional[torch.Tensor], partial: Optional[tuple], uv: torch
         _need(maxima, "partial maxima", torch.float32)
         if sums.numel() < T * heads * splits * n or maxima.numel() < T * heads * splits * 2:
             raise KernelError("latent_values: the partial sums are too small")
-    if gate is not None and (gate.dtype != torch.float32 or gate.stride(1) != 1 or tuple(gate.shape) != (T, heads * e)):
-        raise KernelError("latent_values: the gate must be float32 columns, one for each number of the heads")
+    if gate is not None and (gate.dtype != torch.float32 or gate.stride(1) != 1
+                             or tuple(gate.shape) not in ((T, heads * e), (T, heads))):
+        raise KernelError("latent_values: the gate must be float32 columns, one for each number of the heads or for each head")
+    per_head = gate is not None and gate.shape[1] == heads and e > 1
     _check(_lib("latent").jb_latent_values(
         _ptr(o), _ptr(sums), _ptr(maxima), int(splits), _ptr(uv), _ptr(gate), gate.stride(0) if gate is not None else 0,
-        _ptr(out), dtype_code(out.dtype), T, heads, n, e, stored, _stream()), "latent_values")
+        int(per_head), _ptr(out), dtype_code(out.dtype), T, heads, n, e, stored, _stream()), "latent_values")
 
 
 def gather_rows(pages: torch.Tensor, block_table: torch.Tensor, kv_len: torch.Tensor, start: torch.Tensor,

@@ -404,7 +404,7 @@ def test_products_with_the_exact_gelu_in_their_epilogue_and_behind_them():
     g = torch.Generator().manual_seed(2)
     x = torch.linspace(-6.0, 6.0, 4099)
     out = torch.empty(4099, device="cuda")
-    ops.gelu(x.cuda(), out)
+    ops.activate(x.cuda(), out, "gelu")
     assert float((out.cpu().to(P.DT) - P.gelu(x.to(P.DT))).abs().max()) < 1e-6
     for dtype in (torch.float32, torch.bfloat16):
         for T, W, F in ((3, 64, 200), (70, 96, 136), (300, 256, 512), (20, 36, 50), (9, 256, 20000)):
