@@ -3,8 +3,8 @@ keys and values for each place of the schedule that writes some, and a
 fixed-size state area per slot for mixers that keep state.
 
 Places with the same needs (KVSpec) form a group; a group owns its page pool,
-its storage and, per slot, its list of pages.  A group with a window gives back
-pages whose keys every later query has left behind.  Slots and pages are reused
+its storage and, per slot, its list of pages.  A group with a window or with chunks
+gives back pages whose keys every later query has left behind.  Slots and pages are reused
 by later sequences without being cleared: every read is bounded by the
 sequence's length.  State areas are zeroed when a slot is taken.
 
@@ -42,7 +42,7 @@ class KVGroup:
         # a place whose values are its keys hands out the key pages for both
         self.v: Dict[int, torch.Tensor] = self.k if spec.values_are_keys else {
             p: torch.zeros(v_shape, dtype=dtype, device=device) for p in self.places}
-        # pages[slot][i] holds keys [i*PAGE, (i+1)*PAGE); -1 once a window has passed it
+        # pages[slot][i] holds keys [i*PAGE, (i+1)*PAGE); -1 once a window or a chunk has passed it
         self.pages: List[List[int]] = [[] for _ in range(n_slots)]
 
     def reserve(self, slot: int, new_length: int) -> None:
@@ -58,12 +58,13 @@ class KVGroup:
     def release_passed(self, slot: int, length: int) -> None:
         """With a window w, the next query (position `length`) reads keys
         > length - w; pages wholly at or below that are given back, except the
-        pages that hold one of the first `keep_first` keys, which every query reads."""
-        w = self.spec.window
-        if w <= 0:
+        pages that hold one of the first `keep_first` keys, which every query reads.
+        With chunks the next query reads from the first position of its chunk on."""
+        if not self.spec.gives_back_pages:
             return
         pages = self.pages[slot]
-        first_needed = max(0, length - w + 1)
+        w, chunk = self.spec.window, self.spec.chunk
+        first_needed = max(0, length - w + 1 if w > 0 else 0, length // chunk * chunk if chunk > 0 else 0)
         kept_pages = (self.spec.keep_first + PAGE_SIZE - 1) // PAGE_SIZE
         for i in range(kept_pages, min(len(pages), first_needed // PAGE_SIZE)):
             if pages[i] >= 0:

@@ -79,6 +79,8 @@ class StepContext:
         # (connection, y) of a sublayer whose write into the residual streams is still to come: an arrangement
         # may leave it for the next read to do in the same launch; the model flushes it after the last layer
         self.pending_write = None
+        # tensors of this step that one part leaves for parts of later places (by a name the parts agree on)
+        self.shared: Dict[str, torch.Tensor] = {}
 
     def cache_view(self, place: int) -> CacheView:
         cache = self.cache
@@ -498,11 +500,11 @@ class _DecodeGraph:
                                                   for s, n in zip(slots, lens)]
             table = h[o[8 + 2 * gi]:o[8 + 2 * gi] + B * cap].reshape(B, cap)
             sigs = self.row_sig[k][gi]
-            windowed = g.spec.window > 0
+            windowed = g.spec.gives_back_pages
             for i, s in enumerate(slots):
                 row = pages[s]
                 sig = (s, cache.epochs[s], len(row))
-                if windowed or sigs[i] != sig:       # a window group's rows lose pages as they pass
+                if windowed or sigs[i] != sig:       # such a group's rows lose pages as they pass
                     table[i, :len(row)] = row
                     table[i, len(row):] = -1
                     sigs[i] = sig

@@ -1,1 +1,1 @@
-from . import buludra, forisun, llama, mugedra, ramolix, zivitar  # noqa: F401  (registers Buludra, Forisun, LlamaForCausalLM, Mugedra, Ramolix and Zivitar)
+from . import buludra, forisun, llama, mibezen, mugedra, ramolix, zivitar  # noqa: F401  (registers Buludra, Forisun, LlamaForCausalLM, Mibezen, Mugedra, Ramolix and Zivitar)

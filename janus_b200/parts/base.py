@@ -45,7 +45,8 @@ import torch
 class KVSpec:
     """Keys and values per token.  window = 0 keeps every key; window = w keeps
     the last w keys (the query's own position included), and besides them the
-    first `keep_first` keys of the sequence.  Values may differ from keys in
+    first `keep_first` keys of the sequence.  chunk = c > 0 keeps the keys of the
+    current chunk of c positions (a query sees no key of an earlier one).  Values may differ from keys in
     their number of heads and their size (0: as the keys).  `values_are_keys`:
     the place stores one row per token that serves as key and as value (a
     latent vector that both are made from): no pages of their own for values."""
@@ -56,6 +57,12 @@ class KVSpec:
     n_value_heads: int = 0
     value_dim: int = 0
     values_are_keys: bool = False
+    chunk: int = 0
+
+    @property
+    def gives_back_pages(self) -> bool:
+        """Whether pages of a live sequence may be given back before it ends."""
+        return self.window > 0 or self.chunk > 0
 
     @property
     def v_heads(self) -> int:

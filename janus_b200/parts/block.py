@@ -39,8 +39,15 @@ class PreNormBlock:
             self.mixer.forward(x, residual, ctx, cache_view, writes_cache)
         if self.feed_forward is None:
             return
-        self.feed_forward_norm.forward(residual, x)
-        self.feed_forward.forward(x, residual, ctx)
+        # so may a feed-forward
+        wants = getattr(self.feed_forward, "scratch_to_clear", None)
+        scratch = wants(ctx, residual.shape[0]) if wants is not None else None
+        if scratch is not None:
+            self.feed_forward_norm.forward(residual, x, clear=scratch)
+            self.feed_forward.forward(x, residual, ctx, scratch_cleared=True)
+        else:
+            self.feed_forward_norm.forward(residual, x)
+            self.feed_forward.forward(x, residual, ctx)
 
 
 register_part("arrangement", "pre_norm", PreNormBlock)

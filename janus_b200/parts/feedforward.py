@@ -6,7 +6,7 @@ from __future__ import annotations
 import torch
 
 from .base import FeedForward, register_part
-from .linear import GatedLinear, GeluLinear, Linear
+from .linear import ActivatedLinear, GatedLinear, Linear
 
 
 class SwiGLUFeedForward(FeedForward):
@@ -94,14 +94,16 @@ class GeluGLUFeedForward(FeedForward):
         self.down.forward_add(act, residual)
 
 
-class GeluFeedForward(FeedForward):
-    """down( gelu(up(x)) ), gelu(z) = z (1 + erf(z / sqrt 2)) / 2, added into the residual stream: no gate."""
+class ActivatedFeedForward(FeedForward):
+    """down( act(up(x)) ), added into the residual stream: no gate.  act is "gelu", z (1 + erf(z / sqrt 2)) / 2, or "relu2",
+    relu(z)^2."""
 
-    def __init__(self, hidden_size: int, intermediate_size: int,
+    def __init__(self, hidden_size: int, intermediate_size: int, activation: str,
                  dtype: torch.dtype = torch.bfloat16, device: torch.device = torch.device("cuda")):
         self.hidden_size, self.intermediate_size = hidden_size, intermediate_size
         self.dtype, self.device = dtype, device
-        self.up = GeluLinear(hidden_size, intermediate_size, dtype, device, name="up", pad_width=True)
+        self.up = ActivatedLinear(hidden_size, intermediate_size, dtype, device, name="up", pad_width=True,
+                                  activation=activation)
         self.down = Linear(intermediate_size, hidden_size, dtype, device, name="down", pad_width=True)
 
     def weight_shapes(self):
@@ -121,7 +123,20 @@ class GeluFeedForward(FeedForward):
         self.down.forward_add(act, residual)
 
 
+class GeluFeedForward(ActivatedFeedForward):
+    def __init__(self, hidden_size: int, intermediate_size: int,
+                 dtype: torch.dtype = torch.bfloat16, device: torch.device = torch.device("cuda")):
+        super().__init__(hidden_size, intermediate_size, "gelu", dtype, device)
+
+
+class SquaredReluFeedForward(ActivatedFeedForward):
+    def __init__(self, hidden_size: int, intermediate_size: int,
+                 dtype: torch.dtype = torch.bfloat16, device: torch.device = torch.device("cuda")):
+        super().__init__(hidden_size, intermediate_size, "relu2", dtype, device)
+
+
 register_part("feed_forward", "swiglu", SwiGLUFeedForward)
+register_part("feed_forward", "relu2_mlp", SquaredReluFeedForward)
 register_part("feed_forward", "gelu_mlp", GeluFeedForward)
 register_part("feed_forward", "gelu_glu", GeluGLUFeedForward)
 register_part("feed_forward", "clamped_glu", ClampedGLUFeedForward)

@@ -138,6 +138,13 @@ class RotaryLatentAttention(Mixer):
     The cache holds [c | p] per token, whatever the heads; a layer without a latent of its own (`own_latent` False)
     reads the rows that an earlier place cached, with its own Wuk, Wuv, queries, gate and output.
 
+    Options: `q_rank` m: the queries have a latent of their own, q = Wuq (rms_norm(Wdq h)) with a weight of size m
+    (one launch norms it, finishes the token's row and clears what the product behind it adds into).  `gate` "head": one
+    number per head, sigmoid(Wg h)_h times the head's output; the attention over heads applies it to its sums and the values'
+    kernel to its own.  `pairs` "neighbours": the rotation turns the pair (2 i, 2 i + 1); the rows of the matrices that make
+    the rotated numbers, of the queries and of p alike, are put in the order of the halves when they are loaded, which
+    leaves every score as it is.
+
     Two ways through a step of the bfloat16 engine, picked by an estimate of the time:
     - in the latents' space (single tokens, short portions behind long histories): the query passes Wuk on its side,
       q' = [Wuk^T q | turned q], a cached row is the key of all heads and its first n numbers their value
@@ -151,13 +158,18 @@ class RotaryLatentAttention(Mixer):
     prompt_way: Optional[str] = None         # "heads" or "latents": every prompt step goes that way (for measurements)
 
     def __init__(self, hidden_size: int, num_heads: int, dim: int, rot_dim: int, vdim: int, rank: int, scale: float,
-                 eps: float, position: Optional[PartSpec] = None, gate: bool = True, own_latent: bool = True,
+                 eps: float, position: Optional[PartSpec] = None, gate=True, own_latent: bool = True,
+                 q_rank: Optional[int] = None, pairs: str = "halves",
                  dtype: torch.dtype = torch.bfloat16, device: torch.device = torch.device("cuda")):
         self.hidden_size, self.nh, self.dim, self.rot, self.vdim, self.rank = (
             int(hidden_size), int(num_heads), int(dim), int(rot_dim), int(vdim), int(rank))
+        if gate not in (True, False, "head") or pairs not in ("halves", "neighbours"):
+            raise ValueError(f"a gate is True, False or 'head', pairs are 'halves' or 'neighbours', got {gate!r}, {pairs!r}")
+        self.q_rank = None if q_rank is None else int(q_rank)
+        self.head_gate, self.neighbours = gate == "head", pairs == "neighbours"
         if self.rot % 2:
             raise ValueError(f"{self.rot} rotated numbers do not form pairs")
-        self.scale, self.eps, self.gate, self.own_latent = float(scale), float(eps), bool(gate), bool(own_latent)
+        self.scale, self.eps, self.gate, self.own_latent = float(scale), float(eps), gate is not False, bool(own_latent)
         self.dtype, self.device = dtype, device
         self.row = stored_head_size(self.rank + self.rot, dtype)          # numbers a cached row is stored with
         if self.row > ops.LATENT_MAX_ROW or (dtype == torch.bfloat16
@@ -165,10 +177,16 @@ class RotaryLatentAttention(Mixer):
             raise ValueError(f"cached rows of {self.rank} + {self.rot} numbers are not supported (at most "
                              f"{ops.LATENT_MAX_ROW})")
         self.position = shared_part("position", position, dtype, device) if position is not None else None
-        # columns of the stacked projection: queries, gate, then the row (a view of the first columns serves places
-        # that read another place's rows)
+        # columns of the stacked projection: queries (or their latent), gate, then the row (a view of the first columns
+        # serves places that read another place's rows)
         self.q_width, self.o_width = self.nh * (self.dim + self.rot), self.nh * self.vdim
-        self.row_col = self.q_width + (self.o_width if self.gate else 0)
+        self.gate_width = (self.nh if self.head_gate else self.o_width) if self.gate else 0
+        self.gate_col = self.q_width if self.q_rank is None else self.q_rank
+        self.row_col = self.gate_col + self.gate_width
+        self.uq: Optional[Linear] = None
+        self.q_norm_weight: Optional[torch.Tensor] = None
+        if self.q_rank is not None:
+            self.uq = Linear(self.q_rank, self.q_width, dtype, device, name="uq", pad_width=True)
         self.proj = Linear(hidden_size, self.row_col + (self.rank + self.rot if self.own_latent else 0), dtype, device,
                            name="q_g_dkv" if self.own_latent else "q_g", pad_width=True)
         self.q_only: Optional[Linear] = None
@@ -192,22 +210,42 @@ class RotaryLatentAttention(Mixer):
 
     def weight_shapes(self):
         H, W, n = self.nh, self.hidden_size, self.rank
-        shapes = {"q": ((self.q_width, W), "normal"), "uk": ((H * self.dim, n), "normal"),
-                  "uv": ((H * self.vdim, n), "normal"), "o": ((W, self.o_width), "normal")}
+        shapes = {"uk": ((H * self.dim, n), "normal"), "uv": ((H * self.vdim, n), "normal"),
+                  "o": ((W, self.o_width), "normal")}
+        if self.q_rank is None:
+            shapes["q"] = ((self.q_width, W), "normal")
+        else:
+            m = self.q_rank
+            shapes.update(dq=((m, W), "normal"), dq_norm=((m,), "ones"), uq=((self.q_width, m), "normal"))
         if self.gate:
-            shapes["g"] = ((self.o_width, W), "normal")
+            shapes["g"] = ((self.gate_width, W), "normal")
         if self.own_latent:
             shapes.update(dkv=((n + self.rot, W), "normal"), dkv_norm=((n,), "ones"))
         return shapes
 
-    def load(self, q, uk, uv, o, g=None, dkv=None, dkv_norm=None) -> None:
+    def _halves(self, w: torch.Tensor, heads: int, before: int) -> torch.Tensor:
+        """Rows of `heads` groups of before + r: with pairs of neighbours, the last r of a group as the even ones, then the
+        odd ones."""
+        if not self.neighbours or self.rot == 0:
+            return w
+        group = before + self.rot
+        order = list(range(before)) + [before + i for s in (0, 1) for i in range(s, self.rot, 2)]
+        return w.reshape(heads, group, w.shape[1])[:, order].reshape(heads * group, w.shape[1])
+
+    def load(self, uk, uv, o, q=None, dq=None, dq_norm=None, uq=None, g=None, dkv=None, dkv_norm=None) -> None:
         H, d, r, e, n, W = self.nh, self.dim, self.rot, self.vdim, self.rank, self.hidden_size
         for name, t, shape in (("uk", uk, (H * d, n)), ("uv", uv, (H * e, n)), ("o", o, (W, H * e))):
             if tuple(t.shape) != shape:
                 raise ValueError(f"weight '{name}' of shape {tuple(t.shape)} does not fit {shape}")
         if self.own_latent and (dkv is None or dkv_norm is None or tuple(dkv_norm.shape) != (n,)):
             raise ValueError("a latent attention layer with a latent of its own needs 'dkv' and 'dkv_norm'")
-        self.proj.load([q] + ([g] if self.gate else []) + ([dkv] if self.own_latent else []))
+        if self.q_rank is not None:
+            if tuple(dq_norm.shape) != (self.q_rank,):
+                raise ValueError(f"weight 'dq_norm' of shape {tuple(dq_norm.shape)} does not fit ({self.q_rank},)")
+            self.q_norm_weight = dq_norm.to(device=self.device, dtype=torch.float32).contiguous()
+            self.uq.load([self._halves(uq, H, d)])
+        self.proj.load([self._halves(q, H, d) if self.q_rank is None else dq] + ([g] if self.gate else [])
+                       + ([self._halves(dkv, 1, n)] if self.own_latent else []))
         self.q_only = self.proj.first_rows(self.row_col)
         if self.own_latent:
             self.norm_weight = dkv_norm.to(device=self.device, dtype=torch.float32).contiguous()
@@ -264,15 +302,34 @@ class RotaryLatentAttention(Mixer):
         proj = ws.get("latent_proj", (T, lin.out_features), torch.float32)
         lin.forward(x, proj, y_is_zero=scratch_cleared)
         table = self.position.fused_rotary_table() if self.position is not None else None
-        gate = proj[:, self.q_width:self.row_col] if self.gate else None
+        gate = proj[:, self.gate_col:self.row_col] if self.gate else None
         row = (self.row_col, self.rank, self.row, self.norm_weight, self.eps, group.dest_rows, cache_view.k) \
             if writes_cache else None
         out = ws.get("latent_heads_out", (T, self.nh * self.v_stored), self.dtype)
-        if self._as_heads(ctx):
-            self._attend_as_heads(proj, table, row, gate, out, ctx, cache_view)
+        as_heads = self._as_heads(ctx)
+        # sequences that begin with this step: their rows are the step's own, in the step's order
+        rows = None
+        if as_heads:
+            rows = ws.get("latent_rows", (ctx.kv_total, self.row), self.dtype)
+        fresh = as_heads and row is not None and ctx.kv_total == T
+        if self.q_rank is not None:
+            # the queries by way of their latent; the same launch finishes the token's row
+            proj = self._queries_from_latent(proj, table, row, rows if fresh else None, ctx)
+            row = None
+        if as_heads:
+            self._attend_as_heads(proj, table, row, rows, fresh, gate, out, ctx, cache_view)
         else:
             self._attend_latents(proj, table, row, gate, out, ctx, cache_view)
         self.o.forward_add(out, residual)
+
+    def _queries_from_latent(self, proj, table, row, rows, ctx) -> torch.Tensor:
+        T, ws = proj.shape[0], ctx.workspace
+        q = ws.get("latent_q_proj", (T, self.q_width), torch.float32)
+        clear = q if self.uq.meets_by_adds(T, torch.float32) and q.numel() % 4 == 0 else None
+        a = ws.get("latent_q_down", (T, self.q_rank), self.dtype)
+        ops.latent_down(proj, self.q_rank, self.q_norm_weight, self.eps, a, self.rot, table, ctx.positions, row, rows, clear)
+        self.uq.forward(a, q, y_is_zero=clear is not None)
+        return q
 
     def _attend_latents(self, proj, table, row, gate, out, ctx, cache_view) -> None:
         T, ws, group = proj.shape[0], ctx.workspace, cache_view.group
@@ -290,21 +347,19 @@ class RotaryLatentAttention(Mixer):
                                            ctx.max_kv_len_bound)
         ops.latent_values(o, partial, self.uv, gate, out, H, n, self.vdim, self.v_stored)
 
-    def _attend_as_heads(self, proj, table, row, gate, out, ctx, cache_view) -> None:
+    def _attend_as_heads(self, proj, table, row, rows, fresh, gate, out, ctx, cache_view) -> None:
         T, ws, group = proj.shape[0], ctx.workspace, cache_view.group
         H, ks, vs = self.nh, self.k_stored, self.v_stored
         q = ws.get("latent_q_heads", (T, H * ks), self.dtype)
-        rows = ws.get("latent_rows", (ctx.kv_total, self.row), self.dtype)
-        # sequences that begin with this step: their rows are the step's own, in the step's order
-        fresh = row is not None and ctx.kv_total == T
-        ops.latent_heads(proj, 0, H, self.dim, self.rot, ks, table, ctx.positions, q, row, rows if fresh else None)
+        ops.latent_heads(proj, 0, H, self.dim, self.rot, ks, table, ctx.positions, q, row,
+                         rows if fresh and row is not None else None)
         if not fresh:
             ops.gather_rows(cache_view.k, group.block_table, ctx.kv_len, ctx.kv_start, rows, group.page_size, ctx.n_seqs)
         kv = ws.get("latent_kv", (ctx.kv_total, self.heads_width), self.dtype)
         self.to_heads.forward(rows, kv)
         ops.attention_tc_matrix(q, kv, out, ctx.kv_start, ctx.q_start, ctx.kv_len, ctx.n_seqs, ctx.max_q_len, H, ks, vs,
-                                ctx.max_kv_len_bound, self.scale)
-        if gate is not None:
+                                ctx.max_kv_len_bound, self.scale, gate=gate if self.head_gate else None)
+        if gate is not None and not self.head_gate:
             ops.sigmoid_gate(out, gate, H, self.vdim, vs)
 
 

@@ -136,9 +136,17 @@ class Linear:
             ops.gemm_bf16(x, self.weight, residual, mode="add", label=self.name)
 
 
-class GeluLinear(Linear):
-    """out = gelu(x W^T) in the engine dtype, gelu(z) = z (1 + erf(z / sqrt 2)) / 2: in the product's own epilogue, or,
-    where a decode-sized step would leave SMs idle with K uncut (and in float32), behind a plain product."""
+class ActivatedLinear(Linear):
+    """out = act(x W^T) in the engine dtype (`activation`: a name of `ops.ACTIVATIONS`, "gelu" or "relu2"): in the product's
+    own epilogue, or, where a decode-sized step would leave SMs idle with K uncut (and in float32), behind a plain
+    product."""
+
+    def __init__(self, in_features: int, out_features: int, dtype: torch.dtype, device: torch.device, name: str = "",
+                 pad_width: bool = False, activation: str = "gelu"):
+        super().__init__(in_features, out_features, dtype, device, name, pad_width)
+        if activation not in ops.ACTIVATIONS:
+            raise ValueError(f"activation '{activation}' is not one of {sorted(ops.ACTIVATIONS)}")
+        self.activation = activation
 
     def _behind(self, T: int) -> bool:
         return T <= 64 and self.meets_by_adds(T, torch.float32)
@@ -147,19 +155,19 @@ class GeluLinear(Linear):
         """The plain product's float32 result, if slices of K are added into it: the launch before may clear it."""
         if not self._behind(tokens):
             return None
-        z = ctx.workspace.get("gelu_in", (tokens, self.out_features), torch.float32)
+        z = ctx.workspace.get("activation_in", (tokens, self.out_features), torch.float32)
         return z if z.numel() % 4 == 0 else None
 
     def forward(self, x: torch.Tensor, out: torch.Tensor, ctx, scratch_cleared: bool = False) -> None:
         T = x.shape[0]
         if self.dtype == torch.float32 or self._behind(T):
-            z = ctx.workspace.get("gelu_in", (T, self.out_features), torch.float32)
+            z = ctx.workspace.get("activation_in", (T, self.out_features), torch.float32)
             super().forward(x, z, y_is_zero=scratch_cleared)
-            ops.gelu(z, out)
+            ops.activate(z, out, self.activation)
             return
         if self._padded is not None:
             x = self._padded.rows(x)
-        ops.gemm_bf16(x, self.weight, out, mode="gelu", label=self.name)
+        ops.gemm_bf16(x, self.weight, out, mode=self.activation, label=self.name)
 
 
 class GatedLinear:

@@ -1,7 +1,8 @@
 """RMSNorm: y = x / sqrt(mean(x^2) + eps) * gamma, statistics in float32
 (crates/janus-engine/src/compute/shaders/activations.wgsl:81-133).  The weight
 keeps the dtype it was stored in (the reference keeps 1-D tensors in f32,
-crates/janus-engine/src/compute/engine.rs:448-470)."""
+crates/janus-engine/src/compute/engine.rs:448-470), or is float32 when a constant is added to it (`weight_offset`: designs
+that store a norm's weight around zero)."""
 from __future__ import annotations
 
 from typing import Optional
@@ -13,19 +14,22 @@ from .base import Norm, register_part
 
 
 class RMSNorm(Norm):
-    def __init__(self, width: int, eps: float, dtype: torch.dtype, device: torch.device):
-        self.width, self.eps = int(width), float(eps)
+    def __init__(self, width: int, eps: float, weight_offset: float = 0.0, dtype: torch.dtype = torch.bfloat16,
+                 device: torch.device = torch.device("cuda")):
+        self.width, self.eps, self.offset = int(width), float(eps), float(weight_offset)
         self.dtype, self.device = dtype, device
         self.gamma: Optional[torch.Tensor] = None
 
     def weight_shapes(self):
-        return {"gamma": ((self.width,), "ones")}
+        return {"gamma": ((self.width,), "normal" if self.offset else "ones")}
 
     def load(self, gamma: torch.Tensor) -> None:
         if tuple(gamma.shape) != (self.width,):
             raise ValueError(f"norm weight of shape {tuple(gamma.shape)} does not fit ({self.width},)")
-        if self.dtype == torch.float32:
+        if self.dtype == torch.float32 or self.offset:
             gamma = gamma.to(torch.float32)
+        if self.offset:
+            gamma = gamma + self.offset
         self.gamma = gamma.to(self.device).contiguous()
 
     def forward(self, x: torch.Tensor, out: torch.Tensor, row_index: Optional[torch.Tensor] = None,

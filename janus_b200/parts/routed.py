@@ -24,7 +24,8 @@ feed-forward of that inner width runs for every token and is added; with `shared
 sigmoid(wsg . h), one number per token (the gate's row rides along in the router's product, and because the last
 product is linear the gate multiplies the rows that product reads).  `correction`: a number per expert is added to the
 scores that the choice goes by, and to nothing else (a token's experts are those with the largest corrected scores, its
-weights their scores without the correction).  `scale`: the weights are multiplied by it.
+weights their scores without the correction).  `shares`: a token's weights are divided by their sum (+ 1e-20).  `scale`:
+the weights are multiplied by it.
 """
 from __future__ import annotations
 
@@ -44,14 +45,14 @@ MAX_STREAM_PAIRS = 65535  # pairs of one launch of the streaming kernels
 class RoutedExperts(FeedForward):
     def __init__(self, hidden_size: int, intermediate_size: int, experts: int, top: int, score: str = "sigmoid",
                  groups: Optional[tuple] = None, weight_on: str = "input", shared_size: Optional[int] = None,
-                 shared_gate: bool = False, correction: bool = False, scale: float = 1.0,
+                 shared_gate: bool = False, correction: bool = False, scale: float = 1.0, shares: bool = False,
                  dtype: torch.dtype = torch.bfloat16, device: torch.device = torch.device("cuda")):
         if not 1 <= top <= experts:
             raise ValueError(f"a token uses {top} of {experts} experts")
         if score not in ("sigmoid", "softmax") or weight_on not in ("input", "output"):
             raise ValueError(f"scores are 'sigmoid' or 'softmax' and weigh the 'input' or the 'output', got "
                              f"{score!r}, {weight_on!r}")
-        self.has_correction, self.weight_scale = bool(correction), float(scale)
+        self.has_correction, self.weight_scale, self.shares = bool(correction), float(scale), bool(shares)
         self.correction: Optional[torch.Tensor] = None
         self.softmax, self.weight_on_output = score == "softmax", weight_on == "output"
         self.groups, self.keep = (0, 0) if groups is None else (int(groups[0]), int(groups[1]))
@@ -156,7 +157,8 @@ class RoutedExperts(FeedForward):
         sel_e = ws.get("router_experts", (T, self.top), torch.int32)
         sel_w = ws.get("router_weights", (T, self.top), torch.float32)
         ops.route_topk(logits, self.top, sel_e, sel_w, softmax=self.softmax, groups=self.groups, keep=self.keep,
-                       experts=self.experts, correction=self.correction, scale=self.weight_scale)
+                       experts=self.experts, correction=self.correction, scale=self.weight_scale,
+                       shares=self.shares)
         pairs = T * self.top
         if self.dtype == torch.bfloat16 and not ctx.is_decode and pairs > FEW_PAIRS:
             if self.grouped:
