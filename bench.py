@@ -21,7 +21,7 @@ the same weights (`checked`).
 
 Other modes (one JSON line per item, none of them the headline): --kernels,
 --prompt-lengths, --workload 1b|13b, --deterministic, --plan-check, --cpu-baseline, --float32, --design
-(the Zivitar design, or with --design-model ramolix | mugedra | buludra | forisun another one, beside the Llama decoder at equal layer
+(the Zivitar design, or with --design-model ramolix | mugedra | buludra | forisun | mibezen another one, beside the Llama decoder at equal layer
 sizes: prompt and decode throughput, a step's kernels).
 """
 import argparse
@@ -738,18 +738,34 @@ def forisun_config(width, ff, heads, kv_heads, window, vocab):
                         dict(type=kind, mixer=mixer, mlp=experts), dict(type=kind, mixer=dict(mixer, kv_from=2), mlp=experts)])
 
 
+def mibezen_config(width, ff, heads, kv_heads, window, vocab):
+    """Four layers at the size's width: latent attention as in `forisun_config`, its queries by way of a latent of three
+    quarters of the width, and grouped-query attention with a distance bias, learned sinks and mixed values in chunks of four
+    times the size's window (heads of 128, values of 128; a decode step at 2,048 keys sees them all), each kind once with a dense feed-forward (squared relu, one matrix up) and
+    once with eight experts of half the size's feed-forward of which a token uses two."""
+    latent = dict(heads=heads, dim=128, rot_dim=64, vdim=128, q_rank=width * 3 // 4, kv_rank=512, scale=192 ** -0.5,
+                  rot=dict(dims=64, base=10000.0, scaling=dict(factor=4.0, original=4096, fast=32.0, slow=1.0)))
+    chunked = dict(heads=heads, kv_heads=kv_heads, dim=128, vdim=128, scale=128 ** -0.5, mask=dict(size=4 * window), v_mix=True)
+    dense = dict(kind="dense", ff=ff)
+    experts = dict(kind="moe", expert=dict(ff=ff // 2), router=dict(experts=8, top=2))
+    return dict(architecture="Mibezen", vocab=vocab, width=width, norm=dict(eps=1e-6), logit_softcap=15.0,
+                layers=[dict(type="latent_attention", mixer=latent, mlp=dense), dict(type="attention", mixer=chunked, mlp=experts),
+                        dict(type="attention", mixer=chunked, mlp=dense), dict(type="latent_attention", mixer=latent, mlp=experts)])
+
+
 DESIGNS = {"zivitar": zivitar_config, "ramolix": ramolix_config, "mugedra": mugedra_config, "buludra": buludra_config,
-           "forisun": forisun_config}
+           "forisun": forisun_config, "mibezen": mibezen_config}
 # what a design is measured beside: the Llama decoder, or the design whose kernels are most like its own
 BESIDE = {"zivitar": ("llama",), "ramolix": ("llama",), "mugedra": ("ramolix", "llama"), "buludra": ("mugedra", "llama"),
-          "forisun": ("ramolix", "buludra", "llama")}
+          "forisun": ("ramolix", "buludra", "llama"), "mibezen": ("forisun", "mugedra", "llama")}
 
 
 def run_design(which, design="zivitar"):
-    """A design (Zivitar, Ramolix, Mugedra, Buludra or Forisun) beside the Llama decoder, Mugedra also beside Ramolix, whose
+    """A design (Zivitar, Ramolix, Mugedra, Buludra, Forisun or Mibezen) beside the Llama decoder, Mugedra also beside Ramolix, whose
     mixers (a recurrence behind a short convolution, attention over part of the keys) are most like its own, and
     Buludra also beside Mugedra (two mixers side by side, a recurrence with a matrix state, experts), and Forisun also
-    beside Ramolix (latent attention, norms on the sublayers' outputs) and Buludra (experts weighted on their outputs), at
+    beside Ramolix (latent attention, norms on the sublayers' outputs) and Buludra (experts weighted on their outputs),
+    and Mibezen beside Forisun (latent attention, experts) and Mugedra (attention in chunks, experts), at
     equal layer sizes (random weights, four layer runs):
     prompt steps and decode steps timed on the device, and each step's kernels one by one (`Model.profile`).  One
     JSON line per (size, model)."""

@@ -201,14 +201,15 @@ def one_expert(w, pre: str, h: torch.Tensor) -> torch.Tensor:
     return (silu(h @ w[pre + "gate"].T) * (h @ w[pre + "up"].T)) @ w[pre + "down"].T
 
 
-MARGINS: List[float] = []       # the smallest gap of scores that a choice of experts rested on, per call
+MARGINS: List[float] = []       # the smallest gap of router logits that a choice of experts rested on, per call
 
 
 def choose_experts(z: torch.Tensor, top: int):
     """z [T, E] router logits: the `top` largest of the softmax over all experts, as shares of their own sum."""
     ranked, order = torch.softmax(z, dim=-1).sort(dim=-1, descending=True)
     if top < z.shape[1]:
-        MARGINS.append(float((ranked[:, top - 1] - ranked[:, top]).min()))
+        by_size = z.sort(dim=-1, descending=True).values
+        MARGINS.append(float((by_size[:, top - 1] - by_size[:, top]).min()))
     best = ranked[:, :top]
     return order[:, :top], best / (best.sum(dim=-1, keepdim=True) + 1e-20)
 
