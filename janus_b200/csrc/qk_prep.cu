@@ -190,6 +190,62 @@ __global__ void head_norm_rope_cache_kernel(const float* __restrict__ proj, int 
   }
 }
 
+template <typename TO>
+__device__ __forceinline__ void store4(TO* p, const float4& v) {
+  if constexpr (sizeof(TO) == 4) {
+    *reinterpret_cast<float4*>(p) = v;
+  } else {
+    const __nv_bfloat162 lo = __floats2bfloat162_rn(v.x, v.y), hi = __floats2bfloat162_rn(v.z, v.w);
+    uint2 u;
+    u.x = *reinterpret_cast<const uint32_t*>(&lo);
+    u.y = *reinterpret_cast<const uint32_t*>(&hi);
+    *reinterpret_cast<uint2*>(p) = u;
+  }
+}
+
+// head_norm_rope_cache without norm, rotation and temperature: four numbers a thread (d, e, dp, ep and ld, ld_first whole
+// groups of four at aligned addresses).  One block per token.
+template <typename TO>
+__global__ void __launch_bounds__(256) head_copy_cache_kernel(const float* __restrict__ proj, int ld, TO* __restrict__ q_out,
+                                                              const int* __restrict__ dest, TO* __restrict__ k_cache,
+                                                              TO* __restrict__ v_cache, int H, int G, int d, int e, int dp,
+                                                              int ep, int page_size, int write_kv,
+                                                              const float* __restrict__ first, int ld_first, float mix) {
+  jb::pdl_launch_dependents();
+  jb::pdl_wait();
+  const int t = blockIdx.x;
+  const float* pr = proj + (size_t)t * ld;
+  size_t page = 0;
+  int prow = 0;
+  if (write_kv) {
+    page = (size_t)(dest[t] / page_size);
+    prow = dest[t] % page_size;
+  }
+  const int per_q = dp >> 2, per_k = d >> 2, per_v = e >> 2;
+  const int nq = H * per_q, nk = write_kv ? G * per_k : 0, nv = write_kv ? G * per_v : 0;
+#pragma unroll 4
+  for (int i = threadIdx.x; i < nq + nk + nv; i += 256) {
+    if (i < nq) {
+      const int h = i / per_q, j = (i - h * per_q) << 2;
+      const float4 x = j < d ? *reinterpret_cast<const float4*>(pr + (size_t)h * d + j) : make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+      store4(q_out + ((size_t)t * H + h) * dp + j, x);
+    } else if (i < nq + nk) {
+      const int c = i - nq, g = c / per_k, j = (c - g * per_k) << 2;
+      store4(k_cache + ((page * G + g) * page_size + prow) * dp + j,
+             *reinterpret_cast<const float4*>(pr + (size_t)(H + g) * d + j));
+    } else {
+      const int c = i - nq - nk, g = c / per_v, j = (c - g * per_v) << 2;
+      float4 x = *reinterpret_cast<const float4*>(pr + (size_t)(H + G) * d + (size_t)g * e + j);
+      if (first != nullptr) {
+        const float4 y = *reinterpret_cast<const float4*>(first + (size_t)t * ld_first + (size_t)g * e + j);
+        const float own = 1.0f - mix;
+        x = make_float4(own * x.x + mix * y.x, own * x.y + mix * y.y, own * x.z + mix * y.z, own * x.w + mix * y.w);
+      }
+      store4(v_cache + ((page * G + g) * page_size + prow) * ep + j, x);
+    }
+  }
+}
+
 }  // namespace
 
 // proj: float32 [T, ld]; bq [H d], bk [G d] (either may be null), wq [H d], wk [G d] float32; table: float32
@@ -256,6 +312,17 @@ JB_EXPORT int jb_head_norm_rope_cache(const float* proj, int ld, const float* wq
   JB_REFUSE(dp < d || ep < e, "head_norm_rope_cache: heads of %d and %d cannot be stored in %d and %d columns", d, e, dp, ep);
   JB_REFUSE(rot < 0 || rot > d || (rot & 1), "head_norm_rope_cache: %d rotated dimensions do not fit a head of %d", rot, d);
   JB_REFUSE(ld < H * d + (write_kv ? G * (d + e) : 0), "head_norm_rope_cache: rows of %d floats do not hold the projections", ld);
+  const bool plain = wq == nullptr && wk == nullptr && !unit && temp_every == 0 && (table == nullptr || rot == 0);
+  if (plain && ((d | e | dp | ep | ld | ld_first) & 3) == 0 &&
+      (((uintptr_t)proj | (uintptr_t)q_out | (uintptr_t)k_cache | (uintptr_t)v_cache | (uintptr_t)first) & 15) == 0) {
+    jb::Launch pcfg(dim3(T), dim3(256), 0, stream);
+    if (out_dtype == JB_F32)
+      return (int)cudaLaunchKernelEx(&pcfg.c, head_copy_cache_kernel<float>, proj, ld, (float*)q_out, dest, (float*)k_cache,
+                                     (float*)v_cache, H, G, d, e, dp, ep, page_size, write_kv, first, ld_first, mix);
+    if (out_dtype == JB_BF16)
+      return (int)cudaLaunchKernelEx(&pcfg.c, head_copy_cache_kernel<bf16>, proj, ld, (bf16*)q_out, dest, (bf16*)k_cache,
+                                     (bf16*)v_cache, H, G, d, e, dp, ep, page_size, write_kv, first, ld_first, mix);
+  }
   const int heads = H + (write_kv ? 2 * G : 0);
   jb::Launch cfg(dim3(T), dim3(heads >= 8 ? 256 : heads >= 4 ? 128 : 64), 0, stream);
   cudaError_t err;

@@ -70,10 +70,10 @@ CFG_A = config(160, 64, [
 # values that happen to be 1 or equal: one head, all sizes the same, one expert of one, scales of 1, chunks of one token,
 # chunks of a page, no cap
 CFG_B = config(200, 96, [
-    layer(latent(1, 8, 8, 8, 8, 8, 1.0, 50.0), moe(40, 1, 1)),
+    layer(latent(1, 8, 8, 8, 8, 8, 0.4, 50.0), moe(40, 1, 1)),
     layer(chunked(1, 1, 8, 8, 1.0, 1, True), dense(8)),
     layer(chunked(8, 1, 8, 8, 0.5, 64, True), moe(64, 4, 1)),
-    layer(latent(2, 1, 2, 1, 1, 24, 1.0, 10000.0), dense(64))], cap=None, eps=1e-6)
+    layer(latent(2, 1, 2, 1, 4, 24, 1.0, 10000.0), dense(64))], cap=None, eps=1e-6)
 # sizes that are multiples of nothing: the bfloat16 products run on zero-padded operands, loads are scalar
 CFG_C = config(75, 36, [
     layer(latent(3, 5, 6, 7, 9, 11, 0.4, 100.0, (8.0, 32, 4.0, 1.0)), moe(13, 4, 2)),
@@ -454,8 +454,9 @@ def test_products_with_the_squared_relu_in_their_epilogue_and_behind_them():
 
 @gpu
 @pytest.mark.parametrize("H,G,d,e", [(4, 2, 16, 8), (3, 1, 5, 7), (8, 8, 128, 128), (1, 1, 8, 8), (5, 5, 9, 3)])
+@pytest.mark.parametrize("extra", [3, 4])
 @pytest.mark.parametrize("dtype", [torch.float32, torch.bfloat16])
-def test_queries_and_cache_rows_with_values_of_their_own_size_and_a_share_of_others(H, G, d, e, dtype):
+def test_queries_and_cache_rows_with_values_of_their_own_size_and_a_share_of_others(H, G, d, e, dtype, extra):
     from janus_b200.kernels import ops
     g = torch.Generator().manual_seed(3)
     T, PAGE = 9, 64
@@ -463,10 +464,12 @@ def test_queries_and_cache_rows_with_values_of_their_own_size_and_a_share_of_oth
     ep = up8(e) if dtype == torch.bfloat16 else e
     dp = max(up8(d), ep) if dtype == torch.bfloat16 else d
     tol = 1e-6 if dtype == torch.float32 else 6e-3
-    proj, other = torch.randn(T, H * d + G * (d + e) + 3, generator=g), torch.randn(T, G * e + 5, generator=g)
+    # rows wider than what is read by a whole group of four numbers or not: the kernel for groups of four, and the other one
+    proj, other = torch.randn(T, H * d + G * (d + e) + extra, generator=g), torch.randn(T, G * e + 8, generator=g)
+    off = extra if extra % 4 == 0 else 2
     dest = torch.tensor([3 * PAGE + 63, 0, 1, 2, PAGE + 7, 5, 2 * PAGE, 63, 64], dtype=torch.int32)
     v = proj[:, (H + G) * d:(H + G) * d + G * e].to(P.DT).view(T, G, e)
-    for first, mix in ((None, 0.0), (other.cuda()[:, 2:2 + G * e], 0.3)):
+    for first, mix in ((None, 0.0), (other.cuda()[:, off:off + G * e], 0.3)):
         kc = torch.zeros(4, G, PAGE, dp, dtype=dtype, device="cuda")
         vc = torch.zeros(4, G, PAGE, ep, dtype=dtype, device="cuda")
         q = torch.full((T, H * dp), 7.0, dtype=dtype, device="cuda")
@@ -476,7 +479,7 @@ def test_queries_and_cache_rows_with_values_of_their_own_size_and_a_share_of_oth
         assert rel_err(got[..., :d], proj[:, :H * d].view(T, H, d)) < tol and float(got[..., d:].abs().sum()) == 0.0
         rows = lambda c: c.transpose(1, 2).reshape(4 * PAGE, G, -1).float().cpu()      # noqa: E731
         assert rel_err(rows(kc)[dest.long()][..., :d], proj[:, H * d:(H + G) * d].view(T, G, d)) < tol
-        want = v if first is None else P.mix_values(v, other[:, 2:2 + G * e].to(P.DT).view(T, G, e), torch.tensor(0.3, dtype=P.DT))
+        want = v if first is None else P.mix_values(v, other[:, off:off + G * e].to(P.DT).view(T, G, e), torch.tensor(0.3, dtype=P.DT))
         assert rel_err(rows(vc)[dest.long()][..., :e], want) < tol
         idle = [i for i in range(4 * PAGE) if i not in dest.tolist()]
         assert float(rows(vc)[idle].abs().sum()) == 0.0 and float(rows(kc)[idle].abs().sum()) == 0.0
