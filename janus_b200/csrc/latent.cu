@@ -35,12 +35,76 @@ struct Row {                 // the token's own row: where it comes from and whe
   const int* dest;
   void* c_cache;
   void* rows;                // a second copy, row t of [T, stored] (null: none)
+  int vec;                   // n, r / 2 and stored are whole groups of four, everything lies at aligned addresses
 };
+
+template <typename TO>
+__device__ __forceinline__ void store4(TO* p, const float4& v) {
+  if constexpr (sizeof(TO) == 4) {
+    *reinterpret_cast<float4*>(p) = v;
+  } else {
+    const __nv_bfloat162 lo = __floats2bfloat162_rn(v.x, v.y), hi = __floats2bfloat162_rn(v.z, v.w);
+    uint2 u;
+    u.x = *reinterpret_cast<const uint32_t*>(&lo);
+    u.y = *reinterpret_cast<const uint32_t*>(&hi);
+    *reinterpret_cast<uint2*>(p) = u;
+  }
+}
+__device__ __forceinline__ float4 load4(const float* p) { return *reinterpret_cast<const float4*>(p); }
+__device__ __forceinline__ float squares4(const float4& v, float ss) {
+  return fmaf(v.w, v.w, fmaf(v.z, v.z, fmaf(v.y, v.y, fmaf(v.x, v.x, ss))));
+}
+__device__ __forceinline__ float4 scaled4(const float4& v, float f, const float4& w) {
+  return make_float4((v.x * f) * w.x, (v.y * f) * w.y, (v.z * f) * w.z, (v.w * f) * w.w);
+}
+// The pairs (u, v) of four neighbouring numbers and of those half a row further, turned by cs (cos and sin of the four).
+__device__ __forceinline__ void turn4(const float4& u, const float4& v, const float* cs, float4& a, float4& b) {
+  const float4 p = load4(cs), q = load4(cs + 4);
+  a = make_float4(u.x * p.x - v.x * p.y, u.y * p.z - v.y * p.w, u.z * q.x - v.z * q.y, u.w * q.z - v.w * q.w);
+  b = make_float4(v.x * p.x + u.x * p.y, v.y * p.z + u.y * p.w, v.z * q.x + u.z * q.y, v.w * q.z + u.w * q.w);
+}
+
+// One block norms, turns and writes the row of token t, four numbers a thread.
+template <typename TO>
+__device__ void write_row_vec(const float* x, const Row& row, const float* cs, int t, float* scratch) {
+  float ss = 0.0f;
+  for (int i = threadIdx.x * 4; i < row.n; i += blockDim.x * 4) ss = squares4(load4(x + i), ss);
+  ss = jb::block_sum(ss, scratch);
+  const float inv = 1.0f / sqrtf(ss / (float)row.n + row.eps);
+  TO* out = (TO*)row.c_cache + (size_t)row.dest[t] * row.stored;
+  TO* copy = row.rows != nullptr ? (TO*)row.rows + (size_t)t * row.stored : nullptr;
+  const int half = row.r >> 1;
+  auto put = [&](int i, const float4& v) {
+    store4(out + i, v);
+    if (copy != nullptr) store4(copy + i, v);
+  };
+  for (int i = threadIdx.x * 4; i < row.stored; i += blockDim.x * 4) {
+    if (i < row.n) {
+      put(i, scaled4(load4(x + i), inv, load4(row.w + i)));
+    } else if (i < row.n + row.r) {
+      const int j = i - row.n;
+      if (cs == nullptr) {
+        put(i, load4(x + i));
+      } else if (j < half) {
+        float4 a, b;
+        turn4(load4(x + i), load4(x + i + half), cs + 2 * j, a, b);
+        put(i, a);
+        put(i + half, b);
+      }
+    } else if (copy != nullptr) {
+      store4(copy + i, make_float4(0.0f, 0.0f, 0.0f, 0.0f));
+    }
+  }
+}
 
 // One block norms, turns and writes the row of token t.
 template <typename TO>
 __device__ void write_row(const float* pr, const Row& row, const float* cs, int t, float* scratch) {
   const float* x = pr + row.c_col;
+  if (row.vec) {
+    write_row_vec<TO>(x, row, cs, t, scratch);
+    return;
+  }
   float ss = 0.0f;
   for (int i = threadIdx.x; i < row.n; i += blockDim.x) ss = fmaf(x[i], x[i], ss);
   ss = jb::block_sum(ss, scratch);
@@ -67,19 +131,6 @@ __device__ void write_row(const float* pr, const Row& row, const float* cs, int 
     }
     out[i] = jb::from_f32<TO>(v);
     if (copy != nullptr) copy[i] = jb::from_f32<TO>(v);
-  }
-}
-
-template <typename TO>
-__device__ __forceinline__ void store4(TO* p, const float4& v) {
-  if constexpr (sizeof(TO) == 4) {
-    *reinterpret_cast<float4*>(p) = v;
-  } else {
-    const __nv_bfloat162 lo = __floats2bfloat162_rn(v.x, v.y), hi = __floats2bfloat162_rn(v.z, v.w);
-    uint2 u;
-    u.x = *reinterpret_cast<const uint32_t*>(&lo);
-    u.y = *reinterpret_cast<const uint32_t*>(&hi);
-    *reinterpret_cast<uint2*>(p) = u;
   }
 }
 
@@ -112,10 +163,10 @@ __global__ void __launch_bounds__(256) latent_prep_kernel(const float* __restric
       if (j < d || (j < d + r && cs == nullptr)) {
         store4(o + j, *reinterpret_cast<const float4*>(x + j));
       } else if (j < d + half) {
-        const float4 u = *reinterpret_cast<const float4*>(x + j), v = *reinterpret_cast<const float4*>(x + j + half);
-        const float4 a = *reinterpret_cast<const float4*>(cs + 2 * (j - d)), b = *reinterpret_cast<const float4*>(cs + 2 * (j - d) + 4);
-        store4(o + j, make_float4(u.x * a.x - v.x * a.y, u.y * a.z - v.y * a.w, u.z * b.x - v.z * b.y, u.w * b.z - v.w * b.w));
-        store4(o + j + half, make_float4(v.x * a.x + u.x * a.y, v.y * a.z + u.y * a.w, v.z * b.x + u.z * b.y, v.w * b.z + u.w * b.w));
+        float4 a, b;
+        turn4(load4(x + j), load4(x + j + half), cs + 2 * (j - d), a, b);
+        store4(o + j, a);
+        store4(o + j + half, b);
       } else if (j >= d + r) {
         store4(o + j, make_float4(0.0f, 0.0f, 0.0f, 0.0f));
       }
@@ -136,8 +187,9 @@ __global__ void __launch_bounds__(256) latent_prep_kernel(const float* __restric
 }
 
 // a_out[t] = x / rms(x) * w with x = proj[t, 0 : m], a block per token (blockIdx.y == 0); the token's row, another one
-// (blockIdx.y == 1).  All blocks together set the n_clear float4 at `clear` to zero.
-template <typename TO>
+// (blockIdx.y == 1).  All blocks together set the n_clear float4 at `clear` to zero.  VEC: m and ld are whole groups of
+// four at aligned addresses.
+template <typename TO, bool VEC>
 __global__ void __launch_bounds__(256) latent_down_kernel(const float* __restrict__ proj, int ld, int m,
                                                           const float* __restrict__ w, float eps, TO* __restrict__ a_out,
                                                           const float* __restrict__ table, const int* __restrict__ positions,
@@ -156,6 +208,14 @@ __global__ void __launch_bounds__(256) latent_down_kernel(const float* __restric
     return;
   }
   float ss = 0.0f;
+  if constexpr (VEC) {
+    for (int i = threadIdx.x * 4; i < m; i += blockDim.x * 4) ss = squares4(load4(x + i), ss);
+    ss = jb::block_sum(ss, scratch);
+    const float inv = 1.0f / sqrtf(ss / (float)m + eps);
+    for (int i = threadIdx.x * 4; i < m; i += blockDim.x * 4)
+      store4(a_out + (size_t)t * m + i, scaled4(load4(x + i), inv, load4(w + i)));
+    return;
+  }
   for (int i = threadIdx.x; i < m; i += blockDim.x) ss = fmaf(x[i], x[i], ss);
   ss = jb::block_sum(ss, scratch);
   const float inv = 1.0f / sqrtf(ss / (float)m + eps);
@@ -441,6 +501,13 @@ __global__ void __launch_bounds__(256) gather_rows_kernel(const uint4* __restric
 
 bool aligned16(const void* p) { return ((uintptr_t)p & 15) == 0; }
 
+Row make_row(const float* proj, int ld, const float* table, int c_col, int n, int r, int stored, const float* w, float eps,
+             const int* dest, void* c_cache, void* rows) {
+  const bool vec = ld % 4 == 0 && c_col % 4 == 0 && n % 4 == 0 && r % 8 == 0 && stored % 4 == 0 && aligned16(proj) &&
+                   aligned16(table) && aligned16(w) && aligned16(c_cache) && aligned16(rows);
+  return Row{c_col, n, r, stored, w, eps, dest, c_cache, rows, vec ? 1 : 0};
+}
+
 int check_row(int ld, int r, const Row& row) {
   JB_REFUSE(r < 0 || (r & 1), "latent: %d rotated numbers", r);
   JB_REFUSE(row.c_cache != nullptr && (ld < row.c_col + row.n + row.r || row.stored < row.n + row.r || row.n < 1 ||
@@ -464,7 +531,7 @@ JB_EXPORT int jb_latent_heads(const float* proj, int ld, int q_col, int H, int d
                               const float* w, float eps, const int* dest, void* c_cache, void* rows, int T,
                               cudaStream_t stream) {
   if (T <= 0) return 0;
-  const Row row{c_col, n, r, stored, w, eps, dest, c_cache, rows};
+  const Row row = make_row(proj, ld, table, c_col, n, r, stored, w, eps, dest, c_cache, rows);
   if (const int bad = check_queries(ld, q_col, H, d, r, row)) return bad;
   JB_REFUSE(dp < d + r, "latent_heads: heads of %d numbers cannot be stored in %d columns", d + r, dp);
   const bool vec = ld % 4 == 0 && q_col % 4 == 0 && d % 4 == 0 && r % 8 == 0 && dp % 4 == 0 && aligned16(proj) &&
@@ -493,18 +560,25 @@ JB_EXPORT int jb_latent_down(const float* proj, int ld, int m, const float* w, f
                              const int* dest, void* c_cache, void* rows, float* clear, long long n_clear, int T,
                              cudaStream_t stream) {
   if (T <= 0) return 0;
-  const Row row{c_col, n, r, stored, row_w, eps, dest, c_cache, rows};
+  const Row row = make_row(proj, ld, table, c_col, n, r, stored, row_w, eps, dest, c_cache, rows);
   JB_REFUSE(m < 1 || ld < m, "latent_down: rows of %d floats do not hold %d numbers", ld, m);
   if (const int bad = check_row(ld, r, row)) return bad;
   JB_REFUSE(clear != nullptr && (n_clear % 4 != 0 || !aligned16(clear)), "latent_down: %lld floats to clear", n_clear);
   const long long vecs = clear != nullptr ? n_clear / 4 : 0;
   jb::Launch cfg(dim3(T, c_cache != nullptr ? 2 : 1), dim3(256), 0, stream);
-  if (out_dtype == JB_F32)
-    return (int)cudaLaunchKernelEx(&cfg.c, latent_down_kernel<float>, proj, ld, m, w, eps, (float*)a_out, table, positions,
-                                   (float4*)clear, vecs, row);
-  if (out_dtype == JB_BF16)
-    return (int)cudaLaunchKernelEx(&cfg.c, latent_down_kernel<bf16>, proj, ld, m, w, eps, (bf16*)a_out, table, positions,
-                                   (float4*)clear, vecs, row);
+  const bool vec = ld % 4 == 0 && m % 4 == 0 && aligned16(proj) && aligned16(w) && aligned16(a_out);
+#define JB_GO(TO, VEC)                                                                                                    \
+  return (int)cudaLaunchKernelEx(&cfg.c, latent_down_kernel<TO, VEC>, proj, ld, m, w, eps, (TO*)a_out, table, positions, \
+                                 (float4*)clear, vecs, row)
+  if (out_dtype == JB_F32) {
+    if (vec) JB_GO(float, true);
+    JB_GO(float, false);
+  }
+  if (out_dtype == JB_BF16) {
+    if (vec) JB_GO(bf16, true);
+    JB_GO(bf16, false);
+  }
+#undef JB_GO
   return JB_ERR_BAD_DTYPE;
 }
 
@@ -514,7 +588,7 @@ JB_EXPORT int jb_latent_queries(const float* proj, int ld, int q_col, int H, int
                                 const float* table, const int* positions, void* q_out, int dtype, int c_col, int stored,
                                 const float* w, float eps, const int* dest, void* c_cache, int T, cudaStream_t stream) {
   if (T <= 0) return 0;
-  const Row row{c_col, n, r, stored, w, eps, dest, c_cache, nullptr};
+  const Row row = make_row(proj, ld, table, c_col, n, r, stored, w, eps, dest, c_cache, nullptr);
   if (const int bad = check_queries(ld, q_col, H, d, r, row)) return bad;
   JB_REFUSE(dp < n + r || n < 1 || d < 1, "latent_queries: %d + %d numbers cannot be stored in %d columns", n, r, dp);
   const int vw = dtype == JB_BF16 ? 8 : 4;

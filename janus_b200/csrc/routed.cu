@@ -75,6 +75,7 @@ __global__ void route_topk_kernel(const float* __restrict__ logits, int ld, int 
     }
   }
   int picked[MAX_TOP];
+  float mine = 0.0f;                             // lane k: the k-th weight
   for (int k = 0; k < top; ++k) {
     float best = -CUDART_INF_F;
     int arg = 0x7fffffff;
@@ -100,14 +101,11 @@ __global__ void route_topk_kernel(const float* __restrict__ logits, int ld, int 
     picked[k] = arg;
     if (lane == 0) {
       sel_e[(size_t)t * top + k] = arg;
-      if (!shares) sel_w[(size_t)t * top + k] = score(z[arg]) * scale;
     }
+    if (lane == k) mine = score(z[arg]);
   }
-  if (shares && lane == 0) {
-    float sum = 0.0f;
-    for (int k = 0; k < top; ++k) sum += score(z[picked[k]]);
-    for (int k = 0; k < top; ++k) sel_w[(size_t)t * top + k] = score(z[picked[k]]) / (sum + 1e-20f) * scale;
-  }
+  if (shares) mine = mine / (jb::warp_sum(mine) + 1e-20f);
+  if (lane < top) sel_w[(size_t)t * top + lane] = mine * scale;
 }
 
 template <typename TW> struct Vec;
