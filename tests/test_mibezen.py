@@ -526,7 +526,7 @@ def _wanted(q, k, v, scale, chunk, slopes, sinks, gate):
     return o if gate is None else o * torch.sigmoid(gate)[:, :, None]
 
 
-ATTENTION_SIZES = [(4, 2, 16, 8), (6, 2, 128, 128), (4, 2, 96, 32), (3, 1, 64, 64), (16, 1, 192, 128), (2, 2, 256, 248), (5, 5, 8, 8),
+ATTENTION_SIZES = [(4, 2, 16, 8), (6, 2, 128, 128), (6, 2, 88, 40), (3, 1, 64, 64), (16, 1, 192, 128), (2, 2, 256, 248), (5, 5, 8, 8),
                    (20, 1, 72, 40)]
 
 
