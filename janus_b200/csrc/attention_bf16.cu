@@ -184,6 +184,7 @@ struct Cap {
   const float* sinks;
   const float* gate;
   int ld_gate;
+  float inv_scale;   // 1 / scale, for the slopes
 };
 // A denominator l relative to the maximum m (in units of log2), with what a sink adds to it.
 __device__ __forceinline__ float with_sink(float l, float m, const Cap& cap, int head) {
@@ -195,19 +196,26 @@ __device__ __forceinline__ float with_sink(float l, float m, const Cap& cap, int
 __device__ __forceinline__ float head_gate(const Cap& cap, int token, int head) {
   return cap.gate == nullptr ? 1.0f : 1.0f / (1.0f + expf(-cap.gate[(size_t)token * cap.ld_gate + head]));
 }
-// The slope of a head's distance bias in units of log2(e) (0: none).
+// The slope of a head's distance bias in units of the products before they are scaled (0: none).
 __device__ __forceinline__ float head_slope(const Cap& cap, int head) {
-  return cap.slopes == nullptr ? 0.0f : cap.slopes[head] * LOG2E;
+  return cap.slopes == nullptr ? 0.0f : cap.slopes[head] * cap.inv_scale;
 }
 __device__ __forceinline__ int chunk_lo(int lo, int pos, int chunk) {
   return (chunk > 0 && pos >= 0) ? max(lo, (pos / chunk) * chunk) : lo;
 }
 
-template <int NT>
+template <int NT, bool PER_HEAD>
 __device__ __forceinline__ void softmax_pv(RowState& st, float (&s)[NT][4], const bf16* v_tile, int key_pos0,
                                            const int (&row_pos)[2], const int (&row_lo)[2], const float (&slope)[2],
                                            float scale_log2, const Cap& cap, int lane) {
   const int c = lane & 3;
+  if (PER_HEAD && cap.slopes != nullptr) {   // (never with a cap: the launches refuse both together)
+#pragma unroll
+    for (int j = 0; j < NT; ++j)
+#pragma unroll
+      for (int e = 0; e < 4; ++e)
+        s[j][e] = fmaf(slope[e >> 1], (float)(key_pos0 + j * 8 + 2 * c + (e & 1) - row_pos[e >> 1]), s[j][e]);
+  }
   float mx[2] = {-CUDART_INF_F, -CUDART_INF_F};
 #pragma unroll
   for (int j = 0; j < NT; ++j) {
@@ -217,8 +225,7 @@ __device__ __forceinline__ void softmax_pv(RowState& st, float (&s)[NT][4], cons
       const int kp = key_pos0 + j * 8 + 2 * c + (e & 1);
       const bool ok = kp <= row_pos[r] && kp >= row_lo[r];
       // with a cap c the score s becomes c tanh(s / c), here in units of log2(e)
-      float sc = cap.cap_log2 > 0.0f ? cap.cap_log2 * tanhf(s[j][e] * cap.inv_cap) : s[j][e] * scale_log2;
-      if (cap.slopes != nullptr) sc = fmaf(slope[r], (float)(kp - row_pos[r]), sc);
+      const float sc = cap.cap_log2 > 0.0f ? cap.cap_log2 * tanhf(s[j][e] * cap.inv_cap) : s[j][e] * scale_log2;
       s[j][e] = ok ? sc : -CUDART_INF_F;
       mx[r] = fmaxf(mx[r], s[j][e]);
     }
@@ -338,7 +345,7 @@ __global__ void __launch_bounds__(THREADS) prefill_kernel(
     const bf16* k_tile = kv_s + (size_t)stage * KV_STAGE;
     float s[8][4];
     qk_product<8>(s, q_s + warp * 16 * LD, k_tile, lane);
-    softmax_pv<8>(st, s, k_tile + K_TILE, kb * PAGE, row_pos, row_lo, slope, scale_log2, cap, lane);
+    softmax_pv<8, true>(st, s, k_tile + K_TILE, kb * PAGE, row_pos, row_lo, slope, scale_log2, cap, lane);
     __syncthreads();
   }
 #pragma unroll
@@ -391,7 +398,9 @@ __device__ __forceinline__ void rotate_pair(float x0, float x1, const float* cs,
 }
 
 // part_o: [seq][head][split][VD] float32 (unnormalised), part_ml: [seq][head][split][2] (max, sum).
-template <int DECODE_STAGES>
+// PER_HEAD: there may be slopes, sinks, a gate or values to mix in (a build of its own: the plain one stays as lean as it
+// can be).
+template <int DECODE_STAGES, bool PER_HEAD>
 __global__ void __launch_bounds__(THREADS) decode_kernel(
     const bf16* __restrict__ q, const bf16* __restrict__ k_cache, const bf16* __restrict__ v_cache,
     bf16* __restrict__ out, float* __restrict__ part_o, float* __restrict__ part_ml,
@@ -490,11 +499,18 @@ __global__ void __launch_bounds__(THREADS) decode_kernel(
       if (patch_new) {
         const float* kx = row + (size_t)(nh + kvh) * HD;
         const float* vx = row + (size_t)(nh + nkv) * HD + (size_t)kvh * VD;
-        const float* v1st = fused.first != nullptr ? fused.first + (size_t)seq * fused.first_stride + (size_t)kvh * VD : nullptr;
+        const float* v1st = PER_HEAD && fused.first != nullptr ? fused.first + (size_t)seq * fused.first_stride + (size_t)kvh * VD : nullptr;
         const int dst = fused.dest[seq];
         const size_t g_row = ((size_t)(dst / PAGE) * nkv + kvh) * PAGE + dst % PAGE;
         bf16* k_out = fused.k_out + g_row * HD;
         bf16* v_out = fused.v_out + g_row * VD;
+        // (the value's numbers are asked for before the key's are stored)
+        float v_new[(VD + THREADS - 1) / THREADS];
+#pragma unroll
+        for (int u = 0; u < (VD + THREADS - 1) / THREADS; ++u) {
+          const int i = min((int)threadIdx.x + u * THREADS, VD - 1);
+          v_new[u] = v1st != nullptr ? (1.0f - fused.mix) * vx[i] + fused.mix * v1st[i] : vx[i];
+        }
         for (int i = threadIdx.x; i < HALF; i += THREADS) {
           float y0, y1;
           rotate_pair(kx[i], kx[i + HALF], cs, i, y0, y1);
@@ -504,10 +520,14 @@ __global__ void __launch_bounds__(THREADS) decode_kernel(
             k_out[i] = k0; k_out[i + HALF] = k1;
           }
         }
-        for (int i = threadIdx.x; i < VD; i += THREADS) {
-          const bf16 v = __float2bfloat16_rn(v1st != nullptr ? (1.0f - fused.mix) * vx[i] + fused.mix * v1st[i] : vx[i]);
-          new_kv[LD + i] = v;
-          if (rb == 0) v_out[i] = v;
+#pragma unroll
+        for (int u = 0; u < (VD + THREADS - 1) / THREADS; ++u) {
+          const int i = threadIdx.x + u * THREADS;
+          const bf16 v = __float2bfloat16_rn(v_new[u]);
+          if (i < VD) {
+            new_kv[LD + i] = v;
+            if (rb == 0) v_out[i] = v;
+          }
         }
       }
     }
@@ -518,7 +538,7 @@ __global__ void __launch_bounds__(THREADS) decode_kernel(
       const int head_row = (lane >> 2) + 8 * r;
       row_pos[r] = head_row < n_rows ? pos : -1;
       row_lo[r] = lo;
-      slope[r] = head_slope(cap, kvh * G + g0 + min(head_row, n_rows - 1));
+      slope[r] = PER_HEAD ? head_slope(cap, kvh * G + g0 + min(head_row, n_rows - 1)) : 0.0f;
     }
     __syncthreads();  // q (and the new key and value) are in shared memory for every warp
     for (int kb = kb_start; kb <= kb_end; ++kb) {
@@ -540,7 +560,7 @@ __global__ void __launch_bounds__(THREADS) decode_kernel(
       // this warp's 16 keys of the page
       float s[2][4];
       qk_product<2>(s, q_s, k_tile + warp * 16 * LD, lane);
-      softmax_pv<2>(st, s, k_tile + K_TILE + warp * 16 * LDV, kb * PAGE + warp * 16, row_pos, row_lo, slope,
+      softmax_pv<2, PER_HEAD>(st, s, k_tile + K_TILE + warp * 16 * LDV, kb * PAGE + warp * 16, row_pos, row_lo, slope,
                     scale_log2, cap, lane);
       __syncwarp();  // the warp is done with its rows of this stage before its next loads overwrite them
     }
@@ -584,7 +604,9 @@ __global__ void __launch_bounds__(THREADS) decode_kernel(
     }
     const int head = kvh * G + g0 + row;
     if (n_splits == 1) {
-      out[((size_t)seq * nh + head) * VD + d] = __float2bfloat16_rn(o / with_sink(l, m, cap, head) * head_gate(cap, seq, head));
+      out[((size_t)seq * nh + head) * VD + d] = __float2bfloat16_rn(
+          PER_HEAD ? o / with_sink(l, m, cap, head) * head_gate(cap, seq, head)
+                   : o / (cap.sink > 0.0f ? l + cap.sink * exp2f(-m_use) : l));
     } else {
       const size_t base = ((size_t)seq * nh + head) * n_splits + split;
       part_o[base * VD + d] = o;
@@ -596,16 +618,17 @@ __global__ void __launch_bounds__(THREADS) decode_kernel(
   }
 }
 
+template <bool PER_HEAD>
 __global__ void decode_combine_kernel(const float* __restrict__ part_o, const float* __restrict__ part_ml,
-                                      bf16* __restrict__ out, int n_splits, int nh, Cap cap) {
+                                      bf16* __restrict__ out, int n_splits, Cap cap) {
   jb::pdl_launch_dependents();
   jb::pdl_wait();
-  const size_t item = blockIdx.x;  // seq * nh + head
-  const int head = (int)(item % nh);
+  const int head = blockIdx.x, seq = blockIdx.y;
+  const size_t item = (size_t)seq * gridDim.x + head;
   const float* ml = part_ml + item * n_splits * 2;
   float m = -CUDART_INF_F;
   for (int s = 0; s < n_splits; ++s) m = fmaxf(m, ml[2 * s]);
-  const float open = head_gate(cap, (int)(item / nh), head);
+  const float open = PER_HEAD ? head_gate(cap, seq, head) : 1.0f;
   for (int d = threadIdx.x; d < VD; d += blockDim.x) {
     float o = 0.0f, l = 0.0f;
     for (int s = 0; s < n_splits; ++s) {
@@ -613,7 +636,9 @@ __global__ void decode_combine_kernel(const float* __restrict__ part_o, const fl
       o += part_o[(item * n_splits + s) * VD + d] * f;
       l += ml[2 * s + 1] * f;
     }
-    out[item * VD + d] = __float2bfloat16_rn(o / with_sink(l, m, cap, head) * open);
+    if constexpr (PER_HEAD) l = with_sink(l, m, cap, head);
+    else if (cap.sink > 0.0f) l += cap.sink * exp2f(m == -CUDART_INF_F ? 0.0f : -m);
+    out[item * VD + d] = __float2bfloat16_rn(PER_HEAD ? o / l * open : o / l);
   }
 }
 
@@ -643,23 +668,23 @@ int decode_stages_for(long long ctas, int pages_per_cta) {
   return 3;
 }
 
-template <int ST>
+template <int ST, bool PER_HEAD>
 cudaError_t decode_go(dim3 grid, cudaStream_t stream, bool pdl, const bf16* q, const bf16* k_cache, const bf16* v_cache,
                       bf16* out, float* part_o, float* part_ml, const int* block_table, const int* kv_len, int nh,
                       int nkv, int max_pages, int window, float scale_log2, int n_splits, const FusedInput& fused,
                       const Cap& cap) {
-  static bool configured = false;   // one flag per ring depth
+  static bool configured = false;   // one flag per build
   if (!configured) {
-    cudaError_t e = cudaFuncSetAttribute(decode_kernel<ST>, cudaFuncAttributeMaxDynamicSharedMemorySize, decode_smem(ST));
+    cudaError_t e = cudaFuncSetAttribute(decode_kernel<ST, PER_HEAD>, cudaFuncAttributeMaxDynamicSharedMemorySize, decode_smem(ST));
     if (e != cudaSuccess) return e;
     configured = true;
   }
   if (pdl) {
     jb::Launch cfg(grid, dim3(THREADS), decode_smem(ST), stream);
-    return cudaLaunchKernelEx(&cfg.c, decode_kernel<ST>, q, k_cache, v_cache, out, part_o, part_ml, block_table, kv_len,
+    return cudaLaunchKernelEx(&cfg.c, decode_kernel<ST, PER_HEAD>, q, k_cache, v_cache, out, part_o, part_ml, block_table, kv_len,
                               nh, nkv, max_pages, window, scale_log2, n_splits, fused, cap);
   }
-  decode_kernel<ST><<<grid, THREADS, decode_smem(ST), stream>>>(q, k_cache, v_cache, out, part_o, part_ml, block_table,
+  decode_kernel<ST, PER_HEAD><<<grid, THREADS, decode_smem(ST), stream>>>(q, k_cache, v_cache, out, part_o, part_ml, block_table,
                                                                kv_len, nh, nkv, max_pages, window, scale_log2, n_splits,
                                                                fused, cap);
   return cudaGetLastError();
@@ -672,9 +697,13 @@ cudaError_t decode_dispatch(dim3 grid, cudaStream_t stream, bool pdl, const bf16
                             int n_splits, const FusedInput& fused, const Cap& cap = Cap{}) {
   const long long ctas = (long long)grid.x * grid.y * grid.z;
   const int stages = decode_stages_for(ctas, max(1, max_pages / max(1, n_splits)));
-#define JB_DECODE_GO(ST)                                                                                      \
-  return decode_go<ST>(grid, stream, pdl, q, k_cache, v_cache, out, part_o, part_ml, block_table, kv_len, nh, nkv, \
-                       max_pages, window, scale_log2, n_splits, fused, cap)
+  const bool per_head = cap.slopes != nullptr || cap.sinks != nullptr || cap.gate != nullptr || fused.first != nullptr;
+#define JB_DECODE_GO_AS(ST, PER_HEAD)                                                                             \
+  return decode_go<ST, PER_HEAD>(grid, stream, pdl, q, k_cache, v_cache, out, part_o, part_ml, block_table, kv_len, nh, \
+                                 nkv, max_pages, window, scale_log2, n_splits, fused, cap)
+#define JB_DECODE_GO(ST)                   \
+  if (per_head) JB_DECODE_GO_AS(ST, true); \
+  JB_DECODE_GO_AS(ST, false)
   switch (stages) {
     case 2: JB_DECODE_GO(2);
     case 5: JB_DECODE_GO(5);
@@ -684,6 +713,7 @@ cudaError_t decode_dispatch(dim3 grid, cudaStream_t stream, bool pdl, const bf16
     default: JB_DECODE_GO(3);
   }
 #undef JB_DECODE_GO
+#undef JB_DECODE_GO_AS
 }
 
 }  // namespace
@@ -694,7 +724,8 @@ namespace {
 Cap make_cap(int chunk, float softcap, float scale, float sink, const float* slopes, const float* sinks, const float* gate,
              int ld_gate) {
   const bool capped = softcap > 0.0f;
-  return Cap{chunk, capped ? softcap * LOG2E : 0.0f, capped ? scale / softcap : 0.0f, sink, slopes, sinks, gate, ld_gate};
+  return Cap{chunk, capped ? softcap * LOG2E : 0.0f, capped ? scale / softcap : 0.0f, sink, slopes, sinks, gate, ld_gate,
+             1.0f / scale};
 }
 
 int prefill_launch(const void* q, const void* k_cache, const void* v_cache, void* out,
@@ -741,6 +772,7 @@ JB_EXPORT int jb_attention_bf16_prefill_capped(const void* q, const void* k_cach
                                                int max_pages, int window, float scale, int chunk, float softcap,
                                                float sink, const float* slopes, const float* sinks, const float* gate,
                                                int ld_gate, cudaStream_t stream) {
+  JB_REFUSE(softcap > 0.0f && slopes != nullptr, "attention_bf16: scores are capped or take a distance bias, not both");
   return prefill_launch(q, k_cache, v_cache, out, block_table, q_start, kv_len, n_seqs, max_q_len, nh, nkv, hd,
                         page_size, max_pages, window, scale,
                         make_cap(chunk, softcap, scale, sink, slopes, sinks, gate, ld_gate), stream);
@@ -766,9 +798,10 @@ int decode_launch(const void* q, const void* k_cache, const void* v_cache, void*
                                    scale * LOG2E, n_splits, fused, cap);
   if (le != cudaSuccess) return (int)le;
   if (n_splits > 1) {
-    jb::Launch cfg2(dim3(n_seqs * nh), dim3(VD >= 128 ? 128 : 64), 0, stream);
-    le = cudaLaunchKernelEx(&cfg2.c, decode_combine_kernel, (const float*)part_o, (const float*)part_ml, (bf16*)out,
-                            n_splits, nh, cap);
+    jb::Launch cfg2(dim3(nh, n_seqs), dim3(VD >= 128 ? 128 : 64), 0, stream);
+    const bool per_head = cap.slopes != nullptr || cap.sinks != nullptr || cap.gate != nullptr;
+    le = cudaLaunchKernelEx(&cfg2.c, per_head ? decode_combine_kernel<true> : decode_combine_kernel<false>,
+                            (const float*)part_o, (const float*)part_ml, (bf16*)out, n_splits, cap);
     if (le != cudaSuccess) return (int)le;
   }
   return 0;
@@ -791,6 +824,7 @@ JB_EXPORT int jb_attention_bf16_decode_capped(const void* q, const void* k_cache
                                               int max_pages, int window, float scale, int n_splits, int chunk,
                                               float softcap, float sink, const float* slopes, const float* sinks,
                                               const float* gate, int ld_gate, cudaStream_t stream) {
+  JB_REFUSE(softcap > 0.0f && slopes != nullptr, "attention_bf16: scores are capped or take a distance bias, not both");
   return decode_launch(q, k_cache, v_cache, out, part_o, part_ml, block_table, kv_len, n_seqs, nh, nkv, hd,
                        page_size, max_pages, window, scale, n_splits, FusedInput{}, stream,
                        make_cap(chunk, softcap, scale, sink, slopes, sinks, gate, ld_gate));
@@ -810,6 +844,7 @@ JB_EXPORT int jb_attention_bf16_decode_fused(const float* qkv, int qkv_stride, c
                                              int n_splits, int write_kv, int chunk, float softcap, float sink,
                                              const float* slopes, const float* sinks, const float* gate, int ld_gate,
                                              const float* first, int first_stride, float mix, cudaStream_t stream) {
+  JB_REFUSE(softcap > 0.0f && slopes != nullptr, "attention_bf16: scores are capped or take a distance bias, not both");
   JB_REFUSE(qkv == nullptr || (write_kv && dest == nullptr), "attention_bf16 fused decode: missing input");
   JB_REFUSE(hd % 2 != 0, "attention_bf16 fused decode: head_dim %d must be even for the rotation", hd);
   FusedInput fused{qkv, qkv_stride, cos_sin, dest, (bf16*)k_cache, (bf16*)v_cache, write_kv, first, first_stride, mix};
@@ -879,7 +914,7 @@ JB_EXPORT int jb_attention_bf16_decode_noalloc(const void* q, const void* k_cach
                       FusedInput{});
   if (e != cudaSuccess) return (int)e;
   if (n_splits > 1) {
-    decode_combine_kernel<<<n_seqs * nh, VD >= 128 ? 128 : 64, 0, stream>>>(part_o, part_ml, (bf16*)out, n_splits, nh, Cap{});
+    decode_combine_kernel<false><<<dim3(nh, n_seqs), VD >= 128 ? 128 : 64, 0, stream>>>(part_o, part_ml, (bf16*)out, n_splits, Cap{});
     JB_CHECK_LAUNCH();
   }
   return 0;

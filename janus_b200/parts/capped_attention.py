@@ -63,6 +63,8 @@ class CappedAttention(Mixer):
             raise ValueError(f"a gate is True, False or 'head', a sink True, False or 'learned', got {gate!r}, {sink!r}")
         if value_mix not in (None, "first", "mix"):
             raise ValueError(f"value_mix is None, 'first' or 'mix', got {value_mix!r}")
+        if slopes is not None and softcap > 0.0:
+            raise ValueError("scores are capped or take a distance bias, not both")
         if slopes is not None and len(slopes) != num_heads:
             raise ValueError(f"{len(slopes)} slopes do not fit {num_heads} heads")
         self.qk_norm, self.gate, self.head_gate = qk_norm is True, gate is not False, gate == "head"
